@@ -1,7 +1,7 @@
 // common.cuh - sm_100a PTX helpers shared by the Dia decode kernels.
 //
-// mbarrier + 1-D bulk async copy (TMA engine, SASS UBLKCP) for the weight /
-// KV stream, packed fp32x2 FMA (SASS FFMA2), L2-only loads for data other CTAs
+// mbarrier + 1-D bulk async copy (TMA engine) for the weight /
+// KV stream, packed fp32x2 FMA, L2-only loads for data other CTAs
 // wrote, watchdog-bounded waits (a hang on a shared GPU box is never acceptable:
 // every spin has a cycle budget, after which the kernel records an error code
 // and traps).

@@ -1,5 +1,5 @@
 // icache_bench.cu - what does instruction footprint cost on B200?
-// N distinct straight-line blocks of ~2 KB SASS each are executed round-robin by 8 warps of one CTA per SM;
+// N distinct straight-line blocks of ~2 KB of code each are executed round-robin by 8 warps of one CTA per SM;
 // prints cycles per block as the total footprint grows past the instruction caches.
 #include <cstdio>
 #include <cuda_runtime.h>
