@@ -12,15 +12,15 @@ from pathlib import Path
 from . import build as _build
 
 MIXER_SINK_ATTENTION, MIXER_TALK_ATTENTION, MIXER_HGRN2, MIXER_CHANNEL_DELTA, MIXER_LATENT_ATTENTION, MIXER_MLSTM = 1, 2, 3, 4, 5, 6
-MIXER_GATED_DELTA, MIXER_RETENTION = 7, 8
+MIXER_GATED_DELTA, MIXER_RETENTION, MIXER_ROTARY_ATTENTION, MIXER_GATED_LINEAR, MIXER_MAMBA2, MIXER_PAIR = 7, 8, 9, 10, 11, 12
 FF_NONE, FF_ROUTED_EXPERTS, FF_DENSE = 0, 1, 2
 NORM_DYT, NORM_LAYER, NORM_RMS = 0, 1, 2
 FORM_SEQUENTIAL, FORM_PARALLEL, FORM_STREAMS = 0, 1, 2
-ACT_SILU_GLU, ACT_XIELU, ACT_CLAMPED_GLU, ACT_RELU2 = 0, 1, 2, 3
+ACT_SILU_GLU, ACT_XIELU, ACT_CLAMPED_GLU, ACT_RELU2, ACT_GELU_GLU = 0, 1, 2, 3, 4
 ROUTER_SIGMOID_INPUT, ROUTER_SOFTMAX_TOP, ROUTER_SOFTMAX_GROUPED = 0, 1, 2
 GATE_SIGMOID, GATE_NONE, GATE_SILU = 0, 1, 2
 ROT_INTERLEAVED, ROT_HALF = 0, 1
-ABI_VERSION = 4
+ABI_VERSION = 5
 PRECISION_FP32, PRECISION_BF16 = 0, 1
 E_OK, E_INVAL, E_CUDA, E_NOMEM, E_UNSUPPORTED = 0, -1, -2, -3, -5
 
@@ -51,7 +51,11 @@ class Layer(C.Structure):
                 # further mechanisms of the stream form
                 ("parallel", _i), ("mixer_gate", _i), ("rot_layout", _i), ("rot_dim", _i), ("head_decay", _vp),
                 ("identity_experts", _i), ("group_count", _i), ("group_keep", _i), ("route_scale", _f), ("route_correction", _vp),
-                ("shared_gate", _i)]
+                ("shared_gate", _i),
+                # more mixers, two mixers side by side, the token input
+                ("rot_amp", _f), ("values_are_keys", _i), ("decay_tau", _f), ("conv_b", _vp), ("skip_d", _vp), ("norm_groups", _i),
+                ("part", _vp * 2), ("part_scale", _f * 2), ("side_dim", _i), ("side_ld", _i), ("side_off", _i), ("side_table", _vp),
+                ("w_side_gate", _vp), ("w_side_proj", _vp), ("side_norm", _vp)]
 
 
 class Model(C.Structure):
@@ -75,6 +79,7 @@ _SIGNATURES = {
     "lm_b200_op_attention": (_ci, [_vp, _ci, _vp, _vp, _ci, _ci, _vp, _vp]),
     "lm_b200_op_mixer_kernels": (_ci, [_vp, _ci, _vp, _vp, _ci, _ci, _vp, _vp]),
     "lm_b200_op_ff": (_ci, [_vp, _ci, _vp, _ci, _vp, _vp]),
+    "lm_b200_op_token_input": (_ci, [_vp, _ci, _vp, _vp, _ci, _vp, _vp]),
     "lm_b200_op_linear": (_ci, [_vp, _vp, _vp, _ci, _ci, _ci, _vp]),
     "lm_b200_op_linear_tc": (_ci, [_vp, _vp, _vp, _vp, _ci, _ci, _ci, _vp]),
     "lm_b200_argmax_rows": (_ci, [_vp, _ci, _ci, _vp, _vp]),

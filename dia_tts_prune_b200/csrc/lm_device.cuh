@@ -5,6 +5,7 @@
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
 #include <math_constants.h>
+#include <stdint.h>
 
 namespace lm {
 namespace {
@@ -48,15 +49,61 @@ __device__ __forceinline__ float softplusf_(float z) { return z > 20.f ? z : log
 
 // activation of a gated unit on its gate g and up u products.  kGluSilu: silu(g) u.  kGluClamped: both are clamped first
 // (g from above, u on both sides), the gate's sigmoid is 1.702 times steeper and the up branch is offset by one:
-// g' sigmoid(1.702 g') (u' + 1)
-constexpr int kGluSilu = 0, kGluClamped = 1;
+// g' sigmoid(1.702 g') (u' + 1).  kGluGelu: gelu(g) u with the tanh form of gelu
+constexpr int kGluSilu = 0, kGluClamped = 1, kGluGelu = 2;
+__device__ __forceinline__ float gelu_tanhf_(float z) {
+    return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * fmaf(0.044715f * z * z, z, z)));
+}
 __device__ __forceinline__ float glu_act(int kind, float g, float u, float limit) {
     if (kind == kGluClamped) {
         g = fminf(g, limit);
         u = fminf(fmaxf(u, -limit), limit);
         return g * sigmoidf_(1.702f * g) * (u + 1.0f);
     }
-    return siluf_(g) * u;
+    return (kind == kGluGelu ? gelu_tanhf_(g) : siluf_(g)) * u;
+}
+
+// one warp's dot product of a bf16 weight row with an fp32 activation row (x sc), 16 bytes of weights per lane and load;
+// every lane gets the sum
+// wait_first: the first weight loads go out before pdl_wait, the activations are read after it
+__device__ __forceinline__ float warp_dot(const float* __restrict__ arow, const __nv_bfloat16* __restrict__ wrow, int K, int lda,
+                                          float sc, int lane, bool wait_first = false) {
+    float acc = 0.f;
+    const bool vec = (K % 8 == 0) && (lda % 4 == 0) && ((reinterpret_cast<uintptr_t>(wrow) & 15) == 0) &&
+                     ((reinterpret_cast<uintptr_t>(arow) & 15) == 0);
+    if (vec) {
+        // eight 16-byte weight loads per lane in flight before their products (the sum keeps its order: k ascending)
+        for (int k0 = lane * 8; k0 < K; k0 += 2048) {
+            uint4 wv[8];
+#pragma unroll
+            for (int u = 0; u < 8; ++u) {
+                const int k = k0 + 256 * u;
+                wv[u] = k < K ? *reinterpret_cast<const uint4*>(wrow + k) : make_uint4(0u, 0u, 0u, 0u);
+            }
+            if (wait_first) { pdl_wait(); wait_first = false; }
+#pragma unroll
+            for (int u = 0; u < 8; ++u) {
+                const int k = k0 + 256 * u;
+                if (k >= K) break;
+                const float4 x0 = *reinterpret_cast<const float4*>(arow + k);
+                const float4 x1 = *reinterpret_cast<const float4*>(arow + k + 4);
+                const __nv_bfloat162* p = reinterpret_cast<const __nv_bfloat162*>(&wv[u]);
+                acc = fmaf(x0.x * sc, __low2float(p[0]), acc);
+                acc = fmaf(x0.y * sc, __high2float(p[0]), acc);
+                acc = fmaf(x0.z * sc, __low2float(p[1]), acc);
+                acc = fmaf(x0.w * sc, __high2float(p[1]), acc);
+                acc = fmaf(x1.x * sc, __low2float(p[2]), acc);
+                acc = fmaf(x1.y * sc, __high2float(p[2]), acc);
+                acc = fmaf(x1.z * sc, __low2float(p[3]), acc);
+                acc = fmaf(x1.w * sc, __high2float(p[3]), acc);
+            }
+        }
+    } else {
+        if (wait_first) pdl_wait();
+        for (int k = lane; k < K; k += 32) acc = fmaf(arow[k] * sc, bf(wrow[k]), acc);
+    }
+    if (wait_first) pdl_wait();                               // (K == 0: nothing was loaded)
+    return warp_sum(acc);
 }
 
 // the kernels of a short step are launched with programmatic stream serialization (see pdl_release / pdl_wait)

@@ -51,6 +51,16 @@
 //   latent attention with a turned key part and a window: the cached row is [latent | turned key part]; the latent-space
 //                     query of a head is [q_plain^T W_uk | q_turned] (head_linear + rot_rows); the attention sees the last
 //                     `window` rows
+// Three more mixers, any two of which may also stand side by side in one record (a pair: one stacked input projection, each
+// mixer's kernels on its own columns, their outputs weighted and side by side in front of one output projection):
+//   rotary attention: per-head q / k norms, rotary positions, the projected keys (raw) as values (talk_prep); sliding window and
+//                     sink (sink_attention, the kernels of the sequential form)
+//   gated linear attention: second step of the decay projection with its sigmoid^(1 / tau) (decay_proj); S <- diag(a) S + k v^T
+//                     (column_scan with the write rule); per-head RMS norm x silu(gate) (head_norm_gate)
+//   state-space mixer: convolution, silu, step sizes, decays (ssm_prep); tails (conv_tail); the recurrence with B / C shared by
+//                     groups of heads and the skip term (scalar_gate_scan); gate, then the grouped norm (gate_norm)
+// A record may end with a token input:  x += rms(W_proj (gelu(W_gate x) * e)) w with e the token's slice of a second table
+//   (one streams_step writes what is pending, linear | side_gate_rows, side_act, linear; the next streams_step norms and adds)
 // A PARALLEL stream record lets both sublayers read the streams before either writes: the mixer's output waits in a buffer
 // of its own, and one streams_step writes both outputs (and, with one stream, gave both sublayers their inputs: two norm
 // weights on the same statistics).  The feed-forward may also be a dense squared-relu unit, and the mixture may route by
@@ -135,6 +145,10 @@ struct lm_b200_engine {
     // records whose sublayers read the same streams: the mixer's output beside the feed-forward's, and the feed-forward's input
     float *ymix, *h2;
     void* h2b;
+    // the token input: gate products, their activated form (fp32, bf16 operand)
+    float *side_z, *side_g;
+    void* side_gb;
+    std::vector<lm_b200_layer> parts_of_pairs;   // copies of the parts of pair records (layers[i].part points here)
     bool stream_form = false;
     float* split_ws;                             // partial results of the key splits of a few rows' attention
     unsigned* split_arrived;                     // ... and their arrival counters (zero between launches)
@@ -236,7 +250,7 @@ int check_parallel_layer(const lm_b200_model& m, const lm_b200_layer& l) {
 }
 
 // columns of the stacked projections of a stream record (gate < 0: the mixer has no gate columns)
-struct StreamCols { int q, k, v, ig, fg, gate, lat_q, lat_c, beta, a, n; };
+struct StreamCols { int q, k, v, ig, fg, gate, lat_q, lat_c, beta, a, z, x, a1, n; };
 StreamCols stream_cols(const lm_b200_layer& l) {
     StreamCols c{};
     const int H = l.heads, G = l.kv_heads, d = l.dim, dv = l.vdim;
@@ -245,13 +259,19 @@ StreamCols stream_cols(const lm_b200_layer& l) {
         c.lat_q = at; at += l.q_rank; c.lat_c = at; at += l.kv_rank + l.rot_dim;   // the latent, then the turned key part
     } else if (l.mixer == LM_B200_MIXER_GATED_DELTA) {
         c.q = at; at += G * d; c.k = at; at += G * d; c.v = at; at += H * dv; c.beta = at; at += H; c.a = at; at += H;
-    } else if (l.mixer == LM_B200_MIXER_RETENTION) {
+    } else if (l.mixer == LM_B200_MIXER_RETENTION || l.mixer == LM_B200_MIXER_GATED_LINEAR) {
         c.q = at; at += H * d; c.k = at; at += H * d; c.v = at; at += H * dv;
+    } else if (l.mixer == LM_B200_MIXER_ROTARY_ATTENTION) {
+        c.q = at; at += H * d; c.k = at; at += G * d; c.v = c.k;
+        if (!l.values_are_keys) { c.v = at; at += G * dv; }
+    } else if (l.mixer == LM_B200_MIXER_MAMBA2) {
+        c.z = at; at += H * dv; c.x = at; at += H * dv + 2 * G * d + H;
     } else {
         c.q = at; at += H * d; c.k = at; at += H * d; c.v = at; at += H * dv; c.ig = at; at += H; c.fg = at; at += H;
     }
     c.gate = -1;
     if (l.mixer_gate != LM_B200_GATE_NONE) { c.gate = at; at += H * dv; }
+    if (l.mixer == LM_B200_MIXER_GATED_LINEAR) { c.a1 = at; at += l.rank_a; }
     c.n = (at + 3) & ~3;
     return c;
 }
@@ -259,23 +279,36 @@ StreamCols stream_cols(const lm_b200_layer& l) {
 lm::TalkShape latent_shape(const lm_b200_layer& l) {
     return lm::TalkShape{l.heads, 1, l.kv_rank + l.rot_dim, l.kv_rank, 0, 1.f, nullptr, nullptr, l.sink, l.window > 0 ? l.window : 0};
 }
-// row of the recurrence inputs of a gated delta record: q | k | v | decay | beta
-int delta_rec_cols(const lm_b200_layer& l) {
-    return l.mixer == LM_B200_MIXER_GATED_DELTA ? 2 * l.kv_heads * l.dim + l.heads * l.vdim + 2 * l.heads : 0;
+// the mixers of a stream record: one, or the two parts of a pair
+int n_parts(const lm_b200_layer& l) { return l.mixer == LM_B200_MIXER_PAIR ? 2 : 1; }
+const lm_b200_layer& part_of(const lm_b200_layer& l, int q) { return l.mixer == LM_B200_MIXER_PAIR ? *l.part[q] : l; }
+// columns of a record's mixer output (the operand of its output projection)
+int mix_out_cols(const lm_b200_layer& l) {
+    int n = 0;
+    for (int q = 0; q < n_parts(l); ++q) n += part_of(l, q).heads * part_of(l, q).vdim;
+    return n;
 }
+// row of the recurrence inputs: gated delta q | k | v | decay | beta; gated linear attention decay (heads x dim); state-space mixer
+// x | B | C | decay | step size
+int stream_rec_cols(const lm_b200_layer& l) {
+    switch (l.mixer) {
+        case LM_B200_MIXER_GATED_DELTA:
+        case LM_B200_MIXER_MAMBA2: return 2 * l.kv_heads * l.dim + l.heads * l.vdim + 2 * l.heads;
+        case LM_B200_MIXER_GATED_LINEAR: return l.heads * l.dim;
+        default: return 0;
+    }
+}
+int glu_kind(int act) { return act == LM_B200_ACT_CLAMPED_GLU ? 1 : act == LM_B200_ACT_GELU_GLU ? 2 : 0; }
 bool stream_norm_ok(const lm_b200_norm& n) { return n.w && (n.kind == LM_B200_NORM_LAYER || n.kind == LM_B200_NORM_RMS); }
 // router outputs of a record and the columns of its logits (the shared unit's gate row behind them)
 int route_outputs(const lm_b200_layer& l) { return l.experts + (l.router == LM_B200_ROUTER_SOFTMAX_GROUPED ? l.identity_experts : 0); }
 int route_cols(const lm_b200_layer& l) { return route_outputs(l) + (l.router == LM_B200_ROUTER_SOFTMAX_GROUPED && l.shared_gate ? 1 : 0); }
 
-int check_stream_layer(const lm_b200_model& m, const lm_b200_layer& l) {
-    if (l.streams < 1 || l.streams > 8) return LM_B200_EUNSUPPORTED;
-    if (!stream_norm_ok(l.norm_mix_in)) return LM_B200_EINVAL;
-    if (l.heads <= 0 || l.dim <= 0 || l.vdim <= 0 || !l.w_in || !l.w_o || l.n_in != stream_cols(l).n) return LM_B200_EINVAL;
+// one mixer of a stream record (not a pair)
+int check_stream_mixer(const lm_b200_layer& l) {
+    if (l.heads <= 0 || l.dim <= 0 || l.vdim <= 0 || l.n_in != stream_cols(l).n) return LM_B200_EINVAL;
     if (l.mixer_gate != LM_B200_GATE_SIGMOID && l.mixer_gate != LM_B200_GATE_NONE && l.mixer_gate != LM_B200_GATE_SILU)
         return LM_B200_EINVAL;
-    for (int q = 0; q < (l.ff == LM_B200_FF_NONE ? 1 : 2); ++q)
-        if (!l.hc_in[q] || !l.hc_out[q] || !l.hc_mix[q]) return LM_B200_EINVAL;
     const bool rot_ok = l.rot_dims >= 0 && l.rot_dims % 2 == 0 && (l.rot_dims == 0 || l.rot_freq) &&
                         (l.rot_layout == LM_B200_ROT_INTERLEAVED || l.rot_layout == LM_B200_ROT_HALF);
     switch (l.mixer) {
@@ -302,13 +335,49 @@ int check_stream_layer(const lm_b200_model& m, const lm_b200_layer& l) {
             if (!l.rec_state || !l.head_decay || !rot_ok || l.rot_dims > l.dim) return LM_B200_EINVAL;
             if (l.dim > 256 || l.heads > 32767) return LM_B200_EUNSUPPORTED;
             break;
+        case LM_B200_MIXER_ROTARY_ATTENTION:
+            if (l.kv_heads <= 0 || l.heads % l.kv_heads || l.vdim != l.dim || !l.q_norm || !l.k_norm || !l.k_pages || !l.v_pages || !rot_ok ||
+                l.rot_dims > l.dim || l.mixer_gate != LM_B200_GATE_NONE)
+                return LM_B200_EINVAL;
+            if (l.dim > 256 || l.heads > 65535 || l.rot_layout != LM_B200_ROT_INTERLEAVED) return LM_B200_EUNSUPPORTED;
+            break;
+        case LM_B200_MIXER_GATED_LINEAR:
+            if (l.kv_heads != l.heads || !l.head_norm || !l.rec_state || !l.w_a2 || l.rank_a <= 0 || !(l.decay_tau > 0.f)) return LM_B200_EINVAL;
+            if (l.dim > 256 || l.heads > 65535 || l.rank_a > 1024) return LM_B200_EUNSUPPORTED;
+            break;
+        case LM_B200_MIXER_MAMBA2:
+            if (l.kv_heads <= 0 || l.heads % l.kv_heads || !l.head_norm || !l.rec_state || !l.conv_w || !l.a_log || !l.dt_bias || !l.skip_d ||
+                l.conv_taps < 1 || (l.conv_taps > 1 && !l.conv_tail) || l.norm_groups < 1 || (l.heads * l.vdim) % l.norm_groups ||
+                l.mixer_gate != LM_B200_GATE_NONE)
+                return LM_B200_EINVAL;
+            if (l.dim > 256 || l.heads > 65535 || l.norm_groups > 65535 || l.conv_taps > lm::kMaxTaps) return LM_B200_EUNSUPPORTED;
+            break;
         default: return LM_B200_EUNSUPPORTED;
+    }
+    return LM_B200_OK;
+}
+
+int check_stream_layer(const lm_b200_model& m, const lm_b200_layer& l) {
+    if (l.streams < 1 || l.streams > 8) return LM_B200_EUNSUPPORTED;
+    if (!stream_norm_ok(l.norm_mix_in) || !l.w_in || !l.w_o) return LM_B200_EINVAL;
+    for (int q = 0; q < (l.ff == LM_B200_FF_NONE ? 1 : 2); ++q)
+        if (!l.hc_in[q] || !l.hc_out[q] || !l.hc_mix[q]) return LM_B200_EINVAL;
+    if (l.mixer == LM_B200_MIXER_PAIR && (!l.part[0] || !l.part[1] || l.n_in != l.part[0]->n_in + l.part[1]->n_in)) return LM_B200_EINVAL;
+    for (int q = 0; q < n_parts(l); ++q) {
+        const int rc = check_stream_mixer(part_of(l, q));
+        if (rc != LM_B200_OK) return rc;
+    }
+    if (l.side_dim < 0) return LM_B200_EINVAL;
+    if (l.side_dim > 0) {
+        if (!l.side_table || !l.w_side_gate || !l.w_side_proj || !l.side_norm || l.side_off < 0 || l.side_off + l.side_dim > l.side_ld)
+            return LM_B200_EINVAL;
+        if (l.streams != 1) return LM_B200_EUNSUPPORTED;
     }
     if (l.ff == LM_B200_FF_NONE) return LM_B200_OK;
     if (!stream_norm_ok(l.norm_ff_in)) return LM_B200_EINVAL;
     if (l.parallel && l.norm_ff_in.kind != l.norm_mix_in.kind) return LM_B200_EUNSUPPORTED;
     if (l.ff == LM_B200_FF_DENSE && l.act == LM_B200_ACT_RELU2) return (l.dense_ff > 0 && l.ws_gate_up && l.ws_down) ? LM_B200_OK : LM_B200_EINVAL;
-    if (l.act != LM_B200_ACT_CLAMPED_GLU && l.act != LM_B200_ACT_SILU_GLU) return LM_B200_EUNSUPPORTED;
+    if (l.act != LM_B200_ACT_CLAMPED_GLU && l.act != LM_B200_ACT_SILU_GLU && l.act != LM_B200_ACT_GELU_GLU) return LM_B200_EUNSUPPORTED;
     if (l.ff == LM_B200_FF_DENSE) return (l.dense_ff > 0 && l.ws_gate_up && l.ws_down) ? LM_B200_OK : LM_B200_EINVAL;
     if (l.ff != LM_B200_FF_ROUTED_EXPERTS) return LM_B200_EUNSUPPORTED;
     if (l.experts <= 0 || l.top <= 0 || l.expert_ff <= 0 || l.shared_ff < 0) return LM_B200_EINVAL;
@@ -507,7 +576,7 @@ int mixer_kernels(lm_b200_engine* e, const lm_b200_layer& l, const InCols& c, fl
         case LM_B200_MIXER_HGRN2: {
             LCK(lm::launch_gate_prep(proj, c.n, c.q, c.f, c.v, l.in_bias, l.lower, l.heads * l.dim, l.heads * l.vdim, M, st));
             const lm::ScanInputs si{c.q, 0, c.f, c.v, 0};
-            LCK(lm::launch_column_scan(proj, c.n, si, false, l.heads, l.heads, l.dim, l.vdim, l.rec_state, v.sm, v.rm, n_seq,
+            LCK(lm::launch_column_scan(proj, c.n, si, lm::kScanTied, l.heads, l.heads, l.dim, l.vdim, l.rec_state, v.sm, v.rm, n_seq,
                                        e->outcat, ko, st, false, M <= lm::kRowsKernelMax));
             LCK(lm::launch_head_norm_gate(e->outcat, ko, ob, l.head_norm, nullptr, 0, l.heads, l.vdim, e->m.eps, M, st));
             break;
@@ -524,7 +593,7 @@ int mixer_kernels(lm_b200_engine* e, const lm_b200_layer& l, const InCols& c, fl
             LCK(lm::launch_delta_prep(proj, c.n, c.beta, d, l.conv_tail, v.rm, e->rec, ldr, M, st));
             LCK(lm::launch_conv_tail(proj, c.n, C, l.conv_taps, l.conv_tail, v.sm, n_seq, st));
             const lm::ScanInputs si{0, k0, d0, v0, b0};
-            LCK(lm::launch_column_scan(e->rec, ldr, si, true, l.heads, l.kv_heads, l.dim, l.vdim, l.rec_state, v.sm, v.rm, n_seq,
+            LCK(lm::launch_column_scan(e->rec, ldr, si, lm::kScanDelta, l.heads, l.kv_heads, l.dim, l.vdim, l.rec_state, v.sm, v.rm, n_seq,
                                        e->outcat, ko, st, false, M <= lm::kRowsKernelMax));
             LCK(lm::launch_head_norm_gate(e->outcat, ko, ob, l.head_norm, e->rec + g0, ldr, l.heads, l.vdim, e->m.eps, M, st));
             break;
@@ -586,24 +655,28 @@ int product_ld(lm_b200_engine* e, const float* A, int lda, const void* Ab, const
     return LM_B200_OK;
 }
 
-// y = mixer(h) of a stream record
-int stream_mixer(lm_b200_engine* e, const lm_b200_layer& l, const float* h, const void* hb, const StepView& v, int M, int n_seq,
-                 float* y, cudaStream_t st) {
-    const int D = e->m.width, H = l.heads, nv = H * l.vdim;
+// where one mixer of a record finds its stacked projections and leaves its output: columns of wider rows when two mixers share
+// the record, and the weight its output gets there
+struct MixPlace { float* proj; int ld; float* out; void* out_b; int ldo; float scale; };
+
+// the kernels of one mixer of a stream record, between the stacked projections and the output projection
+int stream_mixer_kernels(lm_b200_engine* e, const lm_b200_layer& l, const MixPlace& at, const StepView& v, int M, int n_seq,
+                         cudaStream_t st) {
+    const int H = l.heads, nv = H * l.vdim, ld = at.ld;
     const bool bf = e->m.precision == LM_B200_PRECISION_BF16 && M >= kTensorRowsMin;
     const StreamCols c = stream_cols(l);
-    int rc = product_ld(e, h, D, hb, l.w_in, e->proj, M, c.n, D, st);
-    if (rc) return rc;
-    const float* gate = c.gate >= 0 ? e->proj + c.gate : nullptr;
+    float* const proj = at.proj;
+    const lm::PageMap pm{e->m.page_table, e->m.max_pages, e->m.page_size};
+    const float* gate = c.gate >= 0 ? proj + c.gate : nullptr;
+    int rc = LM_B200_OK;
     const int gate_act = l.mixer_gate == LM_B200_GATE_SILU ? 2 : 1;
     if (l.mixer == LM_B200_MIXER_LATENT_ATTENTION) {
-        const lm::PageMap pm{e->m.page_table, e->m.max_pages, e->m.page_size};
         // a query head is [dim plain | rot_dim turned]; a cached row is [latent | turned key part]
         const int rd = l.rot_dim, dq = l.dim + rd, RK = l.kv_rank + rd, nq = H * dq, nl = H * RK, no = H * l.kv_rank;
         const lm::RotPart rot{rd, l.rot_dims, l.rot_layout, l.rot_freq};
-        LCK(lm::launch_latent_prep(e->proj, c.n, c.lat_q, l.q_rank, c.lat_c, l.kv_rank, l.q_lat_norm, l.kv_lat_norm, e->m.eps,
+        LCK(lm::launch_latent_prep(proj, ld, c.lat_q, l.q_rank, c.lat_c, l.kv_rank, l.q_lat_norm, l.kv_lat_norm, e->m.eps,
                                    bf ? e->cqb : nullptr, l.latent_pages, pm, v.rm, M, st, rot));
-        rc = product_ld(e, e->proj + c.lat_q, c.n, bf ? e->cqb : nullptr, l.w_uq, e->qk, M, nq, l.q_rank, st);
+        rc = product_ld(e, proj + c.lat_q, ld, bf ? e->cqb : nullptr, l.w_uq, e->qk, M, nq, l.q_rank, st);
         if (rc) return rc;
         // scores q_h . (W_uk,h c_j) = (W_uk,h^T q_h) . c_j: the query goes into the latent space, with the score multiplier;
         // its turned part stands behind it, against the turned key part of the cached row
@@ -617,34 +690,102 @@ int stream_mixer(lm_b200_engine* e, const lm_b200_layer& l, const float* h, cons
             LCK(lm::launch_latent_attention_rows(e->qlat, l.latent_pages, pm, H, l.kv_rank, l.sink, v.rm, e->olat, M, st, rd,
                                                  l.window > 0 ? l.window : 0));
         // sum_j p_j (W_uv,h c_j) = W_uv,h (sum_j p_j c_j), times the sigmoid of the gate columns
-        LCK(lm::launch_head_linear(e->olat, no, l.w_uv, e->att, nv, bf ? e->attb : nullptr, M, H, l.vdim, l.kv_rank, 1.f, gate, c.n, st));
+        LCK(lm::launch_head_linear(e->olat, no, l.w_uv, at.out, at.ldo, at.out_b, M, H, l.vdim, l.kv_rank, at.scale, gate, ld, st));
     } else if (l.mixer == LM_B200_MIXER_GATED_DELTA) {
         const lm::DeltaShape d{H, l.kv_heads, l.dim, l.vdim, l.conv_taps, l.unit_eps, l.conv_w, l.a_log, l.dt_bias};
-        const int k0 = l.kv_heads * l.dim, v0 = 2 * k0, d0 = v0 + nv, b0 = d0 + H, ldr = delta_rec_cols(l);
-        LCK(lm::launch_delta_prep(e->proj, c.n, c.beta, d, l.conv_tail, v.rm, e->rec, ldr, M, st, c.a));
-        LCK(lm::launch_conv_tail(e->proj, c.n, v0 + nv, l.conv_taps, l.conv_tail, v.sm, n_seq, st));
+        const int k0 = l.kv_heads * l.dim, v0 = 2 * k0, d0 = v0 + nv, b0 = d0 + H, ldr = stream_rec_cols(l);
+        LCK(lm::launch_delta_prep(proj, ld, c.beta, d, l.conv_tail, v.rm, e->rec, ldr, M, st, c.a));
+        LCK(lm::launch_conv_tail(proj, ld, v0 + nv, l.conv_taps, l.conv_tail, v.sm, n_seq, st));
         const lm::ScanInputs si{0, k0, d0, v0, b0};
-        LCK(lm::launch_column_scan(e->rec, ldr, si, true, H, l.kv_heads, l.dim, l.vdim, l.rec_state, v.sm, v.rm, n_seq, e->att, nv, st,
+        LCK(lm::launch_column_scan(e->rec, ldr, si, lm::kScanDelta, H, l.kv_heads, l.dim, l.vdim, l.rec_state, v.sm, v.rm, n_seq, at.out, at.ldo, st,
                                    true, M <= lm::kRowsKernelMax));
-        LCK(lm::launch_head_norm_gate(e->att, nv, bf ? e->attb : nullptr, l.head_norm, gate, c.n, H, l.vdim, e->m.eps, M, st, gate_act));
+        LCK(lm::launch_head_norm_gate(at.out, at.ldo, at.out_b, l.head_norm, gate, ld, H, l.vdim, e->m.eps, M, st, gate_act, at.scale));
     } else if (l.mixer == LM_B200_MIXER_RETENTION) {
         // q and k (adjacent in the row) turn in place, k also takes dim^-1/2; decay fixed per head, no write gate, no normaliser
         const lm::RotPart rot{l.dim, l.rot_dims, l.rot_layout, l.rot_freq};
-        LCK(lm::launch_rot_rows(e->proj, c.n, c.q, l.dim, e->proj, c.n, c.q, l.dim, 2 * H, l.dim, rot, H, 1.f,
+        LCK(lm::launch_rot_rows(proj, ld, c.q, l.dim, proj, ld, c.q, l.dim, 2 * H, l.dim, rot, H, 1.f,
                                 1.0f / sqrtf((float)l.dim), v.rm, M, st));
         const lm::ScanInputs si{c.q, c.k, 0, c.v, 0};
-        LCK(lm::launch_scalar_gate_scan(e->proj, c.n, si, H, l.dim, l.vdim, l.rec_state, v.sm, v.rm, n_seq, e->att, nv, st,
+        LCK(lm::launch_scalar_gate_scan(proj, ld, si, H, l.dim, l.vdim, l.rec_state, v.sm, v.rm, n_seq, at.out, at.ldo, st,
                                         l.head_decay, false, M <= lm::kRowsKernelMax));
-        LCK(lm::launch_head_norm_gate(e->att, nv, bf ? e->attb : nullptr, l.head_norm, gate, c.n, H, l.vdim, e->m.eps, M, st, gate_act));
+        LCK(lm::launch_head_norm_gate(at.out, at.ldo, at.out_b, l.head_norm, gate, ld, H, l.vdim, e->m.eps, M, st, gate_act, at.scale));
+    } else if (l.mixer == LM_B200_MIXER_ROTARY_ATTENTION) {
+        // the score multiplier rides on q; the raw key projection is the value when the record says so
+        const lm::TalkShape a{H, l.kv_heads, l.dim, l.vdim, l.rot_dims, l.scale, l.rot_freq, nullptr, nullptr, 0, l.rot_amp};
+        LCK(lm::launch_talk_prep(proj, ld, nullptr, c.q, c.k, c.v, -1, a, l.q_norm, l.k_norm, e->m.eps, l.k_pages, l.v_pages, pm, v.rm, M, st));
+        const lm::AttnShape s{H, l.kv_heads, l.dim, l.window > 0 ? l.window : 0, 0, 1.f, 0.f, nullptr, nullptr, l.sink};
+        LCK(lm::launch_sink_attention(proj + c.q, ld, l.k_pages, l.v_pages, pm, s, v.rm, at.out, at.out_b, e->split_ws, e->split_arrived, M,
+                                      st, at.ldo, at.scale));
+    } else if (l.mixer == LM_B200_MIXER_GATED_LINEAR) {
+        LCK(lm::launch_decay_proj(proj + c.a1, ld, l.w_a2, l.dt_bias, l.decay_tau, e->rec, H * l.dim, l.rank_a, M, st));
+        const lm::ScanInputs si{c.q, c.k, 0, c.v, 0};
+        LCK(lm::launch_column_scan(proj, ld, si, lm::kScanWrite, H, H, l.dim, l.vdim, l.rec_state, v.sm, v.rm, n_seq, at.out, at.ldo, st, false,
+                                   M <= lm::kRowsKernelMax, e->rec, H * l.dim, 1.0f / sqrtf((float)l.dim)));
+        LCK(lm::launch_head_norm_gate(at.out, at.ldo, at.out_b, l.head_norm, gate, ld, H, l.vdim, e->m.eps, M, st, gate_act, at.scale));
+    } else if (l.mixer == LM_B200_MIXER_MAMBA2) {
+        const lm::SsmShape d{H, l.kv_heads, l.dim, l.vdim, l.conv_taps, l.conv_w, l.conv_b, l.a_log, l.dt_bias};
+        const int gn = l.kv_heads * l.dim, C = nv + 2 * gn, ldr = stream_rec_cols(l);
+        LCK(lm::launch_ssm_prep(proj, ld, c.x, d, l.conv_tail, v.rm, e->rec, ldr, M, st));
+        LCK(lm::launch_conv_tail(proj + c.x, ld, C, l.conv_taps, l.conv_tail, v.sm, n_seq, st));
+        const lm::ScanInputs si{nv + gn, nv, C, 0, C + H};       // reads out with C, writes along B, dt as the write strength
+        LCK(lm::launch_scalar_gate_scan(e->rec, ldr, si, H, l.dim, l.vdim, l.rec_state, v.sm, v.rm, n_seq, at.out, at.ldo, st, nullptr, false,
+                                        M <= lm::kRowsKernelMax, l.kv_heads, l.skip_d));
+        LCK(lm::launch_gate_norm(at.out, at.ldo, at.out_b, proj + c.z, ld, l.head_norm, nv, l.norm_groups, e->m.eps, at.scale, M, st));
     } else {
-        LCK(lm::launch_mlstm_gates(e->proj, c.n, c.ig, c.fg, l.in_bias, l.gate_cap, H, l.rec_aux, v.sm, v.rm, n_seq, e->floorb, st));
+        LCK(lm::launch_mlstm_gates(proj, ld, c.ig, c.fg, l.in_bias, l.gate_cap, H, l.rec_aux, v.sm, v.rm, n_seq, e->floorb, st));
         const lm::ScanInputs si{c.q, c.k, c.fg, c.v, c.ig};      // decay in the forget column, write strength in the input column
-        LCK(lm::launch_scalar_gate_scan(e->proj, c.n, si, H, l.dim, l.vdim, l.rec_state, v.sm, v.rm, n_seq, e->olat,
+        LCK(lm::launch_scalar_gate_scan(proj, ld, si, H, l.dim, l.vdim, l.rec_state, v.sm, v.rm, n_seq, e->olat,
                                         H * (l.vdim + 1), st, nullptr, true, M <= lm::kRowsKernelMax));
-        LCK(lm::launch_mlstm_finish(e->olat, H * (l.vdim + 1), e->floorb, 1.0f / sqrtf((float)l.dim), l.head_norm, e->proj + c.gate,
-                                    c.n, e->m.eps, e->att, bf ? e->attb : nullptr, M, H, l.vdim, st));
+        LCK(lm::launch_mlstm_finish(e->olat, H * (l.vdim + 1), e->floorb, 1.0f / sqrtf((float)l.dim), l.head_norm, proj + c.gate,
+                                    ld, e->m.eps, at.out, at.out_b, M, H, l.vdim, st, at.ldo, at.scale));
     }
-    return product_ld(e, e->att, nv, bf ? e->attb : nullptr, l.w_o, y, M, D, nv, st);
+    return LM_B200_OK;
+}
+
+// the mixer kernels of a stream record on its stacked projections proj [M][n_in]: e->att [M][mix_out_cols] (+ the bf16 operand)
+int stream_mixers(lm_b200_engine* e, const lm_b200_layer& l, float* proj, const StepView& v, int M, int n_seq, cudaStream_t st) {
+    const bool bf = e->m.precision == LM_B200_PRECISION_BF16 && M >= kTensorRowsMin;
+    const int ldo = mix_out_cols(l);
+    int in = 0, out = 0;
+    for (int q = 0; q < n_parts(l); ++q) {
+        const lm_b200_layer& p = part_of(l, q);
+        const MixPlace at{proj + in, l.n_in, e->att + out, bf ? (char*)e->attb + 2 * (size_t)out : nullptr, ldo,
+                          l.mixer == LM_B200_MIXER_PAIR ? l.part_scale[q] : 1.f};
+        const int rc = stream_mixer_kernels(e, p, at, v, M, n_seq, st);
+        if (rc) return rc;
+        in += p.n_in;
+        out += p.heads * p.vdim;
+    }
+    return LM_B200_OK;
+}
+
+// y = mixer(h) of a stream record
+int stream_mixer(lm_b200_engine* e, const lm_b200_layer& l, const float* h, const void* hb, const StepView& v, int M, int n_seq,
+                 float* y, cudaStream_t st) {
+    const int D = e->m.width, ko = mix_out_cols(l);
+    const bool bf = e->m.precision == LM_B200_PRECISION_BF16 && M >= kTensorRowsMin;
+    int rc = product_ld(e, h, D, hb, l.w_in, e->proj, M, l.n_in, D, st);
+    if (rc) return rc;
+    rc = stream_mixers(e, l, e->proj, v, M, n_seq, st);
+    if (rc) return rc;
+    return product_ld(e, e->att, ko, bf ? e->attb : nullptr, l.w_o, y, M, D, ko, st);
+}
+
+// y = W_proj (gelu(W_gate x) * e) of a record's token input; x is the residual stream [M][width] (xb: its bf16 copy)
+int token_input(lm_b200_engine* e, const lm_b200_layer& l, const float* x, const void* xb, const int* ids, int M, float* y,
+                cudaStream_t st) {
+    const int D = e->m.width, n = l.side_dim;
+    const lm::TokenSide ts{l.side_table, l.side_ld, l.side_off, n, ids, e->m.vocab};
+    if (M <= lm::kRowsKernelMax) {
+        LCK(lm::launch_side_gate_rows(x, D, l.w_side_gate, ts, e->side_g, M, st));
+        LCK(lm::launch_linear(e->side_g, n, l.w_side_proj, 0, y, D, M, D, n, nullptr, st));
+        return LM_B200_OK;
+    }
+    int rc = product_ld(e, x, D, xb, l.w_side_gate, e->side_z, M, n, D, st);
+    if (rc) return rc;
+    void* gb = xb && tensor_path(e, M, D, n) ? e->side_gb : nullptr;
+    LCK(lm::launch_side_act(e->side_z, ts, gb ? nullptr : e->side_g, gb, M, st));
+    return product_ld(e, e->side_g, n, gb, l.w_side_proj, y, M, D, n, st);
 }
 
 // a dense unit that is not gated: out = max(h W_up^T, 0)^2 W_down^T
@@ -669,16 +810,16 @@ int gated_unit(lm_b200_engine* e, const lm_b200_layer& l, const float* h, const 
     const int D = e->m.width;
     if (hb && tensor_path(e, M, 2 * F, D) && tensor_path(e, M, D, F)) {
         LCK(dia::launch_gemm_tcgen05_bf16(hb, 1, w_gu, 2 * F, e->sgu, M, 2 * F, D, kPlain, nullptr, st));
-        LCK(lm::launch_silu_mul(e->sgu, nullptr, e->smidb, M, F, nullptr, st, l.act == LM_B200_ACT_CLAMPED_GLU ? 1 : 0, limit));
+        LCK(lm::launch_silu_mul(e->sgu, nullptr, e->smidb, M, F, nullptr, st, glu_kind(l.act), limit));
         LCK(dia::launch_gemm_tcgen05_bf16(e->smidb, 1, w_down, D, out, M, D, F, kPlain, nullptr, st));
         return LM_B200_OK;
     }
     if (M <= lm::kRowsKernelMax) {                              // the gate inside the [gate | up] product
-        const lm::GluAct act{l.act == LM_B200_ACT_CLAMPED_GLU ? 1 : 0, limit, limit};
+        const lm::GluAct act{glu_kind(l.act), limit, limit};
         LCK(lm::launch_gated_rows(h, D, nullptr, 0, nullptr, 0, F, D, nullptr, w_gu, e->smid, M, F, st, act));
     } else {
         LCK(lm::launch_linear(h, D, w_gu, 0, e->sgu, 2 * F, M, 2 * F, D, nullptr, st));
-        LCK(lm::launch_silu_mul(e->sgu, e->smid, nullptr, M, F, nullptr, st, l.act == LM_B200_ACT_CLAMPED_GLU ? 1 : 0, limit));
+        LCK(lm::launch_silu_mul(e->sgu, e->smid, nullptr, M, F, nullptr, st, glu_kind(l.act), limit));
     }
     LCK(lm::launch_linear(e->smid, F, w_down, 0, out, D, M, D, F, nullptr, st));
     return LM_B200_OK;
@@ -689,7 +830,7 @@ int gated_unit(lm_b200_engine* e, const lm_b200_layer& l, const float* h, const 
 int stream_ff(lm_b200_engine* e, const lm_b200_layer& l, const float* h, const void* hb, int M, lm::StreamWrite* wr,
               lm::StreamExtra* wx, cudaStream_t st) {
     const int D = e->m.width, E = l.experts, top = l.top, F = l.expert_ff, Sf = l.shared_ff;
-    const int act = l.act == LM_B200_ACT_CLAMPED_GLU ? 1 : 0;
+    const int act = glu_kind(l.act);
     wr->y = e->y; wr->parts = nullptr; wr->slot_of = nullptr; wr->sel_w = nullptr; wr->top = 0;
     if (l.ff == LM_B200_FF_DENSE) {
         if (l.act == LM_B200_ACT_RELU2) return relu2_unit(e, h, hb, M, l.ws_gate_up, l.ws_down, l.dense_ff, e->y, st);
@@ -775,28 +916,41 @@ int lm_b200_engine_create(const lm_b200_model* model, const lm_b200_layer* layer
     if (!e) return LM_B200_ENOMEM;
     e->m = m;
     e->layers.assign(layers, layers + m.n_layer);
+    for (const lm_b200_layer& l : e->layers)
+        if (l.form == LM_B200_FORM_STREAMS && l.mixer == LM_B200_MIXER_PAIR)
+            for (int q = 0; q < 2; ++q) e->parts_of_pairs.push_back(*l.part[q]);
+    size_t next_part = 0;                        // (the vector no longer grows)
+    for (lm_b200_layer& l : e->layers)
+        if (l.form == LM_B200_FORM_STREAMS && l.mixer == LM_B200_MIXER_PAIR)
+            for (int q = 0; q < 2; ++q) l.part[q] = &e->parts_of_pairs[next_part++];
     e->device = device;
     const size_t R = (size_t)m.max_rows, D = (size_t)m.width;
     size_t qk = 0, att = 0, E = 1, top = 1, F = 1, Sf = 1, slots = 1;
     size_t n_in = 0, k_out = 0, n_rec = 0, split_dim = 0;
-    size_t n_streams = 0, n_lat = 0, q_rank = 0, n_heads = 0;
+    size_t n_streams = 0, n_lat = 0, q_rank = 0, n_heads = 0, n_side = 0;
     bool pre = false, any_parallel = false;
     e->stream_form = e->layers[0].form == LM_B200_FORM_STREAMS;
     for (const lm_b200_layer& l : e->layers) {
         if (l.form == LM_B200_FORM_STREAMS) {
             n_streams = (size_t)l.streams;
             n_in = std::max(n_in, (size_t)l.n_in);
-            att = std::max(att, (size_t)l.heads * l.vdim);
-            n_heads = std::max(n_heads, (size_t)l.heads);
-            if (l.mixer == LM_B200_MIXER_LATENT_ATTENTION) {
-                qk = std::max(qk, (size_t)l.heads * (l.dim + l.rot_dim));
-                n_lat = std::max(n_lat, (size_t)l.heads * (l.kv_rank + l.rot_dim));
-                q_rank = std::max(q_rank, (size_t)l.q_rank);
-                if (lm::talk_attention_supported(latent_shape(l))) split_dim = std::max(split_dim, (size_t)l.heads * (l.kv_rank + 2));
-            } else if (l.mixer == LM_B200_MIXER_MLSTM) {
-                n_lat = std::max(n_lat, (size_t)l.heads * (l.vdim + 1));
+            att = std::max(att, (size_t)mix_out_cols(l));
+            for (int q = 0; q < n_parts(l); ++q) {
+                const lm_b200_layer& p = part_of(l, q);
+                n_heads = std::max(n_heads, (size_t)p.heads);
+                if (p.mixer == LM_B200_MIXER_LATENT_ATTENTION) {
+                    qk = std::max(qk, (size_t)p.heads * (p.dim + p.rot_dim));
+                    n_lat = std::max(n_lat, (size_t)p.heads * (p.kv_rank + p.rot_dim));
+                    q_rank = std::max(q_rank, (size_t)p.q_rank);
+                    if (lm::talk_attention_supported(latent_shape(p))) split_dim = std::max(split_dim, (size_t)p.heads * (p.kv_rank + 2));
+                } else if (p.mixer == LM_B200_MIXER_MLSTM) {
+                    n_lat = std::max(n_lat, (size_t)p.heads * (p.vdim + 1));
+                } else if (p.mixer == LM_B200_MIXER_ROTARY_ATTENTION) {
+                    split_dim = std::max(split_dim, (size_t)p.heads * (p.dim + 2));
+                }
+                n_rec = std::max(n_rec, (size_t)stream_rec_cols(p));
             }
-            n_rec = std::max(n_rec, (size_t)delta_rec_cols(l));
+            n_side = std::max(n_side, (size_t)l.side_dim);
             any_parallel = any_parallel || (l.parallel && l.ff != LM_B200_FF_NONE);
             if (l.ff == LM_B200_FF_DENSE) Sf = std::max(Sf, (size_t)l.dense_ff);
             if (l.ff == LM_B200_FF_ROUTED_EXPERTS) {
@@ -841,7 +995,8 @@ int lm_b200_engine_create(const lm_b200_model* model, const lm_b200_layer* layer
                  o_floor = take(R * n_heads * 4), o_unit = take(2 * 4);
     const size_t o_ymix = take(any_parallel ? R * D * 4 : 0), o_h2 = take(any_parallel ? R * D * 4 : 0);
     const size_t o_split = take((size_t)lm::kAttnRowsKernelMax * lm::kAttnSplitsMax * split_dim * 4);
-    size_t max_heads = 1;
+    const size_t o_sidez = take(R * n_side * 4), o_sideg = take(R * n_side * 4);
+    size_t max_heads = std::max<size_t>(1, n_heads);
     for (const lm_b200_layer& l : e->layers) max_heads = std::max(max_heads, (size_t)l.heads);
     const size_t arrived_bytes = (size_t)lm::kAttnRowsKernelMax * max_heads * 4, o_arrived = take(arrived_bytes);
     const size_t o_step = take((size_t)(8 * lm::kRowsKernelMax) * 4), o_logits = take((size_t)lm::kRowsKernelMax * m.vocab * 4);
@@ -849,7 +1004,8 @@ int lm_b200_engine_create(const lm_b200_model* model, const lm_b200_layer* layer
     const size_t o_hb = take(tcb ? R * D * 2 : 0), o_attb = take(tcb ? R * att * 2 : 0), o_packb = take(tcb ? slots * D * 2 : 0),
                  o_midb = take(tcb ? slots * F * 2 : 0), o_smidb = take(tcb ? R * Sf * 2 : 0), o_hwb = take(tcb ? R * D * 2 : 0);
     const size_t o_catb = take(tcb && pre ? R * 2 * D * 2 : 0), o_outcatb = take(tcb ? R * k_out * 2 : 0);
-    const size_t o_cqb = take(tcb ? R * q_rank * 2 : 0), o_h2b = take(tcb && any_parallel ? R * D * 2 : 0);
+    const size_t o_cqb = take(tcb ? R * q_rank * 2 : 0), o_h2b = take(tcb && any_parallel ? R * D * 2 : 0),
+                 o_sidegb = take(tcb ? R * n_side * 2 : 0);
     if (cudaMalloc(&e->arena, off) != cudaSuccess) {
         (void)cudaGetLastError();
         delete e;
@@ -870,6 +1026,7 @@ int lm_b200_engine_create(const lm_b200_model* model, const lm_b200_layer* layer
     e->xs = (float*)(b + o_xs); e->qlat = (float*)(b + o_qlat); e->olat = (float*)(b + o_olat); e->floorb = (float*)(b + o_floor);
     e->unit = (float*)(b + o_unit); e->cqb = b + o_cqb;
     e->ymix = (float*)(b + o_ymix); e->h2 = (float*)(b + o_h2); e->h2b = b + o_h2b;
+    e->side_z = (float*)(b + o_sidez); e->side_g = (float*)(b + o_sideg); e->side_gb = b + o_sidegb;
     e->split_ws = (float*)(b + o_split);
     e->split_arrived = (unsigned*)(b + o_arrived);
     const float unit_host[2] = {0.f, 1.f};
@@ -975,6 +1132,16 @@ int run_stream_layers(lm_b200_engine* e, const StepView& v, int M, int n_seq, fl
             if (rc) return rc;
             wr.mix = l.hc_mix[1];
             wr.out = l.hc_out[1];
+        }
+        if (l.side_dim > 0) {
+            // the residual stream with everything so far written (one stream: the stream itself; its bf16 copy is the operand of a
+            // long step), the token input on it, and its normed output as the write that follows
+            LCK(lm::launch_streams_step(e->xs, s, wr, nullptr, nullptr, eps, nullptr, bf ? e->h : nullptr, hb, M, D, st, wx));
+            rc = token_input(e, l, e->xs, hb, v.token, M, e->y, st);
+            if (rc) return rc;
+            wr = lm::StreamWrite{e->unit + 1, e->unit + 1, e->y, nullptr, nullptr, nullptr, 0};
+            wx = lm::StreamExtra{};
+            wx.y_norm_w = l.side_norm;
         }
         // this sublayer's write with the next layer's read, or with the closing sum of the streams
         if (i + 1 < n) {
@@ -1156,9 +1323,16 @@ int lm_b200_op_mixer_kernels(lm_b200_engine* e, int layer, float* proj, const in
     if (!e || layer < 0 || layer >= e->m.n_layer || !proj || !step || !out || M <= 0 || M > e->m.max_rows || n_seq <= 0)
         return LM_B200_EINVAL;
     const lm_b200_layer& l = e->layers[layer];
-    if (l.form != LM_B200_FORM_PARALLEL) return LM_B200_EUNSUPPORTED;
+    if (l.form != LM_B200_FORM_PARALLEL && l.form != LM_B200_FORM_STREAMS) return LM_B200_EUNSUPPORTED;
     Guard g(e->device);
     if (!g.ok) return LM_B200_ECUDA;
+    if (l.form == LM_B200_FORM_STREAMS) {
+        const int rc = stream_mixers(e, l, proj, view(step, M, n_seq), M, n_seq, S(stream));
+        if (rc) return rc;
+        if (cudaMemcpyAsync(out, e->att, (size_t)M * mix_out_cols(l) * 4, cudaMemcpyDeviceToDevice, S(stream)) != cudaSuccess)
+            return cuda_fail(cudaGetLastError());
+        return LM_B200_OK;
+    }
     const int rc = mixer_kernels(e, l, in_cols(l), proj, view(step, M, n_seq), M, n_seq, nullptr, S(stream));
     if (rc) return rc;
     const size_t w = (size_t)l.heads * l.vdim * 4;
@@ -1200,6 +1374,28 @@ int lm_b200_op_ff(lm_b200_engine* e, int layer, const float* h, int M, float* y,
     Guard g(e->device);
     if (!g.ok) return LM_B200_ECUDA;
     return feed_forward(e, l, h, nullptr, M, y, nullptr, lm::TapOut{}, S(stream));                // no norm: the plain sum, written to y
+}
+
+int lm_b200_op_token_input(lm_b200_engine* e, int layer, const float* x, const int32_t* step, int M, float* out, void* stream) {
+    if (!e || layer < 0 || layer >= e->m.n_layer || !x || !step || !out || M <= 0 || M > e->m.max_rows) return LM_B200_EINVAL;
+    const lm_b200_layer& l = e->layers[layer];
+    if (l.form != LM_B200_FORM_STREAMS || l.side_dim <= 0) return LM_B200_EINVAL;
+    Guard g(e->device);
+    if (!g.ok) return LM_B200_ECUDA;
+    cudaStream_t st = S(stream);
+    const void* xb = nullptr;
+    if (e->m.precision == LM_B200_PRECISION_BF16 && M >= kTensorRowsMin) {
+        LCK(lm::launch_pack_rows_bf16(x, e->hb, M, e->m.width, nullptr, st));
+        xb = e->hb;
+    }
+    const int rc = token_input(e, l, x, xb, view(step, M, 1).token, M, e->y, st);
+    if (rc) return rc;
+    if (cudaMemcpyAsync(out, x, (size_t)M * e->m.width * 4, cudaMemcpyDeviceToDevice, st) != cudaSuccess) return cuda_fail(cudaGetLastError());
+    const lm::StreamWrite wr{e->unit + 1, e->unit + 1, e->y, nullptr, nullptr, nullptr, 0};
+    lm::StreamExtra wx{};
+    wx.y_norm_w = l.side_norm;
+    LCK(lm::launch_streams_step(out, 1, wr, nullptr, nullptr, e->m.eps, nullptr, nullptr, nullptr, M, e->m.width, st, wx));
+    return LM_B200_OK;
 }
 
 int lm_b200_op_linear(const float* A, const void* W_bf16, float* Y, int M, int N, int K, void* stream) {

@@ -37,7 +37,7 @@ struct GroupMap { int* a_row; float* a_scale; int* a_expert; int* n_slots; };   
 // restricted to the `keep` best of `count` groups of neighbours, weights = chosen scores / their sum x scale.  n == 0: not
 // this rule.
 struct GroupedRoute { int n; int n_real; int count; int keep; float scale; const float* correction; };
-// activation of the gated units (kind: kGluSilu / kGluClamped of lm_device.cuh; the clamp of routed / dense and shared units)
+// activation of the gated units (kind: kGluSilu / kGluClamped / kGluGelu of lm_device.cuh; the clamp of routed / dense and shared units)
 struct GluAct { int kind; float limit; float shared_limit; };
 
 cudaError_t launch_embed(const void* table_bf16, const int* ids, float* out, int M, int V, int D, cudaStream_t st);
@@ -65,9 +65,10 @@ cudaError_t launch_router_rows(const float* h, int D, const void* Wr, int E, int
 cudaError_t launch_qk_norm_cache(float* qk, int nq, int nk, const float* qw, const float* kw, float eps, float* kcache,
                                  float* vcache, const PageMap& pm, int kv_heads, int dim, const RowMeta& rm, int M,
                                  cudaStream_t st);
+// ldo: row stride of the output (0: heads * dim); out_scale multiplies it
 cudaError_t launch_sink_attention(const float* qk, int q_stride, const float* kcache, const float* vcache, const PageMap& pm,
                                   const AttnShape& a, const RowMeta& rm, float* out, void* out_bf16, float* split_ws,
-                                  unsigned* arrived, int M, cudaStream_t st);
+                                  unsigned* arrived, int M, cudaStream_t st, int ldo = 0, float out_scale = 1.f);
 cudaError_t launch_router_topk(const float* z, int E, int top, int M, int* sel_e, float* sel_w, cudaStream_t st,
                                const float* bias = nullptr, bool softmax_top = false, const GroupedRoute* gr = nullptr);
 cudaError_t launch_moe_group(const int* sel_e, const float* sel_w, int n_assign, int top, int E, int pad, const GroupMap& gm,
@@ -88,6 +89,7 @@ struct TalkShape {
     const float* rot_freq;                                                      // [rot_dims / 2]
     const float* talk; const float* sink;                                       // [heads][heads], [heads]; each may be null
     int window;                                                                 // > 0: key j is seen from i only when i - j < window
+    float rot_amp;                                                              // multiplies cosine and sine (0 is read as 1)
 };
 struct DeltaShape {
     int heads, kv_heads, dim, vdim, taps;
@@ -120,19 +122,25 @@ cudaError_t launch_conv_tail(const float* proj, int ld, int C, int taps, float* 
 cudaError_t launch_gate_prep(float* proj, int ld, int q_off, int f_off, int v_off, const float* bias, const float* lower, int n_qf,
                              int n_v, int M, cudaStream_t st);
 // early (both scans): launched so that it may start while its predecessor still runs (see launch_pdl_if)
-cudaError_t launch_column_scan(const float* in, int ld, const ScanInputs& si, bool delta, int H, int G, int dim, int vdim,
+// rule: how the scan writes (kScan*); decay / ldd: the decays stand in rows of their own instead of column a_off of `in`;
+// q_mul multiplies q
+constexpr int kScanTied = 0, kScanDelta = 1, kScanWrite = 2;
+cudaError_t launch_column_scan(const float* in, int ld, const ScanInputs& si, int rule, int H, int G, int dim, int vdim,
                                float* state, const SeqMeta& sm, const RowMeta& rm, int n_seq, float* o, int ldo,
-                               cudaStream_t st, bool head_decay = false, bool early = true);
+                               cudaStream_t st, bool head_decay = false, bool early = true, const float* decay = nullptr, int ldd = 0,
+                               float q_mul = 1.f);
 // the same scan with scalar gates per (row, head): S <- a S + (b k) v^T and one more value column that is the constant 1
 // (the normaliser n <- a n + b k, read out as n . q), so state and read-out have vdim + 1 columns per head.  a and b are
 // columns a_off + h and beta_off + h of the input rows.  fixed_decay [H]: a = fixed_decay[h], b = 1 for every token instead.
-// normaliser false: no extra column (state and read-out have vdim columns per head).
+// normaliser false: no extra column (state and read-out have vdim columns per head).  G (0: H): heads of q and k, each serving
+// H / G of the H;  skip [H]: skip[h] v joins the read-out.
 cudaError_t launch_scalar_gate_scan(const float* in, int ld, const ScanInputs& si, int H, int dim, int vdim, float* state,
                                     const SeqMeta& sm, const RowMeta& rm, int n_seq, float* o, int ldo, cudaStream_t st,
-                                    const float* fixed_decay = nullptr, bool normaliser = true, bool early = true);
+                                    const float* fixed_decay = nullptr, bool normaliser = true, bool early = true, int G = 0,
+                                    const float* skip = nullptr);
 // gate_act: 0 the gate columns as they are, 1 their sigmoid, 2 their silu; w may be null (no weight)
 cudaError_t launch_head_norm_gate(float* o, int ldo, void* o_bf16, const float* w, const float* gate, int ldg, int H, int vdim,
-                                  float eps, int M, cudaStream_t st, int gate_act = 0);
+                                  float eps, int M, cudaStream_t st, int gate_act = 0, float out_scale = 1.f);
 
 // ---- the stream layer form (lm_streams.cu): hyper-connected residual streams, latent attention, stabilised matrix memory ----
 // Per row: [x_j <- sum_s mix[s][j] x_s + out[j] (y + sum_t sel_w[t] parts[slot_of[t]])]  (y == nullptr and parts == nullptr:
@@ -143,9 +151,10 @@ struct StreamWrite { const float* mix; const float* out; const float* y; const f
 // More of the same step: y2 / out2 - a second sublayer output written with its own weights (a record whose sublayers read
 // the same streams); ident_h [M][D] - what an assignment without a slot (slot_of < 0, an identity expert) adds, times its
 // weight; y_gate - y is multiplied by sigmoid(y_gate[row * y_gate_ld]); rms - the norm is x / sqrt(mean(x^2) + eps) w;
-// norm_w2 / h2 / h2_b - a second norm weight on the same statistics and where its result goes.
+// norm_w2 / h2 / h2_b - a second norm weight on the same statistics and where its result goes; y_norm_w - y is RMS-normed with
+// this weight before it is written (no parts then).
 struct StreamExtra { const float* y2; const float* out2; const float* ident_h; const float* y_gate; int y_gate_ld; int rms;
-                     const float* norm_w2; float* h2; void* h2_b; };
+                     const float* norm_w2; float* h2; void* h2_b; const float* y_norm_w; };
 cudaError_t launch_streams_step(float* X, int streams, const StreamWrite& wr, const float* in, const float* norm_w, float eps,
                                 const int* rows, float* h, void* h_bf16, int M, int D, cudaStream_t st,
                                 const StreamExtra& ex = StreamExtra{});
@@ -183,6 +192,30 @@ cudaError_t launch_mlstm_gates(float* proj, int ld, int i_off, int f_off, const 
 // o[r][h] = scale * raw[r][h][0:vdim] / (max(|scale * raw[r][h][vdim]|, floor[r][h]) + 1e-6), then / rms over the head, times
 // w[h vdim + c] and sigmoid(gate[r][h vdim + c]); fp32 and the bf16 operand
 cudaError_t launch_mlstm_finish(const float* raw, int ldr, const float* floor_in, float scale, const float* w, const float* gate,
-                                int ldg, float eps, float* out, void* out_bf16, int M, int H, int vdim, cudaStream_t st);
+                                int ldg, float eps, float* out, void* out_bf16, int M, int H, int vdim, cudaStream_t st, int ldo = 0,
+                                float out_scale = 1.f);
+
+// ---- decays, step sizes and gates of the linear-attention mixers; the token input (lm_linear.cu) ----
+// out[r][c] = sigmoid(sum_k a[r][k] W[c][k] + bias[c])^(1 / tau), W bf16 [C][rank], fp32 arithmetic, the same order of sums for
+// any number of rows
+cudaError_t launch_decay_proj(const float* a, int lda, const void* W, const float* bias, float tau, float* out, int C, int rank,
+                              int M, cudaStream_t st);
+struct SsmShape {
+    int heads, groups, state, vdim, taps;
+    const float* conv_w; const float* conv_b; const float* a_log; const float* dt_bias;
+};
+// proj columns x_off ..: x (heads vdim) | B (groups state) | C (groups state) | dt (heads).  rec row: silu(conv) of x | B | C,
+// then the decay exp(-exp(a_log) dt) (heads) and dt = softplus(dt + dt_bias) (heads)
+cudaError_t launch_ssm_prep(const float* proj, int ld, int x_off, const SsmShape& d, const float* tail, const RowMeta& rm, float* rec,
+                            int ldr, int M, cudaStream_t st);
+// o <- o silu(z), RMS-normed in `parts` equal parts of its n columns, x w x out_scale, in place (+ its bf16 copy)
+cudaError_t launch_gate_norm(float* o, int ldo, void* o_bf16, const float* z, int ldz, const float* w, int n, int parts, float eps,
+                             float out_scale, int M, cudaStream_t st);
+// e_r = columns off .. off + n of row ids[r] of the bf16 table
+struct TokenSide { const void* table; int ld; int off; int n; const int* ids; int vocab; };
+// g[r][c] = gelu(z[r][c]) e_r[c], fp32 and / or the bf16 operand
+cudaError_t launch_side_act(const float* z, const TokenSide& ts, float* g, void* g_bf16, int M, cudaStream_t st);
+// the same behind the product z = x W^T in one launch, for a handful of rows
+cudaError_t launch_side_gate_rows(const float* x, int D, const void* W, const TokenSide& ts, float* g, int M, cudaStream_t st);
 
 }  // namespace lm

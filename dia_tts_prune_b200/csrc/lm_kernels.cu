@@ -250,46 +250,7 @@ linear_tile_kernel(const float* __restrict__ A, int lda, const __nv_bfloat16* __
 // ---- the row kernels: a step of a few rows (decoding).  One warp per output element; the weights stream once per row,
 // 16 bytes per lane.  Their epilogues do what the next kernel of a long step would: the DynamicTanh + residual add, the
 // gate, the sum over a row's experts.
-// wait_first: the first weight loads go out before pdl_wait, the activations are read after it
-__device__ __forceinline__ float warp_dot(const float* __restrict__ arow, const __nv_bfloat16* __restrict__ wrow, int K, int lda,
-                                          float sc, int lane, bool wait_first = false) {
-    float acc = 0.f;
-    const bool vec = (K % 8 == 0) && (lda % 4 == 0) && ((reinterpret_cast<uintptr_t>(wrow) & 15) == 0) &&
-                     ((reinterpret_cast<uintptr_t>(arow) & 15) == 0);
-    if (vec) {
-        // eight 16-byte weight loads per lane in flight before their products (the sum keeps its order: k ascending)
-        for (int k0 = lane * 8; k0 < K; k0 += 2048) {
-            uint4 wv[8];
-#pragma unroll
-            for (int u = 0; u < 8; ++u) {
-                const int k = k0 + 256 * u;
-                wv[u] = k < K ? *reinterpret_cast<const uint4*>(wrow + k) : make_uint4(0u, 0u, 0u, 0u);
-            }
-            if (wait_first) { pdl_wait(); wait_first = false; }
-#pragma unroll
-            for (int u = 0; u < 8; ++u) {
-                const int k = k0 + 256 * u;
-                if (k >= K) break;
-                const float4 x0 = *reinterpret_cast<const float4*>(arow + k);
-                const float4 x1 = *reinterpret_cast<const float4*>(arow + k + 4);
-                const __nv_bfloat162* p = reinterpret_cast<const __nv_bfloat162*>(&wv[u]);
-                acc = fmaf(x0.x * sc, __low2float(p[0]), acc);
-                acc = fmaf(x0.y * sc, __high2float(p[0]), acc);
-                acc = fmaf(x0.z * sc, __low2float(p[1]), acc);
-                acc = fmaf(x0.w * sc, __high2float(p[1]), acc);
-                acc = fmaf(x1.x * sc, __low2float(p[2]), acc);
-                acc = fmaf(x1.y * sc, __high2float(p[2]), acc);
-                acc = fmaf(x1.z * sc, __low2float(p[3]), acc);
-                acc = fmaf(x1.w * sc, __high2float(p[3]), acc);
-            }
-        }
-    } else {
-        if (wait_first) pdl_wait();
-        for (int k = lane; k < K; k += 32) acc = fmaf(arow[k] * sc, bf(wrow[k]), acc);
-    }
-    if (wait_first) pdl_wait();                               // (K == 0: nothing was loaded)
-    return warp_sum(acc);
-}
+// (warp_dot: lm_device.cuh)
 
 // The whole warp of output element (a, n): h[a][n] = tapmix(norm(x_new)) of the next sublayer and its tail update, for a
 // row that is its sequence's only row in the step.  Lane o fetches the input o positions back and its tap; the sum runs
@@ -350,7 +311,7 @@ linear_rows_kernel(const float* __restrict__ A, int lda, const __nv_bfloat16* __
     }
 }
 
-// mid[a][n] = act(A_a . Wg_e[n], A_a . Wu_e[n]) (silu(g) u, or the clamped form of glu_act),  W_e = [gate rows (F) | up rows
+// mid[a][n] = act(A_a . Wg_e[n], A_a . Wu_e[n]) (glu_act),  W_e = [gate rows (F) | up rows
 // (F)][K].  blockIdx.y < n_assign: the
 // assignment slot a of the routed experts (row, expert and score from the maps); beyond: row blockIdx.y - n_assign through
 // the shared expert Ws (Sf hidden units) into smid.  One grid for both, so that the two weight streams overlap.
@@ -600,7 +561,8 @@ constexpr int kAttnMaxDimPerLane = 8;                         // head dim <= 256
 // CTA of at least 4 warps: warp w weighs the splits of head h0 + w, then all threads sum.  scratch: >= 4 * 33 floats
 __device__ __forceinline__ void combine_splits(const float* __restrict__ part, int S, int heads, int dim,
                                                const float* __restrict__ sink, float* __restrict__ out,
-                                               __nv_bfloat16* __restrict__ out_b, int r, int h0, int nh, float* scratch) {
+                                               __nv_bfloat16* __restrict__ out_b, int ldo, float out_scale, int r, int h0, int nh,
+                                               float* scratch) {
     static_assert(kAttnSplitsMax <= 32, "one lane per split");
     const size_t stride = (size_t)(dim + 2);
     const float* src0 = part + (size_t)(r * heads + h0) * S * stride;
@@ -627,9 +589,10 @@ __device__ __forceinline__ void combine_splits(const float* __restrict__ part, i
         float o = 0.f;
 #pragma unroll 8
         for (int s = 0; s < S; ++s) o = fmaf(__ldcg(src + s * stride), wgt[s], o);
-        o *= wgt[32];
-        out[((size_t)r * heads + h0 + hh) * dim + c] = o;
-        if (out_b) out_b[((size_t)r * heads + h0 + hh) * dim + c] = __float2bfloat16_rn(o);
+        o *= wgt[32] * out_scale;
+        const size_t at = (size_t)r * ldo + (size_t)(h0 + hh) * dim + c;
+        out[at] = o;
+        if (out_b) out_b[at] = __float2bfloat16_rn(o);
     }
 }
 
@@ -640,7 +603,8 @@ sink_attention_split_kernel(const float* __restrict__ qk, int q_stride, const fl
                             int heads, int kv_heads, int dim, float scale, float cap, const float* __restrict__ temp,
                             const float* __restrict__ slopes, const float* __restrict__ sink, int window, int keep_first,
                             const int* __restrict__ row_slot, const int* __restrict__ row_pos, float* __restrict__ part,
-                            unsigned* __restrict__ arrived, float* __restrict__ out, __nv_bfloat16* __restrict__ out_b) {
+                            unsigned* __restrict__ arrived, float* __restrict__ out, __nv_bfloat16* __restrict__ out_b, int ldo,
+                            float out_scale) {
     __shared__ float sm_m[kSplitWarps][HG], sm_l[kSplitWarps][HG];
     __shared__ bool is_last;
     __shared__ float sm_acc[kSplitWarps][HG][32 * kAttnMaxDimPerLane];
@@ -750,7 +714,7 @@ sink_attention_split_kernel(const float* __restrict__ qk, int q_stride, const fl
     if (!is_last) return;
     __threadfence();
     static_assert(HG <= kSplitWarps, "one warp per head in the merge");
-    combine_splits(part, S, heads, dim, sink, out, out_b, r, h0, nh, sm_acc[0][0]);
+    combine_splits(part, S, heads, dim, sink, out, out_b, ldo, out_scale, r, h0, nh, sm_acc[0][0]);
 }
 
 // ---------------------------------------------------------------------------------------------------------------------
@@ -770,7 +734,7 @@ sink_attention_tile_kernel(const float* __restrict__ qk, int q_stride, const flo
                            int heads, int kv_heads, int dim, float scale, float cap, const float* __restrict__ temp,
                            const float* __restrict__ slopes, const float* __restrict__ sink, int window, int keep_first,
                            const int* __restrict__ row_slot, const int* __restrict__ row_pos, float* __restrict__ out,
-                           __nv_bfloat16* __restrict__ out_b, int M) {
+                           __nv_bfloat16* __restrict__ out_b, int ldo, float out_scale, int M) {
     constexpr int DP = 64 * NC, QS = DP + 4, C4 = DP / 4;
     extern __shared__ __align__(16) float sm[];
     float* Qs = sm;                                           // [64][QS]
@@ -974,8 +938,8 @@ sink_attention_tile_kernel(const float* __restrict__ qk, int q_stride, const flo
         if (row >= n_rows) continue;
         float l = l_run[i];
         if (sink) l += expf(sink_h - m_run[i]);
-        const float inv = l > 0.f ? 1.0f / l : 0.f;
-        const size_t base = ((size_t)(r0 + row) * heads + h) * dim;
+        const float inv = l > 0.f ? out_scale / l : 0.f;
+        const size_t base = (size_t)(r0 + row) * ldo + (size_t)h * dim;
 #pragma unroll
         for (int c = 0; c < NC; ++c)
 #pragma unroll
@@ -1247,7 +1211,7 @@ cudaError_t launch_qk_norm_cache(float* qk, int nq, int nk, const float* qw, con
 template <int NC>
 static cudaError_t launch_attention_tiles(const float* qk, int q_stride, const float* kcache, const float* vcache,
                                           const PageMap& pm, const AttnShape& a, const RowMeta& rm, float* out,
-                                          __nv_bfloat16* out_b, int M, cudaStream_t st) {
+                                          __nv_bfloat16* out_b, int ldo, float out_scale, int M, cudaStream_t st) {
     constexpr int DP = 64 * NC;
     const size_t smem = (size_t)(2 * kTQ * (DP + 4) + kTK * DP + kTQ * kTPStride) * sizeof(float) + 2 * kTQ * sizeof(int);
     static bool attr[64] = {};
@@ -1261,14 +1225,15 @@ static cudaError_t launch_attention_tiles(const float* qk, int q_stride, const f
     }
     sink_attention_tile_kernel<NC><<<dim3((M + kTQ - 1) / kTQ, a.heads), kTileThreads, smem, st>>>(
         qk, q_stride, kcache, vcache, pm.table, pm.max_pages, pm.page_size, a.heads, a.kv_heads, a.dim, a.scale, a.softcap,
-        a.temp, a.slopes, a.sink, a.window, a.keep_first, rm.slot, rm.pos, out, out_b, M);
+        a.temp, a.slopes, a.sink, a.window, a.keep_first, rm.slot, rm.pos, out, out_b, ldo, out_scale, M);
     return cudaGetLastError();
 }
 
 template <int HG>
 static cudaError_t launch_attention_splits(const float* qk, int q_stride, const float* kcache, const float* vcache,
                                            const PageMap& pm, const AttnShape& a, const RowMeta& rm, float* out,
-                                           __nv_bfloat16* out_b, int M, float* split_ws, unsigned* arrived, cudaStream_t st) {
+                                           __nv_bfloat16* out_b, int ldo, float out_scale, int M, float* split_ws, unsigned* arrived,
+                                           cudaStream_t st) {
     const int group = a.heads / a.kv_heads, chunks = (group + HG - 1) / HG;
     // enough CTAs for two per SM, at least 16 keys per split where the window bounds the keys
     const long long max_keys = a.window > 0 ? (long long)a.window + a.keep_first : (long long)pm.max_pages * pm.page_size;
@@ -1277,28 +1242,29 @@ static cudaError_t launch_attention_splits(const float* qk, int q_stride, const 
     S = (int)std::max<long long>(1, std::min<long long>(std::min(S, kAttnSplitsMax), (max_keys + 15) / 16));
     return launch_pdl(sink_attention_split_kernel<HG>, dim3(M, a.kv_heads * chunks, S), dim3(kSplitThreads), 0, st, qk, q_stride,
                       kcache, vcache, pm.table, pm.max_pages, pm.page_size, a.heads, a.kv_heads, a.dim, a.scale, a.softcap, a.temp,
-                      a.slopes, a.sink, a.window, a.keep_first, rm.slot, rm.pos, split_ws, arrived, out, out_b);
+                      a.slopes, a.sink, a.window, a.keep_first, rm.slot, rm.pos, split_ws, arrived, out, out_b, ldo, out_scale);
 }
 
 // a step of a few rows (decoding) splits every row's keys over CTAs; longer steps run the tiled kernel.
 // split_ws: kRowsKernelMax * heads * kAttnSplitsMax * (dim + 2) floats; arrived: kRowsKernelMax * heads zeroed counters
 cudaError_t launch_sink_attention(const float* qk, int q_stride, const float* kcache, const float* vcache, const PageMap& pm,
                                   const AttnShape& a, const RowMeta& rm, float* out, void* out_bf16, float* split_ws,
-                                  unsigned* arrived, int M, cudaStream_t st) {
+                                  unsigned* arrived, int M, cudaStream_t st, int ldo, float out_scale) {
+    if (ldo <= 0) ldo = a.heads * a.dim;
     if (a.dim > 32 * kAttnMaxDimPerLane || a.heads % a.kv_heads) return cudaErrorNotSupported;
     __nv_bfloat16* ob = reinterpret_cast<__nv_bfloat16*>(out_bf16);
     if (M > kAttnRowsKernelMax) {
         switch ((a.dim + 63) / 64) {
-            case 1: return launch_attention_tiles<1>(qk, q_stride, kcache, vcache, pm, a, rm, out, ob, M, st);
-            case 2: return launch_attention_tiles<2>(qk, q_stride, kcache, vcache, pm, a, rm, out, ob, M, st);
-            case 3: return launch_attention_tiles<3>(qk, q_stride, kcache, vcache, pm, a, rm, out, ob, M, st);
-            default: return launch_attention_tiles<4>(qk, q_stride, kcache, vcache, pm, a, rm, out, ob, M, st);
+            case 1: return launch_attention_tiles<1>(qk, q_stride, kcache, vcache, pm, a, rm, out, ob, ldo, out_scale, M, st);
+            case 2: return launch_attention_tiles<2>(qk, q_stride, kcache, vcache, pm, a, rm, out, ob, ldo, out_scale, M, st);
+            case 3: return launch_attention_tiles<3>(qk, q_stride, kcache, vcache, pm, a, rm, out, ob, ldo, out_scale, M, st);
+            default: return launch_attention_tiles<4>(qk, q_stride, kcache, vcache, pm, a, rm, out, ob, ldo, out_scale, M, st);
         }
     }
     const int group = a.heads / a.kv_heads;
-    if (group >= 4) return launch_attention_splits<4>(qk, q_stride, kcache, vcache, pm, a, rm, out, ob, M, split_ws, arrived, st);
-    if (group >= 2) return launch_attention_splits<2>(qk, q_stride, kcache, vcache, pm, a, rm, out, ob, M, split_ws, arrived, st);
-    return launch_attention_splits<1>(qk, q_stride, kcache, vcache, pm, a, rm, out, ob, M, split_ws, arrived, st);
+    if (group >= 4) return launch_attention_splits<4>(qk, q_stride, kcache, vcache, pm, a, rm, out, ob, ldo, out_scale, M, split_ws, arrived, st);
+    if (group >= 2) return launch_attention_splits<2>(qk, q_stride, kcache, vcache, pm, a, rm, out, ob, ldo, out_scale, M, split_ws, arrived, st);
+    return launch_attention_splits<1>(qk, q_stride, kcache, vcache, pm, a, rm, out, ob, ldo, out_scale, M, split_ws, arrived, st);
 }
 
 cudaError_t launch_router_topk(const float* z, int E, int top, int M, int* sel_e, float* sel_w, cudaStream_t st, const float* bias,

@@ -19,11 +19,13 @@
 //                             their two-step projections
 //   conv_tail_kernel          keeps the last taps-1 projected inputs of every scheduled sequence
 //   gate_prep_kernel          silu(q), the bounded forget gate and biases of the gate-tied recurrence, in place
-//   column_scan_kernel        the recurrence of both recurrent mixers, one value column of one head per 8 lanes:
-//                             S <- a S;  [u = beta (v - S^T k)];  S <- S + w u;  o = S^T q, state carried per sequence
+//   column_scan_kernel        the recurrences with a decay per key channel, one value column of one head per 8 lanes:
+//                             S <- a S;  [u = beta (v - S^T k)];  S <- S + w u;  o = S^T q, state carried per sequence (the
+//                             write w is 1 - a, or k with or without the delta)
 //   scalar_gate_scan_kernel   the same column layout for a recurrence with one decay and one write strength per token and
 //                             head, and a normaliser carried as one more value column
-//                             (or a fixed decay per head, write strength 1, no normaliser: retention)
+//                             (or a fixed decay per head, write strength 1, no normaliser: retention; or q and k shared by
+//                             groups of heads and a skip term: the state-space mixer)
 //   head_norm_gate_kernel     per-head RMS norm of the read-out (x weight, x gate or its sigmoid / silu), fp32 in place and
 //                             the bf16 operand
 //   xielu_rows_kernel         the dense feed-forward's activation (xIELU or squared relu) on its slice of the stacked
@@ -105,17 +107,27 @@ __global__ void xielu_rows_kernel(const float* __restrict__ proj, int ld, int of
 // ---------------------------------------------------------------------------------------------------------------------
 // One CTA per row, one warp per q / k head.  q <- rot(rms(q + bias) * qw) * scale in place (the score multiplier rides
 // on q), k likewise without the multiplier into the key pages, v + bias into the value pages, gate <- sigmoid(gate).
+// v_off may be k_off (vdim == dim): the projected key itself, before norm and rotation, is the value.  amp multiplies cosine
+// and sine.
 __global__ void __launch_bounds__(256)
 talk_prep_kernel(float* __restrict__ proj, int ld, const float* __restrict__ bias, int q_off, int k_off, int v_off, int gate_off,
                  int H, int G, int dim, int vdim, const float* __restrict__ qw, const float* __restrict__ kw, float eps,
-                 float scale, const float* __restrict__ freq, int rot_dims, float* __restrict__ kcache,
+                 float scale, const float* __restrict__ freq, int rot_dims, float amp, float* __restrict__ kcache,
                  float* __restrict__ vcache, const int* __restrict__ table, int max_pages, int page_size,
                  const int* __restrict__ row_slot, const int* __restrict__ row_pos) {
+    extern __shared__ float trig[];                           // [rot_dims / 2] sines, then as many cosines, shared by all heads
     pdl_release();
     pdl_wait();
     const int r = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, nwarp = blockDim.x >> 5;
     float* row = proj + (size_t)r * ld;
-    const int pos = row_pos[r];
+    const int pos = row_pos[r], n_turn = rot_dims >> 1;
+    for (int i = tid; i < n_turn; i += blockDim.x) {
+        float sn, cs;
+        sincosf((float)pos * freq[i], &sn, &cs);
+        trig[i] = sn * amp;
+        trig[n_turn + i] = cs * amp;
+    }
+    __syncthreads();
     const int page = table[(size_t)row_slot[r] * max_pages + pos / page_size], off = pos % page_size;
     for (int hh = warp; hh < H + G; hh += nwarp) {
         const bool isq = hh < H;
@@ -135,8 +147,7 @@ talk_prep_kernel(float* __restrict__ proj, int ld, const float* __restrict__ bia
             float a = (row[base + c0] + (bias ? bias[base + c0] : 0.f)) * inv * nw[c0];
             float b = c1 < dim ? (row[base + c1] + (bias ? bias[base + c1] : 0.f)) * inv * nw[c1] : 0.f;
             if (c1 < rot_dims) {
-                float sn, cs;
-                sincosf((float)pos * freq[i], &sn, &cs);
+                const float sn = trig[i], cs = trig[n_turn + i];
                 const float ra = a * cs - b * sn, rb = b * cs + a * sn;
                 a = ra;
                 b = rb;
@@ -679,8 +690,12 @@ __global__ void gate_prep_kernel(float* __restrict__ proj, int ld, int q_off, in
 }
 
 // The recurrence.  Per head a state S [dim][vdim]; every value column c of S evolves on its own:
-//   S[:, c] <- a_t * S[:, c];   DELTA: u = beta_t (v_t[c] - S[:, c] . k_t), S[:, c] += k_t u;   else: S[:, c] += (1 - a_t) v_t[c]
-//   o_t[c] = S[:, c] . q_t
+//   S[:, c] <- a_t * S[:, c];   then by RULE (kScanTied / kScanDelta / kScanWrite of lm_internal.h)
+//     tied:  S[:, c] += (1 - a_t) v_t[c]
+//     delta: u = beta_t (v_t[c] - S[:, c] . k_t), S[:, c] += k_t u
+//     write: S[:, c] += k_t v_t[c]
+//   o_t[c] = S[:, c] . (q_mul q_t)
+// The decays may stand in a buffer of their own (a_in, row stride lda).
 // A column lives in the registers of 8 lanes (lane part holds rows part, part + 8, ...; its dot products are summed in
 // four interleaved partial sums, then across the 8 lanes); a CTA of 4 warps carries 16 columns of one head of one
 // scheduled sequence through the sequence's rows in order, 16 tokens staged in shared memory at a time while the next 16
@@ -688,18 +703,19 @@ __global__ void gate_prep_kernel(float* __restrict__ proj, int ld, int q_off, in
 // back at the end: state[slot][h][c][dim].
 constexpr int kScanThreads = 128, kScanCols = 16, kScanTT = 16;
 
-template <int RP, bool DELTA>
+template <int RP, int RULE>
 __global__ void __launch_bounds__(kScanThreads)
-column_scan_kernel(const float* __restrict__ in, int ld, int q_off, int k_off, int a_off, int v_off, int beta_off, int H, int G,
-                   int dim, int vdim, float* __restrict__ state, const int* __restrict__ seq_slot,
+column_scan_kernel(const float* __restrict__ in, int ld, int q_off, int k_off, const float* __restrict__ a_in, int lda, int v_off,
+                   int beta_off, int H, int G, int dim, int vdim, float* __restrict__ state, const int* __restrict__ seq_slot,
                    const int* __restrict__ seq_row0, const int* __restrict__ seq_count, const int* __restrict__ row_pos,
-                   float* __restrict__ o, int ldo, int head_decay) {
+                   float* __restrict__ o, int ldo, int head_decay, float q_mul) {
     extern __shared__ float sh[];
+    constexpr bool DELTA = RULE == kScanDelta, KEYS = RULE != kScanTied;
     constexpr int DS = 8 * RP;                                // staged row length (channels beyond dim hold zeros)
     float* sq = sh;                                           // [TT][DS]
     float* sa = sq + kScanTT * DS;                            // [TT][DS]
-    float* sk = sa + kScanTT * DS;                            // [TT][DS] (DELTA)
-    float* sv = sk + (DELTA ? kScanTT * DS : 0);              // [TT][16]
+    float* sk = sa + kScanTT * DS;                            // [TT][DS] (KEYS)
+    float* sv = sk + (KEYS ? kScanTT * DS : 0);               // [TT][16]
     float* sb = sv + kScanTT * kScanCols;                     // [TT] (DELTA)
     pdl_release();
     pdl_wait();
@@ -723,18 +739,20 @@ column_scan_kernel(const float* __restrict__ in, int ld, int q_off, int k_off, i
         const int idx = tid + kScanThreads * i, t = idx / DS, d = idx - t * DS;
         src[i] = d < dim ? t * ld + d : -1;
     }
-    const int qh = DELTA ? g : h;
-    float rq[RP], ra[RP], rk[DELTA ? RP : 1], rv[2], rb = 0.f;
+    const int qh = KEYS ? g : h;
+    float rq[RP], ra[RP], rk[KEYS ? RP : 1], rv[2], rb = 0.f;
     auto fetch = [&](int t0) {
         const int nt = min(kScanTT, n - t0);
         const float* base = in + (size_t)(row0 + t0) * ld;
+        const float* abase = a_in + (size_t)(row0 + t0) * lda;
 #pragma unroll
         for (int i = 0; i < RP; ++i) {
-            const bool ok = src[i] >= 0 && (tid + kScanThreads * i) / DS < nt;
-            rq[i] = ok ? base[src[i] + q_off + qh * dim] : 0.f;
-            // head_decay: column a_off + h of the row holds the one decay of all of the head's key channels
-            ra[i] = !ok ? 0.f : head_decay ? base[((tid + kScanThreads * i) / DS) * ld + a_off + h] : base[src[i] + a_off + h * dim];
-            if (DELTA) rk[i] = ok ? base[src[i] + k_off + g * dim] : 0.f;
+            const int t = (tid + kScanThreads * i) / DS, d = (tid + kScanThreads * i) - t * DS;
+            const bool ok = src[i] >= 0 && t < nt;
+            rq[i] = ok ? base[src[i] + q_off + qh * dim] * q_mul : 0.f;
+            // head_decay: column h of the decay row holds the one decay of all of the head's key channels
+            ra[i] = !ok ? 0.f : abase[t * lda + (head_decay ? h : h * dim + d)];
+            if (KEYS) rk[i] = ok ? base[src[i] + k_off + g * dim] : 0.f;
         }
 #pragma unroll
         for (int i = 0; i < 2; ++i) {
@@ -752,7 +770,7 @@ column_scan_kernel(const float* __restrict__ in, int ld, int q_off, int k_off, i
             const int idx = tid + kScanThreads * i;
             sq[idx] = rq[i];
             sa[idx] = ra[i];
-            if (DELTA) sk[idx] = rk[i];
+            if (KEYS) sk[idx] = rk[i];
         }
         sv[tid] = rv[0];
         sv[tid + kScanThreads] = rv[1];
@@ -795,6 +813,19 @@ column_scan_kernel(const float* __restrict__ in, int ld, int q_off, int k_off, i
                     d2 = fmaf(S[r + 2], q[8 * r + 16], d2);
                     d3 = fmaf(S[r + 3], q[8 * r + 24], d3);
                 }
+            } else if (KEYS) {
+                const float* k = sk + t * DS + part;
+#pragma unroll
+                for (int r = 0; r < RP; r += 4) {
+                    S[r] = fmaf(a[8 * r], S[r], k[8 * r] * v);
+                    S[r + 1] = fmaf(a[8 * r + 8], S[r + 1], k[8 * r + 8] * v);
+                    S[r + 2] = fmaf(a[8 * r + 16], S[r + 2], k[8 * r + 16] * v);
+                    S[r + 3] = fmaf(a[8 * r + 24], S[r + 3], k[8 * r + 24] * v);
+                    d0 = fmaf(S[r], q[8 * r], d0);
+                    d1 = fmaf(S[r + 1], q[8 * r + 8], d1);
+                    d2 = fmaf(S[r + 2], q[8 * r + 16], d2);
+                    d3 = fmaf(S[r + 3], q[8 * r + 24], d3);
+                }
             } else {
 #pragma unroll
                 for (int r = 0; r < RP; r += 4) {
@@ -828,12 +859,13 @@ column_scan_kernel(const float* __restrict__ in, int ld, int q_off, int k_off, i
 // The same column layout for a recurrence with scalar gates per (token, head):  S[:, c] <- a_t S[:, c] + (b_t k_t) v_t[c],
 // o_t[c] = S[:, c] . q_t.  Column vdim of every head is the normaliser: its value is the constant 1, so it carries
 // n <- a n + b k and reads out n . q.  State and read-out have vdim + 1 columns per head: state[slot][h][c][dim].
+// q and k have G heads (each serves H / G of the H); skip [H]: skip[h] v_t[c] joins the read-out.
 template <int RP>
 __global__ void __launch_bounds__(kScanThreads)
-scalar_gate_scan_kernel(const float* __restrict__ in, int ld, int q_off, int k_off, int a_off, int v_off, int b_off, int H, int dim,
-                        int vdim, float* __restrict__ state, const int* __restrict__ seq_slot, const int* __restrict__ seq_row0,
+scalar_gate_scan_kernel(const float* __restrict__ in, int ld, int q_off, int k_off, int a_off, int v_off, int b_off, int H, int G,
+                        int dim, int vdim, float* __restrict__ state, const int* __restrict__ seq_slot, const int* __restrict__ seq_row0,
                         const int* __restrict__ seq_count, const int* __restrict__ row_pos, float* __restrict__ o, int ldo,
-                        const float* __restrict__ fixed_decay, int normaliser) {
+                        const float* __restrict__ fixed_decay, int normaliser, const float* __restrict__ skip) {
     extern __shared__ float sh[];
     constexpr int DS = 8 * RP;
     float* sq = sh;                                           // [TT][DS]
@@ -846,9 +878,10 @@ scalar_gate_scan_kernel(const float* __restrict__ in, int ld, int q_off, int k_o
     // fixed_decay: a = fixed_decay[h] and b = 1 for every token (no gate columns are read); normaliser 0: vdim columns
     const int s = blockIdx.x, h = blockIdx.y, col0 = blockIdx.z * kScanCols, vcols = vdim + (normaliser ? 1 : 0);
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, part = lane & 7, cl = warp * 4 + (lane >> 3);
-    const int col = col0 + cl;
+    const int col = col0 + cl, g = h / (H / G);
     const int slot = seq_slot[s], row0 = seq_row0[s], n = seq_count[s], start = row_pos[row0];
     const bool col_ok = col < vcols;
+    const float sd = skip ? skip[h] : 0.f;
     const float a_fix = fixed_decay ? fixed_decay[h] : 0.f;
     float* st = state + (((size_t)slot * H + h) * vcols + (col_ok ? col : 0)) * dim;
     float S[RP];
@@ -870,8 +903,8 @@ scalar_gate_scan_kernel(const float* __restrict__ in, int ld, int q_off, int k_o
 #pragma unroll
         for (int i = 0; i < RP; ++i) {
             const bool ok = src[i] >= 0 && (tid + kScanThreads * i) / DS < nt;
-            rq[i] = ok ? base[src[i] + q_off + h * dim] : 0.f;
-            rk[i] = ok ? base[src[i] + k_off + h * dim] : 0.f;
+            rq[i] = ok ? base[src[i] + q_off + g * dim] : 0.f;
+            rk[i] = ok ? base[src[i] + k_off + g * dim] : 0.f;
         }
 #pragma unroll
         for (int i = 0; i < 2; ++i) {
@@ -902,7 +935,7 @@ scalar_gate_scan_kernel(const float* __restrict__ in, int ld, int q_off, int k_o
         for (int t = 0; t < nt; ++t) {
             const float* q = sq + t * DS + part;
             const float* k = sk + t * DS + part;
-            const float a = sa[t], u = sb[t] * sv[t * kScanCols + cl];
+            const float a = sa[t], v = sv[t * kScanCols + cl], u = sb[t] * v;
             float d0 = 0.f, d1 = 0.f, d2 = 0.f, d3 = 0.f;
 #pragma unroll
             for (int r = 0; r < RP; r += 4) {
@@ -919,7 +952,7 @@ scalar_gate_scan_kernel(const float* __restrict__ in, int ld, int q_off, int k_o
             dot += __shfl_xor_sync(0xffffffffu, dot, 1);
             dot += __shfl_xor_sync(0xffffffffu, dot, 2);
             dot += __shfl_xor_sync(0xffffffffu, dot, 4);
-            if (part == 0 && col_ok) o[(size_t)(row0 + t0 + t) * ldo + h * vcols + col] = dot;
+            if (part == 0 && col_ok) o[(size_t)(row0 + t0 + t) * ldo + h * vcols + col] = fmaf(sd, v, dot);
         }
     }
     if (col_ok) {
@@ -934,7 +967,8 @@ scalar_gate_scan_kernel(const float* __restrict__ in, int ld, int q_off, int k_o
 // o[r][h] <- o[r][h] / sqrt(mean(o[r][h]^2) + eps) * w [* gate[r][h]] in place (one warp per row and head), and its bf16 copy
 // gate_act: 0 the gate columns are used as they are (already activated), 1 sigmoid, 2 silu of them; w may be absent
 __global__ void head_norm_gate_kernel(float* __restrict__ o, int ldo, __nv_bfloat16* __restrict__ o_b, const float* __restrict__ w,
-                                      const float* __restrict__ gate, int ldg, int H, int vdim, float eps, int M, int gate_act) {
+                                      const float* __restrict__ gate, int ldg, int H, int vdim, float eps, int M, int gate_act,
+                                      float out_scale) {
     pdl_release();
     pdl_wait();
     const int idx = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
@@ -951,6 +985,7 @@ __global__ void head_norm_gate_kernel(float* __restrict__ o, int ldo, __nv_bfloa
             const float gz = gate[(size_t)r * ldg + (size_t)h * vdim + c];
             y *= gate_act == 1 ? sigmoidf_(gz) : gate_act == 2 ? siluf_(gz) : gz;
         }
+        y *= out_scale;
         row[c] = y;
         if (o_b) o_b[(size_t)r * ldo + (size_t)h * vdim + c] = __float2bfloat16_rn(y);
     }
@@ -983,8 +1018,8 @@ cudaError_t launch_talk_prep(float* proj, int ld, const float* bias, int q_off, 
                              const TalkShape& a, const float* qw, const float* kw, float eps, float* kcache, float* vcache,
                              const PageMap& pm, const RowMeta& rm, int M, cudaStream_t st) {
     if (a.rot_dims % 2 || a.rot_dims > a.dim) return cudaErrorInvalidValue;
-    return launch_pdl(talk_prep_kernel, dim3(M), dim3(256), 0, st, proj, ld, bias, q_off, k_off, v_off, gate_off, a.heads, a.kv_heads,
-                      a.dim, a.vdim, qw, kw, eps, a.scale, a.rot_freq, a.rot_dims, kcache, vcache, pm.table, pm.max_pages,
+    return launch_pdl(talk_prep_kernel, dim3(M), dim3(256), (size_t)a.rot_dims * sizeof(float), st, proj, ld, bias, q_off, k_off, v_off, gate_off, a.heads, a.kv_heads,
+                      a.dim, a.vdim, qw, kw, eps, a.scale, a.rot_freq, a.rot_dims, a.rot_amp != 0.f ? a.rot_amp : 1.f, kcache, vcache, pm.table, pm.max_pages,
                       pm.page_size, rm.slot, rm.pos);
 }
 
@@ -1075,18 +1110,18 @@ cudaError_t launch_conv_tail(const float* proj, int ld, int C, int taps, float* 
                       sm.count);
 }
 
-template <int RP, bool DELTA>
+template <int RP, int RULE>
 static cudaError_t launch_scan_inst(const float* in, int ld, const ScanInputs& si, int H, int G, int dim, int vdim, float* state,
                                     const SeqMeta& sm, const RowMeta& rm, int n_seq, float* o, int ldo, cudaStream_t st,
-                                    bool head_decay, bool early) {
-    const size_t smem = (size_t)((DELTA ? 3 : 2) * kScanTT * 8 * RP + kScanTT * kScanCols + kScanTT) * 4;
+                                    bool head_decay, bool early, const float* decay, int ldd, float q_mul) {
+    const size_t smem = (size_t)((RULE != kScanTied ? 3 : 2) * kScanTT * 8 * RP + kScanTT * kScanCols + kScanTT) * 4;
     if (smem > 48 * 1024) {
-        cudaError_t e = cudaFuncSetAttribute(column_scan_kernel<RP, DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaError_t e = cudaFuncSetAttribute(column_scan_kernel<RP, RULE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return e;
     }
-    return launch_pdl_if(early, column_scan_kernel<RP, DELTA>, dim3(n_seq, H, (vdim + kScanCols - 1) / kScanCols), dim3(kScanThreads), smem, st,
-                      in, ld, si.q_off, si.k_off, si.a_off, si.v_off, si.beta_off, H, G, dim, vdim, state, sm.slot, sm.row0,
-                      sm.count, rm.pos, o, ldo, head_decay ? 1 : 0);
+    return launch_pdl_if(early, column_scan_kernel<RP, RULE>, dim3(n_seq, H, (vdim + kScanCols - 1) / kScanCols), dim3(kScanThreads), smem, st,
+                      in, ld, si.q_off, si.k_off, decay ? decay : in + si.a_off, decay ? ldd : ld, si.v_off, si.beta_off, H, G, dim, vdim,
+                      state, sm.slot, sm.row0, sm.count, rm.pos, o, ldo, head_decay ? 1 : 0, q_mul);
 }
 
 cudaError_t launch_gate_prep(float* proj, int ld, int q_off, int f_off, int v_off, const float* bias, const float* lower, int n_qf,
@@ -1094,49 +1129,60 @@ cudaError_t launch_gate_prep(float* proj, int ld, int q_off, int f_off, int v_of
     return launch_pdl(gate_prep_kernel, dim3(M), dim3(256), 0, st, proj, ld, q_off, f_off, v_off, bias, lower, n_qf, n_v);
 }
 
-// delta: the delta rule (reads k and beta); otherwise the gate-tied write (its inputs prepared by launch_gate_prep)
-cudaError_t launch_column_scan(const float* in, int ld, const ScanInputs& si, bool delta, int H, int G, int dim, int vdim,
+// kScanTied: its inputs prepared by launch_gate_prep; kScanDelta reads k and beta; kScanWrite reads k
+cudaError_t launch_column_scan(const float* in, int ld, const ScanInputs& si, int rule, int H, int G, int dim, int vdim,
                                float* state, const SeqMeta& sm, const RowMeta& rm, int n_seq, float* o, int ldo,
-                               cudaStream_t st, bool head_decay, bool early) {
+                               cudaStream_t st, bool head_decay, bool early, const float* decay, int ldd, float q_mul) {
     if (dim > 256 || H % G || H > 65535) return cudaErrorNotSupported;
-#define SCAN_CASE(RP)                                                                                                    \
-    return delta ? launch_scan_inst<RP, true>(in, ld, si, H, G, dim, vdim, state, sm, rm, n_seq, o, ldo, st, head_decay, early) \
-                 : launch_scan_inst<RP, false>(in, ld, si, H, G, dim, vdim, state, sm, rm, n_seq, o, ldo, st, head_decay, early)
+#define SCAN_RULE(RP, RULE) \
+    return launch_scan_inst<RP, RULE>(in, ld, si, H, G, dim, vdim, state, sm, rm, n_seq, o, ldo, st, head_decay, early, decay, ldd, q_mul)
+#define SCAN_CASE(RP)                            \
+    switch (rule) {                              \
+        case kScanTied: SCAN_RULE(RP, kScanTied);   \
+        case kScanDelta: SCAN_RULE(RP, kScanDelta); \
+        case kScanWrite: SCAN_RULE(RP, kScanWrite); \
+        default: return cudaErrorInvalidValue;   \
+    }
     if (dim <= 32) SCAN_CASE(4);
     if (dim <= 64) SCAN_CASE(8);
     if (dim <= 128) SCAN_CASE(16);
     SCAN_CASE(32);
 #undef SCAN_CASE
+#undef SCAN_RULE
 }
 
 template <int RP>
-static cudaError_t launch_scalar_scan_inst(const float* in, int ld, const ScanInputs& si, int H, int dim, int vdim, float* state,
+static cudaError_t launch_scalar_scan_inst(const float* in, int ld, const ScanInputs& si, int H, int G, int dim, int vdim, float* state,
                                            const SeqMeta& sm, const RowMeta& rm, int n_seq, float* o, int ldo, cudaStream_t st,
-                                           const float* fixed_decay, bool normaliser, bool early) {
+                                           const float* fixed_decay, bool normaliser, bool early, const float* skip) {
     const size_t smem = (size_t)(2 * kScanTT * 8 * RP + kScanTT * kScanCols + 2 * kScanTT) * 4;
     if (smem > 48 * 1024) {
         cudaError_t e = cudaFuncSetAttribute(scalar_gate_scan_kernel<RP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return e;
     }
     return launch_pdl_if(early, scalar_gate_scan_kernel<RP>, dim3(n_seq, H, (vdim + (normaliser ? 1 : 0) + kScanCols - 1) / kScanCols),
-                      dim3(kScanThreads), smem, st, in, ld, si.q_off, si.k_off, si.a_off, si.v_off, si.beta_off, H, dim, vdim, state,
-                      sm.slot, sm.row0, sm.count, rm.pos, o, ldo, fixed_decay, normaliser ? 1 : 0);
+                      dim3(kScanThreads), smem, st, in, ld, si.q_off, si.k_off, si.a_off, si.v_off, si.beta_off, H, G, dim, vdim, state,
+                      sm.slot, sm.row0, sm.count, rm.pos, o, ldo, fixed_decay, normaliser ? 1 : 0, skip);
 }
 
 cudaError_t launch_scalar_gate_scan(const float* in, int ld, const ScanInputs& si, int H, int dim, int vdim, float* state,
                                     const SeqMeta& sm, const RowMeta& rm, int n_seq, float* o, int ldo, cudaStream_t st,
-                                    const float* fixed_decay, bool normaliser, bool early) {
-    if (dim > 256 || H > 65535) return cudaErrorNotSupported;
-    if (dim <= 32) return launch_scalar_scan_inst<4>(in, ld, si, H, dim, vdim, state, sm, rm, n_seq, o, ldo, st, fixed_decay, normaliser, early);
-    if (dim <= 64) return launch_scalar_scan_inst<8>(in, ld, si, H, dim, vdim, state, sm, rm, n_seq, o, ldo, st, fixed_decay, normaliser, early);
-    if (dim <= 128) return launch_scalar_scan_inst<16>(in, ld, si, H, dim, vdim, state, sm, rm, n_seq, o, ldo, st, fixed_decay, normaliser, early);
-    return launch_scalar_scan_inst<32>(in, ld, si, H, dim, vdim, state, sm, rm, n_seq, o, ldo, st, fixed_decay, normaliser, early);
+                                    const float* fixed_decay, bool normaliser, bool early, int G, const float* skip) {
+    if (G <= 0) G = H;
+    if (dim > 256 || H > 65535 || H % G) return cudaErrorNotSupported;
+#define SCALAR_CASE(RP) \
+    return launch_scalar_scan_inst<RP>(in, ld, si, H, G, dim, vdim, state, sm, rm, n_seq, o, ldo, st, fixed_decay, normaliser, early, skip)
+    if (dim <= 32) SCALAR_CASE(4);
+    if (dim <= 64) SCALAR_CASE(8);
+    if (dim <= 128) SCALAR_CASE(16);
+    SCALAR_CASE(32);
+#undef SCALAR_CASE
 }
 
 cudaError_t launch_head_norm_gate(float* o, int ldo, void* o_bf16, const float* w, const float* gate, int ldg, int H, int vdim,
-                                  float eps, int M, cudaStream_t st, int gate_act) {
+                                  float eps, int M, cudaStream_t st, int gate_act, float out_scale) {
     return launch_pdl(head_norm_gate_kernel, dim3((M * H + 7) / 8), dim3(256), 0, st, o, ldo, reinterpret_cast<__nv_bfloat16*>(o_bf16),
-                      w, gate, ldg, H, vdim, eps, M, gate_act);
+                      w, gate, ldg, H, vdim, eps, M, gate_act, out_scale);
 }
 
 }  // namespace lm

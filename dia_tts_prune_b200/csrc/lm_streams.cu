@@ -13,7 +13,8 @@
 //                             write it is the first read of a step; without in / w it is the plain sum of the streams
 //                             Options: a second output written with its own weights (a record whose sublayers read the same
 //                             streams), a second norm weight on the same statistics, RMS instead of layer norm, the input
-//                             row for assignments without a slot (identity experts), a sigmoid gate number on y
+//                             row for assignments without a slot (identity experts), a sigmoid gate number on y, an RMS norm
+//                             of y before it is written
 //   latent_prep_kernel        RMS norms of the query latent (in place, + bf16 operand) and of the key/value latent (into
 //                             the pages: the latent is all an attention layer of this kind caches - and, behind it, one
 //                             key part turned with the position where the layer has one)
@@ -94,6 +95,12 @@ streams_step_kernel(float* __restrict__ X, const float* __restrict__ mix, const 
     __syncthreads();
     const int r = rows ? rows[blockIdx.x] : blockIdx.x;
     float* xr = X + (size_t)r * s * D;
+    float y_inv = 1.f;                                        // y_norm_w: y / sqrt(mean(y^2) + eps) * y_norm_w is what is written
+    if (write && ex.y_norm_w) {
+        float ss = 0.f;
+        for (int c = tid; c < D; c += blockDim.x) ss = fmaf(y[(size_t)r * D + c], y[(size_t)r * D + c], ss);
+        y_inv = 1.0f / sqrtf(block_sum(ss, red) / (float)D + eps);
+    }
     auto load = [](const float* p, float (&v)[VW]) {
         if (VW == 4) {
             const float4 t = *reinterpret_cast<const float4*>(p);
@@ -121,6 +128,10 @@ streams_step_kernel(float* __restrict__ X, const float* __restrict__ mix, const 
 #pragma unroll
             for (int e = 0; e < VW; ++e) yv[e] = 0.f;
             if (y) load(y + (size_t)r * D + c, yv);
+            if (ex.y_norm_w) {
+#pragma unroll
+                for (int e = 0; e < VW; ++e) yv[e] *= y_inv * ex.y_norm_w[c + e];
+            }
             if (ex.y_gate) {                                  // one gate number per row on the unit's output
                 const float gt = sigmoidf_(ex.y_gate[(size_t)r * ex.y_gate_ld]);
 #pragma unroll
@@ -543,7 +554,7 @@ mlstm_gates_kernel(float* __restrict__ proj, int ld, int i_off, int f_off, const
 __global__ void __launch_bounds__(256)
 mlstm_finish_kernel(const float* __restrict__ raw, int ldr, const float* __restrict__ floor_in, float scale,
                     const float* __restrict__ w, const float* __restrict__ gate, int ldg, float eps, float* __restrict__ out,
-                    __nv_bfloat16* __restrict__ out_b, int M, int H, int vdim) {
+                    __nv_bfloat16* __restrict__ out_b, int ldo, float out_scale, int M, int H, int vdim) {
     pdl_release();
     pdl_wait();
     const int idx = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
@@ -559,10 +570,11 @@ mlstm_finish_kernel(const float* __restrict__ raw, int ldr, const float* __restr
     }
     ss = warp_sum(ss);
     const float inv = 1.0f / sqrtf(ss / (float)vdim + eps);
-    const size_t base = (size_t)r * H * vdim + (size_t)h * vdim;
+    const size_t base = (size_t)r * ldo + (size_t)h * vdim;
     for (int c = lane; c < vdim; c += 32) {
         float y = src[c] * mult * inv * w[(size_t)h * vdim + c];
         if (gate) y *= sigmoidf_(gate[(size_t)r * ldg + (size_t)h * vdim + c]);
+        y *= out_scale;
         out[base + c] = y;
         if (out_b) out_b[base + c] = __float2bfloat16_rn(y);
     }
@@ -658,9 +670,11 @@ cudaError_t launch_mlstm_gates(float* proj, int ld, int i_off, int f_off, const 
 }
 
 cudaError_t launch_mlstm_finish(const float* raw, int ldr, const float* floor_in, float scale, const float* w, const float* gate,
-                                int ldg, float eps, float* out, void* out_bf16, int M, int H, int vdim, cudaStream_t st) {
+                                int ldg, float eps, float* out, void* out_bf16, int M, int H, int vdim, cudaStream_t st, int ldo,
+                                float out_scale) {
+    if (ldo <= 0) ldo = H * vdim;
     return launch_pdl(mlstm_finish_kernel, dim3((M * H + 7) / 8), dim3(256), 0, st, raw, ldr, floor_in, scale, w, gate, ldg, eps,
-                      out, reinterpret_cast<__nv_bfloat16*>(out_bf16), M, H, vdim);
+                      out, reinterpret_cast<__nv_bfloat16*>(out_bf16), ldo, out_scale, M, H, vdim);
 }
 
 }  // namespace lm

@@ -1,5 +1,5 @@
 """Configuration schemas of the decoder-only language models (``config.json`` of a model folder): Pubopel, Kupelix,
-Luketar and Fipadra.
+Luketar, Fipadra and Loduzen.
 
 Every size and every per-model constant comes from the file.  Optional entries that are absent switch their
 mechanism off: no ``mask`` is full causal attention, no ``softcap`` leaves scores uncapped, ``mlp: null`` is a layer
@@ -396,7 +396,106 @@ class FipadraConfig(BaseModel, frozen=True):
                     raise ValueError(f"layer {i}: top ({f.router.top}) exceeds the router outputs a token may choose from ({per})")
 
 
-CONFIGS = {"pubopel": PubopelConfig, "kupelix": KupelixConfig, "luketar": LuketarConfig, "fipadra": FipadraConfig}
+# ---- Loduzen: pre-norm sublayers with RMS norms; windowed attention beside gated linear attention, or a state-space mixer; a gelu
+# ---- gated unit; a per-layer input looked up by the token ----
+class YarnConfig(BaseModel, frozen=True):
+    factor: float = Field(gt=0.0)
+    original: float = Field(gt=0.0)
+    fast: float = Field(gt=0.0)                  # turns over `original` positions where the ramp over the pairs begins ...
+    slow: float = Field(gt=0.0)                  # ... and where it ends
+
+
+class YarnRotConfig(BaseModel, frozen=True):
+    base: float = Field(gt=0.0)
+    dims: int = Field(ge=0)
+    scaling: Optional[YarnConfig] = None
+
+
+class KeyValueAttentionConfig(BaseModel, frozen=True):
+    heads: int = Field(gt=0)
+    kv_heads: Optional[int] = Field(default=None, gt=0)
+    dim: int = Field(gt=0)
+    vdim: int = Field(gt=0)
+    scale: float
+    rot: Optional[YarnRotConfig] = None
+    mask: Optional[WindowConfig] = None
+
+
+class GatedLinearConfig(BaseModel, frozen=True):
+    heads: int = Field(gt=0)
+    dim: int = Field(gt=0)
+    vdim: int = Field(gt=0)
+    tau: float = Field(gt=0.0)                   # decay = sigmoid(z)^(1 / tau)
+
+
+class PairMixerConfig(BaseModel, frozen=True):
+    left: KeyValueAttentionConfig
+    right: GatedLinearConfig
+    left_scale: float = 1.0
+    right_scale: float = 1.0
+
+
+class Mamba2MixerConfig(BaseModel, frozen=True):
+    heads: int = Field(gt=0)
+    vdim: int = Field(gt=0)
+    state: int = Field(gt=0)
+    groups: int = Field(gt=0)                    # groups of heads that share B and C
+    conv: int = Field(ge=1)
+    norm_groups: int = Field(default=1, gt=0)    # equal parts of the row that are normed on their own
+
+
+class LoduzenPairLayer(BaseModel, frozen=True):
+    type: Literal["parallel"]
+    mixer: PairMixerConfig
+    mlp: Optional[DenseMlpConfig] = None
+
+
+class LoduzenMamba2Layer(BaseModel, frozen=True):
+    type: Literal["mamba2"]
+    mixer: Mamba2MixerConfig
+    mlp: Optional[DenseMlpConfig] = None
+
+
+LoduzenLayer = Annotated[Union[LoduzenPairLayer, LoduzenMamba2Layer], Field(discriminator="type")]
+
+
+class TokenSideConfig(BaseModel, frozen=True):
+    dim: int = Field(gt=0)                       # channels per layer of the second embedding table
+
+
+class LoduzenConfig(BaseModel, frozen=True):
+    architecture: Literal["Loduzen"] = "Loduzen"
+    vocab: int = Field(gt=0)
+    width: int = Field(gt=0)
+    layers: list[LoduzenLayer] = Field(min_length=1)
+    norm: NormConfig
+    token_side: Optional[TokenSideConfig] = None
+
+    @classmethod
+    def load(cls, path: str | Path) -> "LoduzenConfig":
+        return cls.model_validate(json.loads(Path(path).read_text(encoding="utf-8")))
+
+    def check(self) -> None:
+        for i, layer in enumerate(self.layers):
+            m = layer.mixer
+            if layer.type == "mamba2":
+                if m.heads % m.groups:
+                    raise ValueError(f"layer {i}: heads ({m.heads}) must be a multiple of groups ({m.groups})")
+                if (m.heads * m.vdim) % m.norm_groups:
+                    raise ValueError(f"layer {i}: {m.heads * m.vdim} channels do not form {m.norm_groups} equal parts")
+                continue
+            a = m.left
+            g = a.kv_heads or a.heads
+            if a.heads % g:
+                raise ValueError(f"layer {i}: heads ({a.heads}) must be a multiple of kv_heads ({g})")
+            if a.vdim != a.dim:
+                raise ValueError(f"layer {i}: the values are the projected keys, so vdim ({a.vdim}) must equal dim ({a.dim})")
+            if a.rot is not None and (a.rot.dims % 2 or a.rot.dims > a.dim):
+                raise ValueError(f"layer {i}: rot.dims ({a.rot.dims}) must be even and at most dim ({a.dim})")
+
+
+CONFIGS = {"pubopel": PubopelConfig, "kupelix": KupelixConfig, "luketar": LuketarConfig, "fipadra": FipadraConfig,
+           "loduzen": LoduzenConfig}
 
 
 def load_config(raw: dict):

@@ -198,13 +198,13 @@ class LMEngine:
         return out
 
     def op_mixer_kernels(self, layer: int, proj: torch.Tensor, parts) -> torch.Tensor:
-        """The mixer kernels of a parallel-form record alone on stacked projections ``proj [M, n_in]`` (its attention or
-        recurrence without the products around it); the state of the sequences in ``parts`` is appended to."""
+        """The mixer kernels of a parallel- or stream-form record alone on stacked projections ``proj [M, n_in]`` (its attention
+        or recurrence without the products around it); the state of the sequences in ``parts`` is appended to."""
         buf, M, S, _ = self._pack([(s, [0] * n, p0, []) for s, n, p0 in parts])
         self.state.sync_table()
         m = self.layers[layer].mixer
         proj = proj.to(device=self.device, dtype=torch.float32).contiguous().clone()
-        out = torch.empty((M, m.heads * m.vdim), dtype=torch.float32, device=self.device)
+        out = torch.empty((M, int(m.w_o.shape[1])), dtype=torch.float32, device=self.device)
         _lm_lib.check(self.lib.lm_b200_op_mixer_kernels(self._h, layer, proj.data_ptr(), buf.data_ptr(), M, S, out.data_ptr(),
                                                         _stream(self.device)), "op_mixer_kernels")
         return out
@@ -214,6 +214,16 @@ class LMEngine:
         y = torch.empty_like(h)
         _lm_lib.check(self.lib.lm_b200_op_ff(self._h, layer, h.data_ptr(), h.shape[0], y.data_ptr(), _stream(self.device)), "op_ff")
         return y
+
+    def op_token_input(self, layer: int, x: torch.Tensor, tokens: list[int]) -> torch.Tensor:
+        """``x [M, width]`` plus the token input of ``layer`` for the rows' ``tokens``."""
+        x = x.to(device=self.device, dtype=torch.float32).contiguous()
+        seq = Sequence(name="", slot=0)
+        buf, M, _, _ = self._pack([(seq, list(tokens), 0, [])])
+        out = torch.empty_like(x)
+        _lm_lib.check(self.lib.lm_b200_op_token_input(self._h, layer, x.data_ptr(), buf.data_ptr(), M, out.data_ptr(),
+                                                      _stream(self.device)), "op_token_input")
+        return out
 
 
 def linear(a: torch.Tensor, w_bf16: torch.Tensor, tensor_cores: bool = False) -> torch.Tensor:

@@ -35,12 +35,20 @@ Beside ``layers.py`` (Dia's RMSNorm / rotary attention / gated MLP modules) this
   * :class:`DenseRelu2` - up projection, squared relu, down projection;
   * options of :class:`RoutedExperts`: scores from the softmax over ALL router outputs, a correction that only the choice
     sees, choice inside the best groups of neighbouring outputs, normalised and scaled weights, identity experts, a
-    sigmoid gate number on the shared unit.
+    sigmoid gate number on the shared unit;
+  * :class:`RotaryAttention` - grouped-query attention with per-head q / k RMS norms, rotary positions (with an amplitude), a
+    sliding window and a value-less sink logit, whose values may be the projected keys themselves;
+  * :class:`GatedLinear` - linear attention with a data-dependent decay per head and key channel, sigmoid(z)^(1 / tau);
+  * :class:`Mamba2` - state-space mixer: short convolution, step sizes, one decay per head, B and C shared by groups of heads, a
+    skip term, the gate before a grouped norm;
+  * :class:`PairMixer` - any two mixers of the stream form side by side on one input, their outputs weighted and added;
+  * ``GatedUnit(act="gelu")`` - the tanh form of gelu on the gate branch;
+  * :class:`TokenInput` - what a layer adds for the token itself: a gated slice of a second embedding table, normed.
 All constants are constructor arguments; a design picks and combines them per layer (:class:`MixLayer` runs its
 sublayers one after the other, :class:`ParallelLayer` feeds one norm to mixer and feed-forward and adds both,
 :class:`StreamLayer` runs pre-norm sublayers over hyper-connected streams - with ``parallel`` both sublayers read the
 streams before either writes).  The arithmetic lives in
-``csrc/lm_kernels.cu``, ``csrc/lm_mixers.cu`` and ``csrc/lm_streams.cu``; these classes only keep device tensors alive
+``csrc/lm_kernels.cu``, ``csrc/lm_mixers.cu``, ``csrc/lm_streams.cu`` and ``csrc/lm_linear.cu``; these classes only keep device tensors alive
 and fill ``lm_b200_layer``.
 """
 
@@ -200,6 +208,28 @@ def rotary_angles(base: float, dims: int, scaling=None) -> torch.Tensor:
                 f = (1.0 - t) * f / factor + t * f
         out.append(f)
     return torch.tensor(out, dtype=torch.float64).to(torch.float32)
+
+
+def yarn_angles(base: float, dims: int, scaling=None) -> tuple[torch.Tensor, float]:
+    """(angle per position of each of the ``dims / 2`` rotary pairs, multiplier of cosine and sine).  ``scaling`` (factor,
+    original, fast, slow): pair i turns at a blend of its full rate and ``1 / factor`` of it, along a linear ramp over i between
+    the pairs that make ``fast`` and ``slow`` turns in ``original`` positions; the multiplier is 1 + ln(factor) / 10."""
+    full = [float(base) ** (-2.0 * i / dims) for i in range(dims // 2)]
+    if scaling is None:
+        return torch.tensor(full, dtype=torch.float64).to(torch.float32), 1.0
+    factor, original = float(scaling.factor), float(scaling.original)
+
+    def pair_with(turns: float) -> float:                         # the (real) pair index that makes `turns` turns
+        return dims * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(float(base)))
+
+    first = max(math.floor(pair_with(float(scaling.fast))), 0)
+    last = min(math.ceil(pair_with(float(scaling.slow))), dims - 1)
+    span = max(last - first, 0.001)
+    out = []
+    for i, f in enumerate(full):
+        slow = min(max((i - first) / span, 0.0), 1.0)
+        out.append(f / factor * slow + f * (1.0 - slow))
+    return torch.tensor(out, dtype=torch.float64).to(torch.float32), 0.1 * math.log(factor) + 1.0
 
 
 class TalkingAttention:
@@ -543,6 +573,158 @@ class Retention:
         rec.rec_state = st.rec_state.data_ptr()
 
 
+class RotaryAttention:
+    kind = "rotary_attention"
+
+    def __init__(self, w_q, w_k, w_v, w_o, q_norm, k_norm, *, heads: int, kv_heads: int, dim: int, scale: float, rot_angles=None,
+                 rot_amp: float = 1.0, window: int | None = None, sink=None, device=None):
+        """``w_v`` None: the values are the projected keys, before norm and rotation.  ``sink [heads]``: logits that join the
+        softmax's denominator only.  ``rot_amp`` multiplies cosine and sine."""
+        self.heads, self.kv_heads, self.dim, self.vdim, self.scale = int(heads), int(kv_heads), int(dim), int(dim), float(scale)
+        if (tuple(w_q.shape)[0] != heads * dim or tuple(w_k.shape)[0] != kv_heads * dim or heads % kv_heads
+                or (w_v is not None and tuple(w_v.shape)[0] != kv_heads * dim)):
+            raise ValueError("projection shapes do not match heads x dim")
+        self.own_values = w_v is not None
+        self.in_rows, self.in_bias, self.w_o = [w_q, w_k] + ([w_v] if self.own_values else []), None, w_o
+        self.q_norm, self.k_norm = _f32(q_norm, device), _f32(k_norm, device)
+        self.rot = None if rot_angles is None or rot_angles.numel() == 0 else _f32(rot_angles, device)
+        self.rot_amp, self.window = float(rot_amp), int(window) if window else 0
+        self.sink = None if sink is None else _f32(sink, device)
+
+    def state_spec(self) -> StateSpec:
+        return StateSpec(kv=(self.kv_heads, self.dim, self.dim))
+
+    def fill(self, rec, st) -> None:
+        from ._lm_lib import GATE_NONE, MIXER_ROTARY_ATTENTION, ROT_INTERLEAVED
+        rec.mixer, rec.mixer_gate = MIXER_ROTARY_ATTENTION, GATE_NONE
+        rec.heads, rec.kv_heads, rec.dim, rec.vdim, rec.scale = self.heads, self.kv_heads, self.dim, self.vdim, self.scale
+        rec.values_are_keys, rec.window = 0 if self.own_values else 1, self.window
+        rec.q_norm, rec.k_norm = self.q_norm.data_ptr(), self.k_norm.data_ptr()
+        rec.rot_dims = 2 * self.rot.numel() if self.rot is not None else 0
+        rec.rot_freq = self.rot.data_ptr() if self.rot is not None else None
+        rec.rot_layout, rec.rot_amp = ROT_INTERLEAVED, self.rot_amp
+        rec.sink = self.sink.data_ptr() if self.sink is not None else None
+        rec.k_pages, rec.v_pages = st.k_pages.data_ptr(), st.v_pages.data_ptr()
+
+
+class GatedLinear:
+    kind = "gated_linear"
+
+    def __init__(self, w_q, w_k, w_v, w_gate, w_a1, w_a2, w_o, head_norm, *, heads: int, dim: int, vdim: int, tau: float, b_a=None,
+                 gate: str | None = "silu", device=None):
+        """Per head S_t = diag(alpha_t) S_(t-1) + k_t v_t^T, o_t = S_t^T q_t dim^-1/2 with alpha = sigmoid(w_a2 w_a1 h + b_a)^(1 / tau)
+        per head and key channel; o / rms(o) x ``head_norm [vdim]`` x gate(w_gate h)."""
+        self.heads, self.dim, self.vdim, self.tau = int(heads), int(dim), int(vdim), float(tau)
+        self.rank, self.gate = int(w_a1.shape[0]), gate
+        if (tuple(w_q.shape)[0] != heads * dim or tuple(w_k.shape)[0] != heads * dim or tuple(w_v.shape)[0] != heads * vdim
+                or tuple(w_a2.shape) != (heads * dim, self.rank)):
+            raise ValueError("projection shapes do not match heads x dim")
+        self.in_rows = [w_q, w_k, w_v] + ([w_gate] if gate is not None else []) + [w_a1]
+        self.in_bias, self.w_o = None, w_o
+        self.w_a2 = _bf16(w_a2, device)
+        self.b_a = None if b_a is None else _f32(b_a, device)
+        self.head_norm = _f32(head_norm, device)
+
+    def state_spec(self) -> StateSpec:
+        return StateSpec(recurrent=(self.heads, self.vdim, self.dim))
+
+    def fill(self, rec, st) -> None:
+        from ._lm_lib import MIXER_GATED_LINEAR
+        rec.mixer, rec.mixer_gate = MIXER_GATED_LINEAR, _gate_kind(self.gate)
+        rec.heads, rec.kv_heads, rec.dim, rec.vdim = self.heads, self.heads, self.dim, self.vdim
+        rec.rank_a, rec.decay_tau, rec.w_a2 = self.rank, self.tau, self.w_a2.data_ptr()
+        rec.dt_bias = self.b_a.data_ptr() if self.b_a is not None else None
+        rec.head_norm, rec.rec_state = self.head_norm.data_ptr(), st.rec_state.data_ptr()
+
+
+class Mamba2:
+    kind = "mamba2"
+
+    def __init__(self, w_in, conv_w, conv_b, dt_bias, a_log, skip, norm, w_o, *, heads: int, state: int, groups: int, vdim: int,
+                 norm_groups: int = 1, device=None):
+        """``w_in`` rows: z (heads x vdim) | x (heads x vdim) | B (groups x state) | C (groups x state) | dt (heads); ``conv_w`` over
+        the channels of x | B | C.  Per head S <- exp(-exp(a_log) dt) S + dt B x^T, y = S^T C + skip x; y silu(z) is normed in
+        ``norm_groups`` equal parts, x ``norm``."""
+        self.heads, self.dim, self.kv_heads, self.vdim = int(heads), int(state), int(groups), int(vdim)
+        self.channels, self.taps, self.norm_groups = heads * vdim + 2 * groups * state, int(conv_w.shape[1]), int(norm_groups)
+        if tuple(w_in.shape)[0] != heads * vdim + self.channels + heads or tuple(conv_w.shape)[0] != self.channels or heads % groups:
+            raise ValueError("projection shapes do not match heads x vdim and groups x state")
+        self.in_rows, self.in_bias, self.w_o = [w_in], None, w_o
+        self.conv_w, self.conv_b = _f32(conv_w, device), None if conv_b is None else _f32(conv_b, device)
+        self.dt_bias, self.a_log, self.skip, self.norm = (_f32(t, device) for t in (dt_bias, a_log, skip, norm))
+
+    def state_spec(self) -> StateSpec:
+        return StateSpec(recurrent=(self.heads, self.vdim, self.dim), conv=(self.taps, self.channels))
+
+    def fill(self, rec, st) -> None:
+        from ._lm_lib import GATE_NONE, MIXER_MAMBA2
+        rec.mixer, rec.mixer_gate = MIXER_MAMBA2, GATE_NONE
+        rec.heads, rec.kv_heads, rec.dim, rec.vdim = self.heads, self.kv_heads, self.dim, self.vdim
+        rec.conv_taps, rec.norm_groups = self.taps, self.norm_groups
+        rec.conv_w, rec.conv_b = self.conv_w.data_ptr(), self.conv_b.data_ptr() if self.conv_b is not None else None
+        rec.a_log, rec.dt_bias, rec.skip_d = self.a_log.data_ptr(), self.dt_bias.data_ptr(), self.skip.data_ptr()
+        rec.head_norm, rec.rec_state, rec.conv_tail = self.norm.data_ptr(), st.rec_state.data_ptr(), st.conv_tail.data_ptr()
+
+
+def _stack_rows(mixer, device) -> tuple[torch.Tensor, torch.Tensor | None]:
+    """A stream mixer's stacked input projections, padded to a multiple of 4 rows, and their biases (None: no biases)."""
+    rows = [_bf16(r, device) for r in mixer.in_rows]
+    n = sum(int(r.shape[0]) for r in rows)
+    n_in = (n + 3) & ~3
+    if n_in > n:
+        rows.append(torch.zeros((n_in - n, int(rows[0].shape[1])), dtype=torch.bfloat16, device=device))
+    bias = None
+    if mixer.in_bias is not None:
+        b = torch.cat([_f32(x, device).reshape(-1) for x in mixer.in_bias])
+        bias = torch.cat([b, torch.zeros(n_in - b.numel(), dtype=torch.float32, device=device)]).contiguous()
+    return torch.cat(rows, dim=0).contiguous(), bias
+
+
+class PairMixer:
+    kind = "pair"
+
+    def __init__(self, left, right, left_scale: float = 1.0, right_scale: float = 1.0, device=None):
+        """``left_scale`` left(h) + ``right_scale`` right(h): the rows of both mixers' projections are one stacked matrix, and their
+        output projections stand side by side in another (the scales go on the outputs in front of it)."""
+        self.parts, self.scales = (left, right), (float(left_scale), float(right_scale))
+        stacked = [_stack_rows(m, device) for m in self.parts]
+        self.part_rows, self.part_bias = [int(w.shape[0]) for w, _ in stacked], [b for _, b in stacked]
+        self.in_rows, self.in_bias = [w for w, _ in stacked], None
+        self.w_o = torch.cat([_bf16(m.w_o, device) for m in self.parts], dim=1)
+        self._records: list = []
+
+    def state_spec(self) -> StateSpec:
+        return StateSpec(parts=tuple(m.state_spec() for m in self.parts))
+
+    def fill(self, rec, st) -> None:
+        import ctypes as C
+
+        from ._lm_lib import GATE_NONE, MIXER_PAIR, Layer
+        rec.mixer, rec.mixer_gate = MIXER_PAIR, GATE_NONE
+        for q, mixer in enumerate(self.parts):
+            sub = Layer()
+            mixer.fill(sub, st.parts[q])
+            sub.n_in = self.part_rows[q]
+            sub.in_bias = self.part_bias[q].data_ptr() if self.part_bias[q] is not None else None
+            self._records.append(sub)                             # alive until the engine has copied it
+            rec.part[q], rec.part_scale[q] = C.addressof(sub), self.scales[q]
+
+
+class TokenInput:
+    def __init__(self, table, offset: int, w_gate, w_proj, norm, device=None):
+        """x <- x + rms(w_proj (gelu(w_gate x) * e)) ``norm`` with e = columns ``offset`` .. of the token's row of ``table`` (bfloat16
+        on the device, shared by the layers)."""
+        self.table, self.offset, self.dim = table, int(offset), int(w_gate.shape[0])
+        if table.dtype != torch.bfloat16 or not table.is_contiguous() or self.offset + self.dim > int(table.shape[1]):
+            raise ValueError("the token table must be contiguous bfloat16 and hold the layer's columns")
+        self.w_gate, self.w_proj, self.norm = _bf16(w_gate, device), _bf16(w_proj, device), _f32(norm, device)
+
+    def fill(self, rec) -> None:
+        rec.side_dim, rec.side_ld, rec.side_off = self.dim, int(self.table.shape[1]), self.offset
+        rec.side_table, rec.w_side_gate, rec.w_side_proj = self.table.data_ptr(), self.w_gate.data_ptr(), self.w_proj.data_ptr()
+        rec.side_norm = self.norm.data_ptr()
+
+
 class DenseRelu2:
     def __init__(self, w_up, w_down, device=None):
         """``down(max(up h, 0)^2)``."""
@@ -560,8 +742,11 @@ class RmsNorm:
 
 
 class GatedUnit:
-    def __init__(self, w_gate, w_up, w_down, *, limit: float | None, device=None):
-        """``down(act(gate h, up h))``; with ``limit`` the clamped activation, without it silu(g) u."""
+    def __init__(self, w_gate, w_up, w_down, *, limit: float | None = None, act: str = "silu", device=None):
+        """``down(act(gate h, up h))``; with ``limit`` the clamped activation, without it silu(g) u or gelu(g) u (``act``)."""
+        if act not in ("silu", "gelu") or (limit is not None and act != "silu"):
+            raise ValueError("act must be 'silu' or 'gelu'; the clamped activation has a form of its own")
+        self.act = act
         self.ff, self.limit = int(w_gate.shape[0]), None if limit is None else float(limit)
         self.w_gate_up, self.w_down = _bf16(torch.cat([w_gate, w_up], dim=0), device), _bf16(w_down, device)
 
@@ -573,32 +758,28 @@ class StreamLayer:
     with another layer's weights): each record gets a state of its own."""
 
     def __init__(self, norm1, hc1: HyperConnection, mixer, ff=None, norm2=None, hc2: HyperConnection | None = None, device=None,
-                 parallel: bool = False, rms: bool = False):
+                 parallel: bool = False, rms: bool = False, side: TokenInput | None = None):
         """``parallel``: the feed-forward reads the streams as they were before the mixer's write, and both outputs are
-        written at once (with one stream: x += mixer(norm1 x) + ff(norm2 x)).  ``rms``: the norms are RMS norms."""
+        written at once (with one stream: x += mixer(norm1 x) + ff(norm2 x)).  ``rms``: the norms are RMS norms.  ``side``: a
+        token input after the feed-forward (one stream)."""
         self.mixer, self.ff, self.hc1, self.hc2 = mixer, ff, hc1, hc2
         self.parallel, self.rms = bool(parallel), bool(rms)
         self.norm1 = _f32(norm1, device)
         self.norm2 = None if norm2 is None else _f32(norm2, device)
         if ff is not None and (norm2 is None or hc2 is None or hc2.streams != hc1.streams):
             raise ValueError("a feed-forward sublayer needs its norm and hyper-connection weights")
-        rows = [_bf16(r, device) for r in mixer.in_rows]
-        n = sum(int(r.shape[0]) for r in rows)
-        self.n_in = (n + 3) & ~3
-        if self.n_in > n:
-            rows.append(torch.zeros((self.n_in - n, int(rows[0].shape[1])), dtype=torch.bfloat16, device=device))
-        self.w_in = torch.cat(rows, dim=0).contiguous()
-        self.in_bias = None
-        if mixer.in_bias is not None:
-            b = torch.cat([_f32(x, device).reshape(-1) for x in mixer.in_bias])
-            self.in_bias = torch.cat([b, torch.zeros(self.n_in - b.numel(), dtype=torch.float32, device=device)]).contiguous()
+        self.side = side
+        if side is not None and hc1.streams != 1:
+            raise ValueError("a token input needs one residual stream")
+        self.w_in, self.in_bias = _stack_rows(mixer, device)
+        self.n_in = int(self.w_in.shape[0])
         self.w_o = _bf16(mixer.w_o, device)
 
     def state_spec(self) -> StateSpec:
         return self.mixer.state_spec()
 
     def fill(self, rec, st) -> None:
-        from ._lm_lib import (ACT_CLAMPED_GLU, ACT_RELU2, ACT_SILU_GLU, FF_DENSE, FF_NONE, FF_ROUTED_EXPERTS, FORM_STREAMS,
+        from ._lm_lib import (ACT_CLAMPED_GLU, ACT_GELU_GLU, ACT_RELU2, ACT_SILU_GLU, FF_DENSE, FF_NONE, FF_ROUTED_EXPERTS, FORM_STREAMS,
                               NORM_LAYER, NORM_RMS, ROUTER_SIGMOID_INPUT, ROUTER_SOFTMAX_GROUPED, ROUTER_SOFTMAX_TOP)
         norm_kind = NORM_RMS if self.rms else NORM_LAYER
         rec.form, rec.streams, rec.parallel = FORM_STREAMS, self.hc1.streams, 1 if self.parallel else 0
@@ -609,6 +790,8 @@ class StreamLayer:
         self.mixer.fill(rec, st)
         rec.n_in, rec.w_in, rec.w_o = self.n_in, self.w_in.data_ptr(), self.w_o.data_ptr()
         rec.in_bias = self.in_bias.data_ptr() if self.in_bias is not None else None
+        if self.side is not None:
+            self.side.fill(rec)
         rec.ff = FF_NONE
         f = self.ff
         if f is None:
@@ -622,6 +805,8 @@ class StreamLayer:
         rec.act_limit = f.limit if f.limit is not None else 0.0
         if isinstance(f, GatedUnit):
             rec.ff, rec.dense_ff = FF_DENSE, f.ff
+            if f.act == "gelu":
+                rec.act = ACT_GELU_GLU
             rec.ws_gate_up, rec.ws_down = f.w_gate_up.data_ptr(), f.w_down.data_ptr()
             return
         rec.ff = FF_ROUTED_EXPERTS

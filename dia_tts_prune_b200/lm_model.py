@@ -18,11 +18,12 @@ from pathlib import Path
 import torch
 
 from .checkpoint import load_safetensors
-from .lm_config import FipadraConfig, KupelixConfig, LuketarConfig, PubopelConfig, load_config
+from .lm_config import FipadraConfig, KupelixConfig, LoduzenConfig, LuketarConfig, PubopelConfig, load_config
 from .lm_engine import LMEngine
-from .lm_layers import (ChannelDelta, DenseRelu2, DenseXielu, DynamicTanh, GatedDelta, GatedUnit, Hgrn2, HyperConnection,
-                        LatentAttention, LayerNorm, LayerRun, MixLayer, MLstm, ParallelLayer, Retention, RmsNorm, RoutedExperts,
-                        SinkAttention, StreamLayer, TalkingAttention, TapMix, rotary_angles)
+from .lm_layers import (ChannelDelta, DenseRelu2, DenseXielu, DynamicTanh, GatedDelta, GatedLinear, GatedUnit, Hgrn2,
+                        HyperConnection, LatentAttention, LayerNorm, LayerRun, Mamba2, MixLayer, MLstm, PairMixer, ParallelLayer,
+                        Retention, RmsNorm, RotaryAttention, RoutedExperts, SinkAttention, StreamLayer, TalkingAttention, TapMix,
+                        TokenInput, rotary_angles, yarn_angles)
 from .lm_state import OutOfPages, PagedState, Sequence
 
 
@@ -175,6 +176,44 @@ def build_fipadra_layers(cfg: FipadraConfig, w: dict[str, torch.Tensor], device)
     return layers, RmsNorm(w["final.norm"], device)
 
 
+def build_loduzen_layers(cfg: LoduzenConfig, w: dict[str, torch.Tensor], device) -> tuple[list[StreamLayer], RmsNorm]:
+    """The layer records of a Loduzen checkpoint (tensor names ``l<i>.norm1``, ``l<i>.mix.left.q``, ``l<i>.mix.right.a1``,
+    ``l<i>.mix.in``, ``l<i>.mlp.*``, ``l<i>.side.*``, ``side.embed``): stream records with one plain residual stream, RMS norms, the
+    sublayers one after the other, and a token input at the end of every layer."""
+    residual = HyperConnection.residual(device)
+    table = None
+    if cfg.token_side is not None:
+        table = w["side.embed"].detach().to(device=device, dtype=torch.bfloat16).contiguous()
+    layers = []
+    for i, lc in enumerate(cfg.layers):
+        p, m = f"l{i}.mix.", lc.mixer
+        t = lambda name: w[p + name]                             # noqa: E731
+        if lc.type == "mamba2":
+            mixer = Mamba2(t("in"), t("conv"), t("conv.b"), t("dt_bias"), t("A_log"), t("D"), t("norm"), t("o"), heads=m.heads,
+                           state=m.state, groups=m.groups, vdim=m.vdim, norm_groups=m.norm_groups, device=device)
+        else:
+            a, r = m.left, m.right
+            angles, amp = yarn_angles(a.rot.base, a.rot.dims, a.rot.scaling) if a.rot is not None and a.rot.dims > 0 else (None, 1.0)
+            left = RotaryAttention(t("left.q"), t("left.k"), None, t("left.o"), t("left.q.norm"), t("left.k.norm"), heads=a.heads,
+                                   kv_heads=a.kv_heads or a.heads, dim=a.dim, scale=a.scale, rot_angles=angles, rot_amp=amp,
+                                   window=a.mask.size if a.mask else None, sink=torch.zeros(a.heads), device=device)
+            right = GatedLinear(t("right.q"), t("right.k"), t("right.v"), t("right.g"), t("right.a1"), t("right.a2"), t("right.o"),
+                                t("right.norm"), heads=r.heads, dim=r.dim, vdim=r.vdim, tau=r.tau, b_a=t("right.a2.b"), gate="silu",
+                                device=device)
+            mixer = PairMixer(left, right, m.left_scale, m.right_scale, device=device)
+        ff = norm2 = side = None
+        if lc.mlp is not None:
+            q = f"l{i}.mlp."
+            norm2 = w[f"l{i}.norm2"]
+            ff = GatedUnit(w[q + "gate"], w[q + "up"], w[q + "down"], act="gelu", device=device)
+        if table is not None:
+            q = f"l{i}.side."
+            side = TokenInput(table, i * cfg.token_side.dim, w[q + "gate"], w[q + "proj"], w[q + "norm"], device=device)
+        layers.append(StreamLayer(w[f"l{i}.norm1"], residual, mixer, ff, norm2, residual if ff is not None else None, device=device,
+                                  rms=True, side=side))
+    return layers, RmsNorm(w["final.norm"], device)
+
+
 @dataclass
 class Request:
     name: str
@@ -261,8 +300,8 @@ class Scheduler:
 
 
 class CausalLM:
-    def __init__(self, cfg: PubopelConfig | KupelixConfig | LuketarConfig | FipadraConfig, weights: dict[str, torch.Tensor], dtype: str = "bfloat16", device=None,
-                 max_tokens: int = 4096, max_sequences: int = 8, page_size: int = 16, max_rows: int = 1024,
+    def __init__(self, cfg: PubopelConfig | KupelixConfig | LuketarConfig | FipadraConfig | LoduzenConfig,
+                 weights: dict[str, torch.Tensor], dtype: str = "bfloat16", device=None, max_tokens: int = 4096, max_sequences: int = 8, page_size: int = 16, max_rows: int = 1024,
                  max_sequence_tokens: int | None = None, step_graphs: bool = True):
         if dtype not in ("bfloat16", "float32"):
             raise ValueError("dtype must be 'bfloat16' or 'float32'")
@@ -277,6 +316,9 @@ class CausalLM:
             self.layers, final_norm = build_fipadra_layers(cfg, weights, self.device)
             taps, logit_scale = 0, cfg.logit_scale
             head, embed_norm = weights["embed"], weights["embed.norm"]    # logits against the table itself; a norm behind the lookup
+        elif isinstance(cfg, LoduzenConfig):
+            self.layers, final_norm = build_loduzen_layers(cfg, weights, self.device)
+            taps, logit_scale, head = 0, 1.0, weights["embed"]    # logits against the table itself
         elif isinstance(cfg, KupelixConfig):
             self.layers, final_norm = build_kupelix_layers(cfg, weights, self.device)
             taps, logit_scale = 0, cfg.logit_scale

@@ -27,6 +27,7 @@ class StateSpec:
     conv: tuple[int, int] | None = None             # (taps, channels): the last taps - 1 inputs of a short convolution
     latent: int | None = None                       # size of a paged latent vector per token (keys and values are made from it)
     aux: int = 0                                    # fp32 numbers per slot beside a recurrent state (running maxima)
+    parts: tuple = ()                               # StateSpecs of a record's mixers, when it has several
 
 
 class OutOfPages(RuntimeError):
@@ -51,6 +52,7 @@ class RecordState:
     conv_tail: torch.Tensor | None
     latent_pages: torch.Tensor | None = None
     rec_aux: torch.Tensor | None = None
+    parts: tuple = ()                               # RecordStates of the spec's parts
 
 
 class PagedState:
@@ -68,23 +70,13 @@ class PagedState:
         self.n_pages = -(-int(max_tokens) // self.page_size) + self.n_slots
         self.taps = int(taps)
         self.specs = [sp if isinstance(sp, StateSpec) else StateSpec(kv=(sp[0], sp[1], sp[1]), tap_tails=2) for sp in layers]
-        f32 = dict(dtype=torch.float32, device=self.device)
-        # K and V pages per record: [page][kv head][page_size][size], float32 (None for a record without attention)
-        self.k_pages = [torch.zeros((self.n_pages, sp.kv[0], self.page_size, sp.kv[1]), **f32) if sp.kv else None
-                        for sp in self.specs]
-        self.v_pages = [torch.zeros((self.n_pages, sp.kv[0], self.page_size, sp.kv[2]), **f32) if sp.kv else None
-                        for sp in self.specs]
-        # the last taps - 1 normed inputs of the tap-mix sublayers of every record: [slot][taps - 1][width]
-        t1 = max(self.taps - 1, 1)
-        self.tails = [tuple(torch.zeros((self.n_slots, t1, width), **f32) for _ in range(sp.tap_tails)) for sp in self.specs]
-        # recurrent matrix states [slot][head][value channel][key channel] and short-convolution tails [slot][taps - 1][channels]
-        self.rec_states = [torch.zeros((self.n_slots, sp.recurrent[0], sp.recurrent[1], sp.recurrent[2]), **f32)
-                           if sp.recurrent else None for sp in self.specs]
-        self.conv_tails = [torch.zeros((self.n_slots, max(sp.conv[0] - 1, 1), sp.conv[1]), **f32) if sp.conv else None
-                           for sp in self.specs]
-        # latent pages [page][page_size][size] share the page table with the K/V pages; per-slot numbers [slot][aux]
-        self.latent_pages = [torch.zeros((self.n_pages, self.page_size, sp.latent), **f32) if sp.latent else None for sp in self.specs]
-        self.rec_aux = [torch.zeros((self.n_slots, sp.aux), **f32) if sp.aux else None for sp in self.specs]
+        self.width = int(width)
+        self.records = [self._allocate(sp) for sp in self.specs]
+        # the same buffers by kind, one entry per record (None where a record has no such part of its own)
+        self.k_pages, self.v_pages = [r.k_pages for r in self.records], [r.v_pages for r in self.records]
+        self.tails, self.conv_tails = [r.tails for r in self.records], [r.conv_tail for r in self.records]
+        self.rec_states, self.rec_aux = [r.rec_state for r in self.records], [r.rec_aux for r in self.records]
+        self.latent_pages = [r.latent_pages for r in self.records]
         self._table_host = torch.zeros((self.n_slots, self.max_pages), dtype=torch.int32).pin_memory() \
             if self.device.type == "cuda" else torch.zeros((self.n_slots, self.max_pages), dtype=torch.int32)
         self.page_table = torch.zeros((self.n_slots, self.max_pages), dtype=torch.int32, device=self.device)
@@ -93,10 +85,28 @@ class PagedState:
         self._free_slots = list(range(self.n_slots - 1, -1, -1))
         self.sequences: dict[str, Sequence] = {}
 
-    def record_state(self, i: int) -> "RecordState":
+    def _allocate(self, sp: StateSpec) -> RecordState:
+        def f32(*shape):
+            return torch.zeros(shape, dtype=torch.float32, device=self.device)
+
+        kv, rec, conv = sp.kv, sp.recurrent, sp.conv
+        return RecordState(
+            # K and V pages: [page][kv head][page_size][size] (None for a record without attention)
+            k_pages=f32(self.n_pages, kv[0], self.page_size, kv[1]) if kv else None,
+            v_pages=f32(self.n_pages, kv[0], self.page_size, kv[2]) if kv else None,
+            # the last taps - 1 normed inputs of the tap-mix sublayers: [slot][taps - 1][width]
+            tails=tuple(f32(self.n_slots, max(self.taps - 1, 1), self.width) for _ in range(sp.tap_tails)),
+            # recurrent matrix states [slot][head][value channel][key channel], short-convolution tails [slot][taps - 1][channels]
+            rec_state=f32(self.n_slots, rec[0], rec[1], rec[2]) if rec else None,
+            conv_tail=f32(self.n_slots, max(conv[0] - 1, 1), conv[1]) if conv else None,
+            # latent pages [page][page_size][size] share the page table with the K/V pages; per-slot numbers [slot][aux]
+            latent_pages=f32(self.n_pages, self.page_size, sp.latent) if sp.latent else None,
+            rec_aux=f32(self.n_slots, sp.aux) if sp.aux else None,
+            parts=tuple(self._allocate(q) for q in sp.parts))
+
+    def record_state(self, i: int) -> RecordState:
         """The buffers of layer record ``i`` (what its ``fill`` points the kernels at)."""
-        return RecordState(self.k_pages[i], self.v_pages[i], self.tails[i], self.rec_states[i], self.conv_tails[i],
-                           self.latent_pages[i], self.rec_aux[i])
+        return self.records[i]
 
     # ---- bookkeeping -----------------------------------------------------------------------------------------
     @property

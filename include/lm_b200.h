@@ -33,7 +33,7 @@
 extern "C" {
 #endif
 
-#define LM_B200_ABI_VERSION 4
+#define LM_B200_ABI_VERSION 5
 
 enum lm_b200_status { LM_B200_OK = 0, LM_B200_EINVAL = -1, LM_B200_ECUDA = -2, LM_B200_ENOMEM = -3, LM_B200_EUNSUPPORTED = -5 };
 
@@ -45,7 +45,11 @@ enum lm_b200_mixer_kind {
     LM_B200_MIXER_LATENT_ATTENTION = 5, /* queries through a normed latent, keys / values up-projected from one cached normed latent, sink, elementwise gate */
     LM_B200_MIXER_MLSTM = 6,            /* matrix memory with exponential input gate, running maximum and normaliser */
     LM_B200_MIXER_GATED_DELTA = 7,      /* gated delta rule with ONE decay per head and token, short convolutions, silu output gate */
-    LM_B200_MIXER_RETENTION = 8         /* linear attention with a fixed decay per head, rotary q / k, no softmax, no denominator */
+    LM_B200_MIXER_RETENTION = 8,        /* linear attention with a fixed decay per head, rotary q / k, no softmax, no denominator */
+    LM_B200_MIXER_ROTARY_ATTENTION = 9, /* grouped-query attention, per-head q / k norms, rotary positions, window, sink; values = a projection of their own or the raw keys */
+    LM_B200_MIXER_GATED_LINEAR = 10,    /* linear attention with a data-dependent decay per head and key channel (two-step projection), silu output gate */
+    LM_B200_MIXER_MAMBA2 = 11,          /* state-space duality: short convolution, step sizes, one decay per head, gate before a grouped norm */
+    LM_B200_MIXER_PAIR = 12             /* two mixers side by side on the same input: part_scale[0] mixer_0(h) + part_scale[1] mixer_1(h) */
 };
 enum lm_b200_ff_kind { LM_B200_FF_NONE = 0, LM_B200_FF_ROUTED_EXPERTS = 1, LM_B200_FF_DENSE = 2 };
 enum lm_b200_norm_kind { LM_B200_NORM_DYT = 0, LM_B200_NORM_LAYER = 1, LM_B200_NORM_RMS = 2 };
@@ -53,7 +57,8 @@ enum lm_b200_layer_form { LM_B200_FORM_SEQUENTIAL = 0, LM_B200_FORM_PARALLEL = 1
 /* XIELU: up, activation, down.  SILU_GLU / CLAMPED_GLU: gated units [gate | up] -> down with silu(g) u, or with
  * g' = min(g, limit), u' = clamp(u, -limit, limit): g' sigmoid(1.702 g') (u' + 1) */
 enum lm_b200_act_kind { LM_B200_ACT_SILU_GLU = 0, LM_B200_ACT_XIELU = 1, LM_B200_ACT_CLAMPED_GLU = 2,
-                        LM_B200_ACT_RELU2 = 3 /* dense, not gated: up, max(z, 0)^2, down */ };
+                        LM_B200_ACT_RELU2 = 3, /* dense, not gated: up, max(z, 0)^2, down */
+                        LM_B200_ACT_GELU_GLU = 4 /* gated unit with the tanh form of gelu: gelu(g) u */ };
 /* SIGMOID_INPUT: score sigmoid(z) multiplies the chosen expert's input.  SOFTMAX_TOP: the softmax over the chosen logits
  * alone weighs the experts' outputs */
 /* SOFTMAX_GROUPED: scores = softmax over ALL router outputs; the choice is made on score + correction, only inside the
@@ -167,6 +172,35 @@ typedef struct lm_b200_layer {
     float route_scale;             /* multiplies the normalised weights */
     const float *route_correction; /* [experts + identity_experts] added to the scores for the choice only; NULL: none */
     int32_t shared_gate;           /* != 0: w_router has one more row behind the router outputs, g; the shared unit's output is times sigmoid(g . h) */
+
+    /* ---- more mixers of the stream form, two mixers side by side, and the per-layer token input ----
+     * w_in of the mixers below, in this order:
+     *   ROTARY_ATTENTION  q (heads*dim) | k (kv_heads*dim) | v (kv_heads*dim, unless values_are_keys)
+     *   GATED_LINEAR      q (heads*dim) | k (heads*dim) | v (heads*vdim) | gate (heads*vdim, unless GATE_NONE) | a1 (rank_a)
+     *   MAMBA2            z (heads*vdim) | x (heads*vdim) | B (kv_heads*dim) | C (kv_heads*dim) | dt (heads)
+     * ROTARY_ATTENTION (vdim == dim): q_norm / k_norm [dim] per-head RMS norms, rot_dims / rot_freq as in TALK_ATTENTION, cosines and
+     * sines times rot_amp, `scale`, `window`, `sink`, k_pages / v_pages.
+     * GATED_LINEAR: S_t = diag(alpha_t) S_(t-1) + k_t v_t^T, o_t = S_t^T q_t with q times dim^-1/2 and alpha = sigmoid(w_a2 (a1 rows h)
+     * + dt_bias)^(1 / decay_tau), dt_bias [heads*dim] (NULL: none); o / rms(o) head_norm [vdim] gate.
+     * MAMBA2: `dim` is the state size and `kv_heads` the groups that share B and C; x, B, C pass conv_w [heads*vdim + 2 kv_heads*dim]
+     * [conv_taps] + conv_b and silu (conv_tail keeps the inputs); dt = softplus(dt + dt_bias [heads]); S_t = exp(-exp(a_log) dt) S_(t-1)
+     * + dt B x^T, y = S^T C + skip_d x; y silu(z) is RMS-normed in norm_groups equal parts, times head_norm [heads*vdim].
+     * rec_state of both: [slots][heads][vdim][dim].
+     * PAIR: part[0 / 1] are mixer descriptions (their sizes, weights and state; w_in and w_o are this record's, which stacks the
+     * rows of part 0, then those of part 1, each padded to its n_in, and has w_o [width][heads_0*vdim_0 + heads_1*vdim_1]). */
+    float rot_amp;                 /* multiplies cosine and sine (0 is read as 1) */
+    int32_t values_are_keys;       /* != 0: the value rows are the key projections before norm and rotation */
+    float decay_tau;
+    const float *conv_b;           /* channels of conv_w; NULL: none */
+    const float *skip_d;           /* [heads] */
+    int32_t norm_groups;
+    const struct lm_b200_layer *part[2]; /* copied at engine creation */
+    float part_scale[2];
+    /* After the feed-forward (one stream): e = the columns side_off .. side_off + side_dim of the token's row of side_table;
+     * y = w_side_proj (gelu(w_side_gate x) * e);  x <- x + y / rms(y) * side_norm. */
+    int32_t side_dim, side_ld, side_off; /* side_dim 0: none; side_table is bf16 [vocab][side_ld] */
+    const void *side_table, *w_side_gate, *w_side_proj; /* [side_dim][width], [width][side_dim] */
+    const float *side_norm;        /* [width] */
 } lm_b200_layer;
 
 typedef struct lm_b200_model {
@@ -212,12 +246,14 @@ int lm_b200_op_mixer(lm_b200_engine *e, int layer, const float *h, const int32_t
  * norms (q in place), the page append and the attention; out [M][heads * dim] */
 int lm_b200_op_attention(lm_b200_engine *e, int layer, float *qk, const int32_t *step, int M, int n_seq, float *out,
                          void *stream);
-/* a parallel record's mixer kernels alone on given stacked projections proj [M][n_in] (modified in place; state is
- * appended as in a step): out [M][heads * vdim], before the output projection */
+/* a parallel or stream record's mixer kernels alone on given stacked projections proj [M][n_in] (modified in place; state is
+ * appended as in a step): out [M][heads * vdim] (a pair: both parts' columns side by side), before the output projection */
 int lm_b200_op_mixer_kernels(lm_b200_engine *e, int layer, float *proj, const int32_t *step, int M, int n_seq, float *out,
                              void *stream);
 /* y = ff(h): router, expert groups, shared expert; the sum over a row's experts */
 int lm_b200_op_ff(lm_b200_engine *e, int layer, const float *h, int M, float *y, void *stream);
+/* out = x + rms(w_side_proj (gelu(w_side_gate x) * e)) * side_norm for the rows' tokens (a stream record's token input) */
+int lm_b200_op_token_input(lm_b200_engine *e, int layer, const float *x, const int32_t *step, int M, float *out, void *stream);
 /* Y[M][N] = A[M][K] . W[N][K]^T */
 int lm_b200_op_linear(const float *A, const void *W_bf16, float *Y, int M, int N, int K, void *stream);
 /* the same on the tensor cores: A is rounded to bf16 into a_bf16 [M][K] first.  K a multiple of 8, N of 4, else
