@@ -23,7 +23,8 @@ path); `value` is the sum over ranks divided by the slowest rank's time (weak sc
 sizes of a real model: prefill and decode throughput through `CausalLM`, and its GEMM / attention kernels beside Dia's
 at equal size (one JSON line, metric `lm_layer_throughput`).  `--lm --lm-design luketar` measures the Luketar design
 beside Kupelix and Pubopel at equal width and its mixers beside Kupelix's.  `--lm --lm-design fipadra` measures the Fipadra
-design beside Luketar at equal width and its mixers beside their likes in Luketar and Kupelix.  `--lm --lm-design kupelix` measures the Kupelix design
+design beside Luketar at equal width and its mixers beside their likes in Luketar and Kupelix.  `--lm --lm-design loduzen`
+measures the Loduzen design beside Fipadra with dense units.  `--lm --lm-design kupelix` measures the Kupelix design
 instead: its prefill and decode throughput beside Pubopel's at equal width, heads and vocabulary, its attention kernel
 beside Pubopel's on the same causal workload, and its recurrence kernels against the bytes and state updates they must move.
 """
@@ -1081,6 +1082,130 @@ def run_lm_fipadra(args) -> None:
                       "gpu_launches": launch_count() - launches0, "clocks": clocks, "lm": out}))
 
 
+# ---- --lm --lm-design loduzen: the Loduzen design beside Fipadra at equal width, its mixers beside their likes -----------------
+LODUZEN_SIZES = {
+    # the widths, head counts, window and vocabularies of FIPADRA_SIZES; linear attention with as many heads of the same size beside
+    # the softmax attention, a state-space mixer of twice the width with 128 states and 8 / 4 groups, a gated unit with the
+    # parameter count of Fipadra's squared-relu unit, and a token input of 256 / 128 channels per layer
+    "w2048": dict(width=2048, kinds=["parallel", "mamba2", "parallel", "mamba2"], heads=16, kv_heads=4, dim=128, window=1024,
+                  lin_heads=16, lin_dim=128, lin_vdim=128, ssm_heads=64, ssm_vdim=64, ssm_state=128, ssm_groups=8, norm_groups=8,
+                  taps=4, ff=4096, side=256, rot_dims=64, vocab=32768,
+                  yarn=dict(factor=4.0, original=4096, fast=32.0, slow=1.0)),
+    "w1024": dict(width=1024, kinds=["parallel", "mamba2", "parallel", "mamba2"], heads=8, kv_heads=2, dim=128, window=1024,
+                  lin_heads=8, lin_dim=128, lin_vdim=128, ssm_heads=32, ssm_vdim=64, ssm_state=128, ssm_groups=4, norm_groups=4,
+                  taps=4, ff=1024, side=128, rot_dims=64, vocab=16384,
+                  yarn=dict(factor=4.0, original=4096, fast=32.0, slow=1.0)),
+}
+
+
+def run_lm_loduzen(args) -> None:
+    import torch
+    from dia_tts_prune_b200 import synthetic as SY
+    from dia_tts_prune_b200.lm_config import FipadraConfig, KupelixConfig, LoduzenConfig, PubopelConfig
+    from dia_tts_prune_b200.lm_engine import launch_count
+    from dia_tts_prune_b200.lm_model import CausalLM
+
+    if not torch.cuda.is_available():
+        raise SystemExit("bench.py needs a CUDA device: the product path has no CPU fallback")
+    dev = torch.device("cuda", 0)
+    torch.cuda.set_device(dev)
+    try:
+        with open(os.path.join(REPO, "MEASURED_PEAKS.json")) as f:
+            pk = json.load(f)
+        hbm, tf, src = float(pk["hbm_gbs"]), float(pk["bf16_tflops"]), "measured"
+    except Exception:
+        hbm, tf, src = 6650.0, 1590.0, "fallback"
+    flush = torch.zeros(160 << 20, dtype=torch.uint8, device=dev)             # > the 126 MB L2
+    W, K = max(args.warmup, 3), max(args.steps, 3)
+    sampler = ClockSampler(0)
+    sampler.start()
+    launches0 = launch_count()
+    out = {}
+    T, ctx, R = args.lm_prompt, args.lm_context, args.lm_rows
+    for name in (args.lm_sizes.split(",") if args.lm_sizes else LODUZEN_SIZES):
+        sz, fsz, ksz, psz = LODUZEN_SIZES[name], FIPADRA_SIZES[name], KUPELIX_SIZES[name], LM_SIZES[name]
+        D, H, G, d, V, win, kinds = sz["width"], sz["heads"], sz["kv_heads"], sz["dim"], sz["vocab"], sz["window"], sz["kinds"]
+        toks = torch.randint(0, V, (T,), generator=torch.Generator().manual_seed(7)).tolist()
+        cap = max(T, 8 * (ctx + 32 * (K + 2))) + 64
+        res = {"config": dict(sz)}
+        kw = dict(dtype="bfloat16", device=dev, max_tokens=cap, max_sequences=8, page_size=64, max_rows=R)
+        cfg = SY.loduzen_config(**sz)
+        model = CausalLM(LoduzenConfig.model_validate(cfg), SY.loduzen_weights(cfg, WEIGHT_SEED, dev), **kw)
+        res["loduzen"] = _lm_prefill_decode(model, toks, T, ctx, W, K, flush)
+        # products per token: stacked input projections and output projection of a mixer, feed-forward, token input
+        lh, ld, lv, sh, sv, sn, sg = (sz[k] for k in ("lin_heads", "lin_dim", "lin_vdim", "ssm_heads", "ssm_vdim", "ssm_state", "ssm_groups"))
+        cols = {"parallel": D * (H * d + G * d + 2 * lh * ld + 2 * lh * lv + 16) + 16 * lh * ld + D * (H * d + lh * lv),
+                "mamba2": D * (2 * sh * sv + 2 * sg * sn + sh) + D * sh * sv}
+        rest = 3 * D * sz["ff"] + 2 * D * sz["side"]
+        keys = sum(min(t + 1, win) for t in range(T))             # (query, key) pairs of a windowed prompt
+        mixer_flops = {"parallel": 4.0 * H * d * keys + 4.0 * T * lh * ld * lv, "mamba2": 4.0 * T * sh * sv * sn}
+        flops = 2.0 * T * sum(cols[k] + rest for k in kinds) + sum(mixer_flops[k] for k in kinds) + 2.0 * D * V
+        w_bytes = 2.0 * (sum(cols[k] + rest for k in kinds) + D * V)
+        state = {"parallel": 8.0 * min(ctx, win) * G * d + 8.0 * lh * ld * lv, "mamba2": 8.0 * sh * sv * sn}
+        state_bytes = sum(state[k] for k in kinds) + 8.0 * len(kinds) * D
+        pf, b1 = res["loduzen"]["prefill"], res["loduzen"]["decode_b1"]
+        pf.update(model_tflops=flops / pf["ms"] / 1e9, frac_of_bf16_peak=flops / pf["ms"] / 1e9 / tf)
+        b1.update(algorithmic_bytes=w_bytes + state_bytes, gb_per_s=(w_bytes + state_bytes) / b1["ms_per_step"] / 1e6,
+                  frac_of_hbm_peak=(w_bytes + state_bytes) / b1["ms_per_step"] / 1e6 / hbm)
+        model.engine.close()
+        del model
+        torch.cuda.empty_cache()
+        fcfg = _fipadra_config({**fsz, "kinds": ["latent_attention", "retention", "latent_attention", "delta"], "experts": 0})
+        model = CausalLM(FipadraConfig.model_validate(fcfg), SY.fipadra_weights(fcfg, WEIGHT_SEED, dev), **kw)
+        res["fipadra_dense"] = _lm_prefill_decode(model, toks, T, ctx, W, K, flush)
+        model.engine.close()
+        del model
+        torch.cuda.empty_cache()
+
+        # -- mixers alone (projections, kernels, output projection; no feed-forward): one-layer models of either design
+        def timed(m1, n_seq, rows_each, start):
+            h = torch.randn(n_seq * min(rows_each, R), D, device=dev)
+            seqs = [m1.state.open(f"s{i}") for i in range(n_seq)]
+            for sq in seqs:
+                m1.state.reserve(sq, start + rows_each)
+            def run():
+                for r0 in range(0, rows_each, R):
+                    n = min(R, rows_each - r0)
+                    m1.engine.op_mixer(0, h[:n_seq * n], [(sq, n, start + r0) for sq in seqs])
+            ms = _event_ms(run, 2, K, flush)
+            for i in range(n_seq):
+                m1.state.close(f"s{i}")
+            return ms
+
+        kw1 = dict(dtype="bfloat16", device=dev, max_tokens=8 * T + 64, max_sequences=8, page_size=64, max_rows=R)
+        mixers = {}
+        # a pair does the work of Pubopel's attention (same heads and window) and of Kupelix's hgrn2 (same recurrent state); the
+        # state-space mixer's like is Fipadra's retention with as many heads as give the same recurrent state
+        c_pub = SY.pubopel_config(**{**psz, "layers": 1, "vocab": 256, "experts": 1, "top": 1, "expert_ff": 8, "shared_ff": 0,
+                                     "window": win, "keep_first": 0})
+        c_hgr = SY.kupelix_config(**{**ksz, "kinds": ["hgrn2"], "heads": lh, "dim": ld, "vdim": lv, "vocab": 256, "ff": 8})
+        c_ret = _fipadra_config({**fsz, "kinds": ["retention"], "heads": sh * sv * sn // (128 * 128), "vocab": 256, "ff": 0, "experts": 0})
+        twins = {"parallel": [("pubopel_attention", CausalLM, PubopelConfig, c_pub, SY.pubopel_weights),
+                              ("kupelix_hgrn2", CausalLM, KupelixConfig, c_hgr, SY.kupelix_weights)],
+                 "mamba2": [("fipadra_retention", CausalLM, FipadraConfig, c_ret, SY.fipadra_weights)]}
+        for kind, likes in twins.items():
+            c1 = SY.loduzen_config(**{**sz, "kinds": [kind], "vocab": 256, "ff": 0, "side": 0})
+            models = [("loduzen", CausalLM(LoduzenConfig.model_validate(c1), SY.loduzen_weights(c1, 3, dev), **kw1))]
+            models += [(label, cls(conf.model_validate(c), weights(c, 3, dev), **kw1)) for label, cls, conf, c, weights in likes]
+            ent = {}
+            for label, (n_seq, rows_each, start) in {"prefill_1x%d" % T: (1, T, 0), "prefill_8x%d" % (T // 8): (8, T // 8, 0),
+                                                     "decode_b8": (8, 1, ctx)}.items():
+                ent[label] = {f"{who}_ms": timed(m1, n_seq, rows_each, start) for who, m1 in models}
+            mixers[kind] = ent
+            for _, m1 in models:
+                m1.engine.close()
+            del models
+            torch.cuda.empty_cache()
+        res["mixers"] = mixers
+        out[name] = res
+    clocks = sampler.stop()
+    print(json.dumps({"metric": "lm_layer_throughput", "design": "loduzen", "impl": "ours", "n_gpus": 1, "steps": K, "warmup": W,
+                      "dtype": "bf16", "data": "synthetic (random weights, random token ids)",
+                      "peaks": {"hbm_gbs": hbm, "bf16_tflops": tf, "source": src},
+                      "timing": "CUDA events, median; a 160 MB buffer is rewritten between timed iterations (L2 flush)",
+                      "gpu_launches": launch_count() - launches0, "clocks": clocks, "lm": out}))
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -1103,17 +1228,18 @@ def main():
     ap.add_argument("--lm", action="store_true",
                     help="instead of the headline workload: prefill / decode throughput of the decoder-only language-model path "
                          "(Pubopel, random weights) at layer sizes of a real model, beside Dia's kernels at equal size")
-    ap.add_argument("--lm-design", default="pubopel", choices=["pubopel", "kupelix", "luketar", "fipadra"],
+    ap.add_argument("--lm-design", default="pubopel", choices=["pubopel", "kupelix", "luketar", "fipadra", "loduzen"],
                     help="--lm: the design that is measured (kupelix: beside Pubopel at equal width, and its kernels beside Pubopel's; "
                          "luketar: beside Kupelix and Pubopel at equal width, and its mixers beside Kupelix's; fipadra: beside Luketar at equal "
-                         "width, and its mixers beside their likes in Luketar and Kupelix)")
+                         "width, and its mixers beside their likes in Luketar and Kupelix; loduzen: beside Fipadra with dense units at equal "
+                         "width, and its mixers beside their likes in Pubopel, Kupelix and Fipadra)")
     ap.add_argument("--lm-sizes", default="", help="--lm: comma-separated subset of " + ",".join(LM_SIZES))
     ap.add_argument("--lm-prompt", type=int, default=4096, help="--lm: prompt tokens of the prefill measurement")
     ap.add_argument("--lm-rows", type=int, default=4096, help="--lm: most rows of one engine step (longer prompts run in portions)")
     ap.add_argument("--lm-context", type=int, default=1024, help="--lm: tokens each sequence holds before the decode measurement")
     args = ap.parse_args()
     if args.lm:
-        {"kupelix": run_lm_kupelix, "luketar": run_lm_luketar, "fipadra": run_lm_fipadra}.get(args.lm_design, run_lm)(args)
+        {"kupelix": run_lm_kupelix, "luketar": run_lm_luketar, "fipadra": run_lm_fipadra, "loduzen": run_lm_loduzen}.get(args.lm_design, run_lm)(args)
         return
     if args.impl == "reference":
         run_reference(args)

@@ -12,9 +12,8 @@
 //   side_act_kernel           token input: gelu(z) times the token's slice of the second embedding table
 //   side_gate_rows_kernel     the same with the product in front, for a handful of rows
 //
-// The recurrences themselves are column_scan_kernel (write rule) and scalar_gate_scan_kernel (shared q / k heads and a skip
-// term) of lm_mixers.cu, the convolution's tail is kept by conv_tail_kernel, and the token input's own norm and residual add
-// are options of streams_step_kernel.
+// The recurrences themselves run in lm_scan.cu, the convolution's tail is kept by conv_tail_kernel of lm_mixers.cu, and the
+// token input's own norm and residual add are options of streams_step_kernel.
 #include <algorithm>
 
 #include <cuda_bf16.h>

@@ -19,20 +19,13 @@
 //                             their two-step projections
 //   conv_tail_kernel          keeps the last taps-1 projected inputs of every scheduled sequence
 //   gate_prep_kernel          silu(q), the bounded forget gate and biases of the gate-tied recurrence, in place
-//   column_scan_kernel        the recurrences with a decay per key channel, one value column of one head per 8 lanes:
-//                             S <- a S;  [u = beta (v - S^T k)];  S <- S + w u;  o = S^T q, state carried per sequence (the
-//                             write w is 1 - a, or k with or without the delta)
-//   scalar_gate_scan_kernel   the same column layout for a recurrence with one decay and one write strength per token and
-//                             head, and a normaliser carried as one more value column
-//                             (or a fixed decay per head, write strength 1, no normaliser: retention; or q and k shared by
-//                             groups of heads and a skip term: the state-space mixer)
 //   head_norm_gate_kernel     per-head RMS norm of the read-out (x weight, x gate or its sigmoid / silu), fp32 in place and
 //                             the bf16 operand
 //   xielu_rows_kernel         the dense feed-forward's activation (xIELU or squared relu) on its slice of the stacked
 //                             projections
 // talk_attention_kernel also serves attention over cached latent rows (one key/value head whose value rows are the leading
-// channels of its key rows) and takes a window; delta_prep_kernel and column_scan_kernel also serve the delta rule with ONE
-// decay per head; layernorm_rows_kernel also computes the RMS norm.
+// channels of its key rows) and takes a window; delta_prep_kernel also serves the delta rule with ONE decay per head;
+// layernorm_rows_kernel also computes the RMS norm.  The recurrences run in lm_scan.cu.
 #include <algorithm>
 
 #include <cuda_bf16.h>
@@ -689,281 +682,6 @@ __global__ void gate_prep_kernel(float* __restrict__ proj, int ld, int q_off, in
         for (int c = threadIdx.x; c < n_v; c += blockDim.x) row[v_off + c] += bias[v_off + c];
 }
 
-// The recurrence.  Per head a state S [dim][vdim]; every value column c of S evolves on its own:
-//   S[:, c] <- a_t * S[:, c];   then by RULE (kScanTied / kScanDelta / kScanWrite of lm_internal.h)
-//     tied:  S[:, c] += (1 - a_t) v_t[c]
-//     delta: u = beta_t (v_t[c] - S[:, c] . k_t), S[:, c] += k_t u
-//     write: S[:, c] += k_t v_t[c]
-//   o_t[c] = S[:, c] . (q_mul q_t)
-// The decays may stand in a buffer of their own (a_in, row stride lda).
-// A column lives in the registers of 8 lanes (lane part holds rows part, part + 8, ...; its dot products are summed in
-// four interleaved partial sums, then across the 8 lanes); a CTA of 4 warps carries 16 columns of one head of one
-// scheduled sequence through the sequence's rows in order, 16 tokens staged in shared memory at a time while the next 16
-// are on their way into registers.  The state is read when the sequence's first row is not position 0, and written
-// back at the end: state[slot][h][c][dim].
-constexpr int kScanThreads = 128, kScanCols = 16, kScanTT = 16;
-
-template <int RP, int RULE>
-__global__ void __launch_bounds__(kScanThreads)
-column_scan_kernel(const float* __restrict__ in, int ld, int q_off, int k_off, const float* __restrict__ a_in, int lda, int v_off,
-                   int beta_off, int H, int G, int dim, int vdim, float* __restrict__ state, const int* __restrict__ seq_slot,
-                   const int* __restrict__ seq_row0, const int* __restrict__ seq_count, const int* __restrict__ row_pos,
-                   float* __restrict__ o, int ldo, int head_decay, float q_mul) {
-    extern __shared__ float sh[];
-    constexpr bool DELTA = RULE == kScanDelta, KEYS = RULE != kScanTied;
-    constexpr int DS = 8 * RP;                                // staged row length (channels beyond dim hold zeros)
-    float* sq = sh;                                           // [TT][DS]
-    float* sa = sq + kScanTT * DS;                            // [TT][DS]
-    float* sk = sa + kScanTT * DS;                            // [TT][DS] (KEYS)
-    float* sv = sk + (KEYS ? kScanTT * DS : 0);               // [TT][16]
-    float* sb = sv + kScanTT * kScanCols;                     // [TT] (DELTA)
-    pdl_release();
-    pdl_wait();
-    const int s = blockIdx.x, h = blockIdx.y, col0 = blockIdx.z * kScanCols;
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, part = lane & 7, cl = warp * 4 + (lane >> 3);
-    const int col = col0 + cl, g = h / (H / G);
-    const int slot = seq_slot[s], row0 = seq_row0[s], n = seq_count[s], start = row_pos[row0];
-    const bool col_ok = col < vdim;
-    float* st = state + (((size_t)slot * H + h) * vdim + (col_ok ? col : 0)) * dim;
-    float S[RP];
-#pragma unroll
-    for (int r = 0; r < RP; ++r) {
-        const int d = part + 8 * r;
-        S[r] = (start > 0 && col_ok && d < dim) ? st[d] : 0.f;
-    }
-    // Staging: a chunk of 16 tokens is 16 * DS = 128 * RP elements per input; thread tid owns elements tid + 128 i, the
-    // same (token in chunk, channel) for every chunk.
-    int src[RP];                                              // (token in chunk) * ld + channel, -1: a channel beyond dim
-#pragma unroll
-    for (int i = 0; i < RP; ++i) {
-        const int idx = tid + kScanThreads * i, t = idx / DS, d = idx - t * DS;
-        src[i] = d < dim ? t * ld + d : -1;
-    }
-    const int qh = KEYS ? g : h;
-    float rq[RP], ra[RP], rk[KEYS ? RP : 1], rv[2], rb = 0.f;
-    auto fetch = [&](int t0) {
-        const int nt = min(kScanTT, n - t0);
-        const float* base = in + (size_t)(row0 + t0) * ld;
-        const float* abase = a_in + (size_t)(row0 + t0) * lda;
-#pragma unroll
-        for (int i = 0; i < RP; ++i) {
-            const int t = (tid + kScanThreads * i) / DS, d = (tid + kScanThreads * i) - t * DS;
-            const bool ok = src[i] >= 0 && t < nt;
-            rq[i] = ok ? base[src[i] + q_off + qh * dim] * q_mul : 0.f;
-            // head_decay: column h of the decay row holds the one decay of all of the head's key channels
-            ra[i] = !ok ? 0.f : abase[t * lda + (head_decay ? h : h * dim + d)];
-            if (KEYS) rk[i] = ok ? base[src[i] + k_off + g * dim] : 0.f;
-        }
-#pragma unroll
-        for (int i = 0; i < 2; ++i) {
-            const int idx = tid + kScanThreads * i, t = idx / kScanCols, c = idx - t * kScanCols;
-            rv[i] = (t < nt && col0 + c < vdim) ? base[(size_t)t * ld + v_off + h * vdim + col0 + c] : 0.f;
-        }
-        if (DELTA && tid < nt) rb = base[(size_t)tid * ld + beta_off + h];
-    };
-    fetch(0);
-    for (int t0 = 0; t0 < n; t0 += kScanTT) {
-        const int nt = min(kScanTT, n - t0);
-        __syncthreads();                                      // the previous chunk is consumed
-#pragma unroll
-        for (int i = 0; i < RP; ++i) {
-            const int idx = tid + kScanThreads * i;
-            sq[idx] = rq[i];
-            sa[idx] = ra[i];
-            if (KEYS) sk[idx] = rk[i];
-        }
-        sv[tid] = rv[0];
-        sv[tid + kScanThreads] = rv[1];
-        if (DELTA && tid < kScanTT) sb[tid] = rb;
-        __syncthreads();
-        if (t0 + kScanTT < n) fetch(t0 + kScanTT);            // in flight during the recurrence below
-#pragma unroll 4
-        for (int t = 0; t < nt; ++t) {
-            const float* q = sq + t * DS + part;
-            const float* a = sa + t * DS + part;
-            const float v = sv[t * kScanCols + cl];
-            float d0 = 0.f, d1 = 0.f, d2 = 0.f, d3 = 0.f;
-            if (DELTA) {
-                const float* k = sk + t * DS + part;
-                float e0 = 0.f, e1 = 0.f, e2 = 0.f, e3 = 0.f;
-#pragma unroll
-                for (int r = 0; r < RP; r += 4) {
-                    S[r] *= a[8 * r];
-                    S[r + 1] *= a[8 * r + 8];
-                    S[r + 2] *= a[8 * r + 16];
-                    S[r + 3] *= a[8 * r + 24];
-                    e0 = fmaf(S[r], k[8 * r], e0);
-                    e1 = fmaf(S[r + 1], k[8 * r + 8], e1);
-                    e2 = fmaf(S[r + 2], k[8 * r + 16], e2);
-                    e3 = fmaf(S[r + 3], k[8 * r + 24], e3);
-                }
-                float dk = (e0 + e1) + (e2 + e3);
-                dk += __shfl_xor_sync(0xffffffffu, dk, 1);
-                dk += __shfl_xor_sync(0xffffffffu, dk, 2);
-                dk += __shfl_xor_sync(0xffffffffu, dk, 4);
-                const float u = sb[t] * (v - dk);
-#pragma unroll
-                for (int r = 0; r < RP; r += 4) {
-                    S[r] = fmaf(k[8 * r], u, S[r]);
-                    S[r + 1] = fmaf(k[8 * r + 8], u, S[r + 1]);
-                    S[r + 2] = fmaf(k[8 * r + 16], u, S[r + 2]);
-                    S[r + 3] = fmaf(k[8 * r + 24], u, S[r + 3]);
-                    d0 = fmaf(S[r], q[8 * r], d0);
-                    d1 = fmaf(S[r + 1], q[8 * r + 8], d1);
-                    d2 = fmaf(S[r + 2], q[8 * r + 16], d2);
-                    d3 = fmaf(S[r + 3], q[8 * r + 24], d3);
-                }
-            } else if (KEYS) {
-                const float* k = sk + t * DS + part;
-#pragma unroll
-                for (int r = 0; r < RP; r += 4) {
-                    S[r] = fmaf(a[8 * r], S[r], k[8 * r] * v);
-                    S[r + 1] = fmaf(a[8 * r + 8], S[r + 1], k[8 * r + 8] * v);
-                    S[r + 2] = fmaf(a[8 * r + 16], S[r + 2], k[8 * r + 16] * v);
-                    S[r + 3] = fmaf(a[8 * r + 24], S[r + 3], k[8 * r + 24] * v);
-                    d0 = fmaf(S[r], q[8 * r], d0);
-                    d1 = fmaf(S[r + 1], q[8 * r + 8], d1);
-                    d2 = fmaf(S[r + 2], q[8 * r + 16], d2);
-                    d3 = fmaf(S[r + 3], q[8 * r + 24], d3);
-                }
-            } else {
-#pragma unroll
-                for (int r = 0; r < RP; r += 4) {
-                    const float a0 = a[8 * r], a1 = a[8 * r + 8], a2 = a[8 * r + 16], a3 = a[8 * r + 24];
-                    S[r] = fmaf(a0, S[r], (1.0f - a0) * v);
-                    S[r + 1] = fmaf(a1, S[r + 1], (1.0f - a1) * v);
-                    S[r + 2] = fmaf(a2, S[r + 2], (1.0f - a2) * v);
-                    S[r + 3] = fmaf(a3, S[r + 3], (1.0f - a3) * v);
-                    d0 = fmaf(S[r], q[8 * r], d0);
-                    d1 = fmaf(S[r + 1], q[8 * r + 8], d1);
-                    d2 = fmaf(S[r + 2], q[8 * r + 16], d2);
-                    d3 = fmaf(S[r + 3], q[8 * r + 24], d3);
-                }
-            }
-            float dot = (d0 + d1) + (d2 + d3);
-            dot += __shfl_xor_sync(0xffffffffu, dot, 1);
-            dot += __shfl_xor_sync(0xffffffffu, dot, 2);
-            dot += __shfl_xor_sync(0xffffffffu, dot, 4);
-            if (part == 0 && col_ok) o[(size_t)(row0 + t0 + t) * ldo + h * vdim + col] = dot;
-        }
-    }
-    if (col_ok) {
-#pragma unroll
-        for (int r = 0; r < RP; ++r) {
-            const int d = part + 8 * r;
-            if (d < dim) st[d] = S[r];
-        }
-    }
-}
-
-// The same column layout for a recurrence with scalar gates per (token, head):  S[:, c] <- a_t S[:, c] + (b_t k_t) v_t[c],
-// o_t[c] = S[:, c] . q_t.  Column vdim of every head is the normaliser: its value is the constant 1, so it carries
-// n <- a n + b k and reads out n . q.  State and read-out have vdim + 1 columns per head: state[slot][h][c][dim].
-// q and k have G heads (each serves H / G of the H); skip [H]: skip[h] v_t[c] joins the read-out.
-template <int RP>
-__global__ void __launch_bounds__(kScanThreads)
-scalar_gate_scan_kernel(const float* __restrict__ in, int ld, int q_off, int k_off, int a_off, int v_off, int b_off, int H, int G,
-                        int dim, int vdim, float* __restrict__ state, const int* __restrict__ seq_slot, const int* __restrict__ seq_row0,
-                        const int* __restrict__ seq_count, const int* __restrict__ row_pos, float* __restrict__ o, int ldo,
-                        const float* __restrict__ fixed_decay, int normaliser, const float* __restrict__ skip) {
-    extern __shared__ float sh[];
-    constexpr int DS = 8 * RP;
-    float* sq = sh;                                           // [TT][DS]
-    float* sk = sq + kScanTT * DS;                            // [TT][DS]
-    float* sv = sk + kScanTT * DS;                            // [TT][16]
-    float* sa = sv + kScanTT * kScanCols;                     // [TT]
-    float* sb = sa + kScanTT;                                 // [TT]
-    pdl_release();
-    pdl_wait();
-    // fixed_decay: a = fixed_decay[h] and b = 1 for every token (no gate columns are read); normaliser 0: vdim columns
-    const int s = blockIdx.x, h = blockIdx.y, col0 = blockIdx.z * kScanCols, vcols = vdim + (normaliser ? 1 : 0);
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, part = lane & 7, cl = warp * 4 + (lane >> 3);
-    const int col = col0 + cl, g = h / (H / G);
-    const int slot = seq_slot[s], row0 = seq_row0[s], n = seq_count[s], start = row_pos[row0];
-    const bool col_ok = col < vcols;
-    const float sd = skip ? skip[h] : 0.f;
-    const float a_fix = fixed_decay ? fixed_decay[h] : 0.f;
-    float* st = state + (((size_t)slot * H + h) * vcols + (col_ok ? col : 0)) * dim;
-    float S[RP];
-#pragma unroll
-    for (int r = 0; r < RP; ++r) {
-        const int d = part + 8 * r;
-        S[r] = (start > 0 && col_ok && d < dim) ? st[d] : 0.f;
-    }
-    int src[RP];
-#pragma unroll
-    for (int i = 0; i < RP; ++i) {
-        const int idx = tid + kScanThreads * i, t = idx / DS, d = idx - t * DS;
-        src[i] = d < dim ? t * ld + d : -1;
-    }
-    float rq[RP], rk[RP], rv[2], ra = 0.f, rb = 0.f;
-    auto fetch = [&](int t0) {
-        const int nt = min(kScanTT, n - t0);
-        const float* base = in + (size_t)(row0 + t0) * ld;
-#pragma unroll
-        for (int i = 0; i < RP; ++i) {
-            const bool ok = src[i] >= 0 && (tid + kScanThreads * i) / DS < nt;
-            rq[i] = ok ? base[src[i] + q_off + g * dim] : 0.f;
-            rk[i] = ok ? base[src[i] + k_off + g * dim] : 0.f;
-        }
-#pragma unroll
-        for (int i = 0; i < 2; ++i) {
-            const int idx = tid + kScanThreads * i, t = idx / kScanCols, c = col0 + (idx - t * kScanCols);
-            rv[i] = t < nt ? (c < vdim ? base[(size_t)t * ld + v_off + h * vdim + c] : ((c == vdim && normaliser) ? 1.f : 0.f)) : 0.f;
-        }
-        if (tid < nt) {
-            ra = fixed_decay ? a_fix : base[(size_t)tid * ld + a_off + h];
-            rb = fixed_decay ? 1.f : base[(size_t)tid * ld + b_off + h];
-        }
-    };
-    fetch(0);
-    for (int t0 = 0; t0 < n; t0 += kScanTT) {
-        const int nt = min(kScanTT, n - t0);
-        __syncthreads();
-#pragma unroll
-        for (int i = 0; i < RP; ++i) {
-            const int idx = tid + kScanThreads * i;
-            sq[idx] = rq[i];
-            sk[idx] = rk[i];
-        }
-        sv[tid] = rv[0];
-        sv[tid + kScanThreads] = rv[1];
-        if (tid < kScanTT) { sa[tid] = ra; sb[tid] = rb; }
-        __syncthreads();
-        if (t0 + kScanTT < n) fetch(t0 + kScanTT);
-#pragma unroll 4
-        for (int t = 0; t < nt; ++t) {
-            const float* q = sq + t * DS + part;
-            const float* k = sk + t * DS + part;
-            const float a = sa[t], v = sv[t * kScanCols + cl], u = sb[t] * v;
-            float d0 = 0.f, d1 = 0.f, d2 = 0.f, d3 = 0.f;
-#pragma unroll
-            for (int r = 0; r < RP; r += 4) {
-                S[r] = fmaf(a, S[r], k[8 * r] * u);
-                S[r + 1] = fmaf(a, S[r + 1], k[8 * r + 8] * u);
-                S[r + 2] = fmaf(a, S[r + 2], k[8 * r + 16] * u);
-                S[r + 3] = fmaf(a, S[r + 3], k[8 * r + 24] * u);
-                d0 = fmaf(S[r], q[8 * r], d0);
-                d1 = fmaf(S[r + 1], q[8 * r + 8], d1);
-                d2 = fmaf(S[r + 2], q[8 * r + 16], d2);
-                d3 = fmaf(S[r + 3], q[8 * r + 24], d3);
-            }
-            float dot = (d0 + d1) + (d2 + d3);
-            dot += __shfl_xor_sync(0xffffffffu, dot, 1);
-            dot += __shfl_xor_sync(0xffffffffu, dot, 2);
-            dot += __shfl_xor_sync(0xffffffffu, dot, 4);
-            if (part == 0 && col_ok) o[(size_t)(row0 + t0 + t) * ldo + h * vcols + col] = fmaf(sd, v, dot);
-        }
-    }
-    if (col_ok) {
-#pragma unroll
-        for (int r = 0; r < RP; ++r) {
-            const int d = part + 8 * r;
-            if (d < dim) st[d] = S[r];
-        }
-    }
-}
-
 // o[r][h] <- o[r][h] / sqrt(mean(o[r][h]^2) + eps) * w [* gate[r][h]] in place (one warp per row and head), and its bf16 copy
 // gate_act: 0 the gate columns are used as they are (already activated), 1 sigmoid, 2 silu of them; w may be absent
 __global__ void head_norm_gate_kernel(float* __restrict__ o, int ldo, __nv_bfloat16* __restrict__ o_b, const float* __restrict__ w,
@@ -1110,73 +828,9 @@ cudaError_t launch_conv_tail(const float* proj, int ld, int C, int taps, float* 
                       sm.count);
 }
 
-template <int RP, int RULE>
-static cudaError_t launch_scan_inst(const float* in, int ld, const ScanInputs& si, int H, int G, int dim, int vdim, float* state,
-                                    const SeqMeta& sm, const RowMeta& rm, int n_seq, float* o, int ldo, cudaStream_t st,
-                                    bool head_decay, bool early, const float* decay, int ldd, float q_mul) {
-    const size_t smem = (size_t)((RULE != kScanTied ? 3 : 2) * kScanTT * 8 * RP + kScanTT * kScanCols + kScanTT) * 4;
-    if (smem > 48 * 1024) {
-        cudaError_t e = cudaFuncSetAttribute(column_scan_kernel<RP, RULE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-        if (e != cudaSuccess) return e;
-    }
-    return launch_pdl_if(early, column_scan_kernel<RP, RULE>, dim3(n_seq, H, (vdim + kScanCols - 1) / kScanCols), dim3(kScanThreads), smem, st,
-                      in, ld, si.q_off, si.k_off, decay ? decay : in + si.a_off, decay ? ldd : ld, si.v_off, si.beta_off, H, G, dim, vdim,
-                      state, sm.slot, sm.row0, sm.count, rm.pos, o, ldo, head_decay ? 1 : 0, q_mul);
-}
-
 cudaError_t launch_gate_prep(float* proj, int ld, int q_off, int f_off, int v_off, const float* bias, const float* lower, int n_qf,
                              int n_v, int M, cudaStream_t st) {
     return launch_pdl(gate_prep_kernel, dim3(M), dim3(256), 0, st, proj, ld, q_off, f_off, v_off, bias, lower, n_qf, n_v);
-}
-
-// kScanTied: its inputs prepared by launch_gate_prep; kScanDelta reads k and beta; kScanWrite reads k
-cudaError_t launch_column_scan(const float* in, int ld, const ScanInputs& si, int rule, int H, int G, int dim, int vdim,
-                               float* state, const SeqMeta& sm, const RowMeta& rm, int n_seq, float* o, int ldo,
-                               cudaStream_t st, bool head_decay, bool early, const float* decay, int ldd, float q_mul) {
-    if (dim > 256 || H % G || H > 65535) return cudaErrorNotSupported;
-#define SCAN_RULE(RP, RULE) \
-    return launch_scan_inst<RP, RULE>(in, ld, si, H, G, dim, vdim, state, sm, rm, n_seq, o, ldo, st, head_decay, early, decay, ldd, q_mul)
-#define SCAN_CASE(RP)                            \
-    switch (rule) {                              \
-        case kScanTied: SCAN_RULE(RP, kScanTied);   \
-        case kScanDelta: SCAN_RULE(RP, kScanDelta); \
-        case kScanWrite: SCAN_RULE(RP, kScanWrite); \
-        default: return cudaErrorInvalidValue;   \
-    }
-    if (dim <= 32) SCAN_CASE(4);
-    if (dim <= 64) SCAN_CASE(8);
-    if (dim <= 128) SCAN_CASE(16);
-    SCAN_CASE(32);
-#undef SCAN_CASE
-#undef SCAN_RULE
-}
-
-template <int RP>
-static cudaError_t launch_scalar_scan_inst(const float* in, int ld, const ScanInputs& si, int H, int G, int dim, int vdim, float* state,
-                                           const SeqMeta& sm, const RowMeta& rm, int n_seq, float* o, int ldo, cudaStream_t st,
-                                           const float* fixed_decay, bool normaliser, bool early, const float* skip) {
-    const size_t smem = (size_t)(2 * kScanTT * 8 * RP + kScanTT * kScanCols + 2 * kScanTT) * 4;
-    if (smem > 48 * 1024) {
-        cudaError_t e = cudaFuncSetAttribute(scalar_gate_scan_kernel<RP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-        if (e != cudaSuccess) return e;
-    }
-    return launch_pdl_if(early, scalar_gate_scan_kernel<RP>, dim3(n_seq, H, (vdim + (normaliser ? 1 : 0) + kScanCols - 1) / kScanCols),
-                      dim3(kScanThreads), smem, st, in, ld, si.q_off, si.k_off, si.a_off, si.v_off, si.beta_off, H, G, dim, vdim, state,
-                      sm.slot, sm.row0, sm.count, rm.pos, o, ldo, fixed_decay, normaliser ? 1 : 0, skip);
-}
-
-cudaError_t launch_scalar_gate_scan(const float* in, int ld, const ScanInputs& si, int H, int dim, int vdim, float* state,
-                                    const SeqMeta& sm, const RowMeta& rm, int n_seq, float* o, int ldo, cudaStream_t st,
-                                    const float* fixed_decay, bool normaliser, bool early, int G, const float* skip) {
-    if (G <= 0) G = H;
-    if (dim > 256 || H > 65535 || H % G) return cudaErrorNotSupported;
-#define SCALAR_CASE(RP) \
-    return launch_scalar_scan_inst<RP>(in, ld, si, H, G, dim, vdim, state, sm, rm, n_seq, o, ldo, st, fixed_decay, normaliser, early, skip)
-    if (dim <= 32) SCALAR_CASE(4);
-    if (dim <= 64) SCALAR_CASE(8);
-    if (dim <= 128) SCALAR_CASE(16);
-    SCALAR_CASE(32);
-#undef SCALAR_CASE
 }
 
 cudaError_t launch_head_norm_gate(float* o, int ldo, void* o_bf16, const float* w, const float* gate, int ldg, int H, int vdim,

@@ -28,7 +28,7 @@
 //   mlstm_finish_kernel       read-out / (max(|n . q|, floor) + 1e-6), per-head RMS norm, weight, sigmoid gate
 //
 // The attention itself is talk_attention_kernel of lm_mixers.cu with ONE key/value head whose key and value pages are
-// the same latent pages (keys = values = c, head size = latent size), and the recurrence is scalar_gate_scan_kernel.
+// the same latent pages (keys = values = c, head size = latent size), and the recurrence runs in lm_scan.cu.
 #include <algorithm>
 
 #include <cuda_bf16.h>

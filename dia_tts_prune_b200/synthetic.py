@@ -381,3 +381,76 @@ def fipadra_weights(cfg: dict, seed: int = 1234, device="cpu") -> dict:
                     unit(p + "mlp.shared.", f["shared"]["ff"])
                     w[p + "mlp.shared.sg"] = mat(1, D)
     return w
+
+
+def loduzen_config(width: int, kinds: list[str], heads: int, dim: int, vocab: int, kv_heads: int = 0, window: int = 0,
+                   lin_heads: int = 0, lin_dim: int = 0, lin_vdim: int = 0, ssm_heads: int = 0, ssm_vdim: int = 0, ssm_state: int = 0,
+                   ssm_groups: int = 1, norm_groups: int = 1, taps: int = 4, ff: int = 0, side: int = 0, rot_dims: int = 0,
+                   yarn: dict | None = None) -> dict:
+    """A Loduzen ``config.json`` as a dictionary: one layer per entry of ``kinds`` (``parallel`` / ``mamba2``), each with a dense
+    unit of ``ff`` hidden units (none when 0) and a token input of ``side`` channels (none when 0).  ``yarn``: rotary scaling."""
+    layers = []
+    for kind in kinds:
+        if kind == "parallel":
+            rot = {"base": 10000.0, "dims": rot_dims or dim}
+            if yarn:
+                rot["scaling"] = dict(yarn)
+            left = {"heads": heads, "kv_heads": kv_heads or heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "rot": rot}
+            if window:
+                left["mask"] = {"size": window}
+            m = {"left": left, "left_scale": 0.8, "right_scale": 0.6,
+                 "right": {"heads": lin_heads or heads, "dim": lin_dim or dim, "vdim": lin_vdim or dim, "tau": 16.0}}
+        else:
+            m = {"heads": ssm_heads, "vdim": ssm_vdim, "state": ssm_state, "groups": ssm_groups, "conv": taps, "norm_groups": norm_groups}
+        layers.append({"type": kind, "mixer": m, "mlp": {"kind": "dense", "ff": ff} if ff else None})
+    cfg = {"architecture": "Loduzen", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "layers": layers}
+    if side:
+        cfg["token_side"] = {"dim": side}
+    return cfg
+
+
+def loduzen_weights(cfg: dict, seed: int = 1234, device="cpu", rank: int = 16) -> dict:
+    """Random bfloat16 tensors under the checkpoint's names: matrices ~ N(0, 1 / fan_in), norm weights near one, decays mostly
+    close to one; ``rank``: inner size of the two-step decay projections."""
+    import torch
+    g = torch.Generator(device=device).manual_seed(seed)
+    D, V = cfg["width"], cfg["vocab"]
+
+    def mat(n, k, gain=1.0):
+        return (torch.randn((n, k), generator=g, device=device) * (gain * k ** -0.5)).to(torch.bfloat16)
+
+    def vec(n, mean, spread):
+        return (mean + spread * torch.randn((n,), generator=g, device=device)).to(torch.bfloat16)
+
+    w = {"embed": torch.randn((V, D), generator=g, device=device).to(torch.bfloat16), "final.norm": vec(D, 1.0, 0.05)}
+    side = (cfg.get("token_side") or {}).get("dim", 0)
+    if side:
+        w["side.embed"] = torch.randn((V, side * len(cfg["layers"])), generator=g, device=device).to(torch.bfloat16)
+    for i, lc in enumerate(cfg["layers"]):
+        p, m = f"l{i}.", lc["mixer"]
+        w[p + "norm1"] = vec(D, 1.0, 0.05)
+        if lc["type"] == "parallel":
+            a, q = m["left"], p + "mix.left."
+            H, G, d = a["heads"], a["kv_heads"], a["dim"]
+            w[q + "q"], w[q + "k"], w[q + "o"] = mat(H * d, D), mat(G * d, D), mat(D, H * d)
+            w[q + "q.norm"], w[q + "k.norm"] = vec(d, 1.0, 0.05), vec(d, 1.0, 0.05)
+            r, q = m["right"], p + "mix.right."
+            H, d, dv = r["heads"], r["dim"], r["vdim"]
+            w[q + "q"], w[q + "k"], w[q + "v"], w[q + "g"] = mat(H * d, D), mat(H * d, D), mat(H * dv, D), mat(H * dv, D)
+            w[q + "a1"], w[q + "a2"], w[q + "a2.b"] = mat(rank, D), mat(H * d, rank), vec(H * d, 1.0, 0.5)
+            w[q + "norm"], w[q + "o"] = vec(dv, 1.0, 0.05), mat(D, H * dv)
+        else:
+            H, N, G, dv, taps = m["heads"], m["state"], m["groups"], m["vdim"], m["conv"]
+            q, C = p + "mix.", H * dv + 2 * G * N
+            w[q + "in"] = mat(H * dv + C + H, D)
+            w[q + "conv"] = (torch.randn((C, taps), generator=g, device=device) * taps ** -0.5).to(torch.bfloat16)
+            w[q + "conv.b"] = vec(C, 0.0, 0.1)
+            w[q + "dt_bias"], w[q + "A_log"], w[q + "D"] = vec(H, -3.0, 1.0), vec(H, 0.5, 0.5), vec(H, 1.0, 0.1)
+            w[q + "norm"], w[q + "o"] = vec(H * dv, 1.0, 0.05), mat(D, H * dv)
+        f = lc.get("mlp")
+        if f:
+            w[p + "norm2"] = vec(D, 1.0, 0.05)
+            w[p + "mlp.gate"], w[p + "mlp.up"], w[p + "mlp.down"] = mat(f["ff"], D), mat(f["ff"], D), mat(D, f["ff"])
+        if side:
+            w[p + "side.gate"], w[p + "side.proj"], w[p + "side.norm"] = mat(side, D), mat(D, side), vec(D, 0.3, 0.05)
+    return w

@@ -183,7 +183,7 @@ def test_matrix_memory_with_other_state_shapes(heads, dim, vdim):
 @pytest.mark.parametrize("make", [small_config, odd_config, plain_config])
 def test_whole_prompt_logits_and_layer_streams(make):
     cfg = make()
-    model, w = build(cfg, 11)
+    model, w = build(cfg, 14)
     toks = tokens(cfg, 61, 2)
     ref, streams = O.forward(cfg, w, toks, keep_layers=True)
     got, got_streams = whole(model, "a", toks, keep_layers=True)
