@@ -8,11 +8,11 @@
 //   o_t[c] = q_mul (S[:, c] . q_t) [+ skip_h v_t[c]]
 // A normaliser is one more value column whose value is the constant 1.  q and k may be shared by groups of heads.
 //
-// A warp carries 8 columns of one head of one scheduled sequence: lane = 8 g + part holds columns 2 g, 2 g + 1, rows
-// 32 j + 4 part + (0 .. 3), so the vectors of a token are read from shared memory in 16-byte pieces that serve both columns, and
-// the arithmetic is packed fp32x2.  Sixteen tokens are staged at a time (asynchronous copies, two buffers).  A dot product is
-// summed in four interleaved partial sums per lane and then across the 8 lanes (distances 4, 2, 1); the read-outs of four
-// tokens and two columns share one such exchange.  The order of operations of a column depends on nothing but the column.
+// A group of P = 8, 16 or 32 lanes carries two columns of one head of one scheduled sequence; lane `part` of it holds the rows
+// 4 P j + 4 part + (0 .. 3) of both, at most 8 per column, so that even one sequence gives enough warps.  The vectors of a token are
+// read from shared memory in 16-byte pieces that serve both columns, and the arithmetic is packed fp32x2.  Sixteen tokens are
+// staged at a time (asynchronous copies, two buffers).  A dot product is summed in four interleaved partial sums per lane and
+// then across the P lanes (distances P / 2 .. 1); the read-outs of four tokens and two columns share one such exchange.  The order of operations of a column depends on nothing but the column.
 // The state is read when the sequence's first row is not position 0 and written back at the end: state[slot][h][c][dim].
 #include <algorithm>
 
@@ -27,7 +27,10 @@ namespace lm {
 namespace {
 
 constexpr int kTokens = 16;                                   // tokens per staged chunk
-constexpr int kMaxWarps = 4;
+constexpr int kMaxWarps = 8;
+
+// lanes that share a pair of columns
+template <int DP> constexpr int kParts = DP > 64 ? DP / 8 : 8;
 
 using f2 = unsigned long long;                                // two packed fp32
 __device__ __forceinline__ f2 pack2(float lo, float hi) {
@@ -81,13 +84,13 @@ __global__ void __launch_bounds__(kMaxWarps * 32, 1)
 state_scan_kernel(const ScanArgs p) {
     extern __shared__ __align__(16) float sh[];
     constexpr bool KEYS = RULE != kScanTied;
-    constexpr int J = DP / 32, VECS = 1 + (KEYS ? 1 : 0) + (VA ? 1 : 0);
-    const int VC = 8 * (blockDim.x >> 5);                     // value columns of the CTA
+    constexpr int P = kParts<DP>, CW = 64 / P, J = DP / (4 * P), VECS = 1 + (KEYS ? 1 : 0) + (VA ? 1 : 0);
+    const int VC = CW * (blockDim.x >> 5);                    // value columns of the CTA
     const int stage = kTokens * (VECS * DP + VC + 2);
     pdl_release();
     pdl_wait();
     const int s = blockIdx.x, h = blockIdx.y, col0 = blockIdx.z * VC, g = h / (p.H / p.G);
-    const int tid = threadIdx.x, lane = tid & 31, part = lane & 7, cb = (tid >> 5) * 8 + (lane >> 3) * 2;   // first column in the CTA
+    const int tid = threadIdx.x, lane = tid & 31, part = lane & (P - 1), cb = (tid >> 5) * CW + lane / P * 2;   // first column in the CTA
     const int slot = p.seq_slot[s], row0 = p.seq_row0[s], n = p.seq_count[s], start = p.row_pos[row0];
     const float a_fix = p.fixed_decay ? p.fixed_decay[h] : 0.f, sd = p.skip ? p.skip[h] : 0.f;
     const bool vec_state = p.dim % 4 == 0;
@@ -101,7 +104,7 @@ state_scan_kernel(const ScanArgs p) {
         st[c] = p.state + (((size_t)slot * p.H + h) * p.vcols + (col < p.vcols ? col : 0)) * p.dim;
 #pragma unroll
         for (int j = 0; j < J; ++j) {
-            const int d = 32 * j + 4 * part;
+            const int d = 4 * P * j + 4 * part;
             float4 t = make_float4(0.f, 0.f, 0.f, 0.f);
             if (live && d < p.dim) {
                 if (vec_state) t = *reinterpret_cast<const float4*>(st[c] + d);
@@ -192,9 +195,9 @@ state_scan_kernel(const ScanArgs p) {
                 ulonglong2 kk[J];
 #pragma unroll
                 for (int j = 0; j < J; ++j) {
-                    kk[j] = k[8 * j];
+                    kk[j] = k[P * j];
                     ulonglong2 aa;
-                    if (VA) aa = a[8 * j];
+                    if (VA) aa = a[P * j];
                     else aa.x = aa.y = as;
 #pragma unroll
                     for (int c = 0; c < 2; ++c) {
@@ -206,7 +209,7 @@ state_scan_kernel(const ScanArgs p) {
                 }
                 float e0 = sum2(e[0][0], e[0][1]), e1 = sum2(e[1][0], e[1][1]);
 #pragma unroll
-                for (int o = 4; o > 0; o >>= 1) {
+                for (int o = P / 2; o > 0; o >>= 1) {
                     e0 += __shfl_xor_sync(0xffffffffu, e0, o);
                     e1 += __shfl_xor_sync(0xffffffffu, e1, o);
                 }
@@ -214,7 +217,7 @@ state_scan_kernel(const ScanArgs p) {
                 const f2 u[2] = {pack2(u0, u0), pack2(u1, u1)};
 #pragma unroll
                 for (int j = 0; j < J; ++j) {
-                    const ulonglong2 qq = q[8 * j];
+                    const ulonglong2 qq = q[P * j];
 #pragma unroll
                     for (int c = 0; c < 2; ++c) {
                         S[c][2 * j] = fma2(kk[j].x, u[c], S[c][2 * j]);
@@ -229,11 +232,11 @@ state_scan_kernel(const ScanArgs p) {
                 const f2 one = pack2(1.f, 1.f), minus = pack2(-1.f, -1.f);
 #pragma unroll
                 for (int j = 0; j < J; ++j) {
-                    const ulonglong2 qq = q[8 * j];
+                    const ulonglong2 qq = q[P * j];
                     ulonglong2 aa, kk;
-                    if (VA) aa = a[8 * j];
+                    if (VA) aa = a[P * j];
                     else aa.x = aa.y = as;
-                    if (KEYS) kk = k[8 * j];
+                    if (KEYS) kk = k[P * j];
                     else { kk.x = fma2(aa.x, minus, one); kk.y = fma2(aa.y, minus, one); }     // tied: 1 - a
 #pragma unroll
                     for (int c = 0; c < 2; ++c) {
@@ -247,37 +250,40 @@ state_scan_kernel(const ScanArgs p) {
             d0 = sum2(acc[0][0], acc[0][1]);
             d1 = sum2(acc[1][0], acc[1][1]);
         };
-        // lane `part` of a column pair stores token t + (part >> 1), column part & 1
-        auto store = [&](int t, float dot) {
-            const int col = col0 + cb + (part & 1);
-            if (col < p.vcols)
-                p.o[(size_t)(row0 + t0 + t) * p.ldo + h * p.vcols + col] = fmaf(sd, sv[t * VC + cb + (part & 1)], dot * p.q_mul);
+        auto store = [&](int t, int c, float dot) {
+            const int col = col0 + cb + c;
+            if (col < p.vcols) p.o[(size_t)(row0 + t0 + t) * p.ldo + h * p.vcols + col] = fmaf(sd, sv[t * VC + cb + c], dot * p.q_mul);
         };
         int t = 0;
         for (; t + 4 <= nt; t += 4) {
             float d[8];
 #pragma unroll
             for (int i = 0; i < 4; ++i) token(t + i, d[2 * i], d[2 * i + 1]);
+            // eight values over P lanes: at the first three distances a lane keeps the half of the values that its bit names and
+            // gives the other away, then the last value is summed over the lanes that hold it
 #pragma unroll
-            for (int o = 4; o > 0; o >>= 1) {                 // d[i], i < 2 o: keep the half that this lane's bit names, give the other away
+            for (int m = 4, o = P / 2; m > 0; m >>= 1, o >>= 1) {
                 const bool up = part & o;
 #pragma unroll
-                for (int i = 0; i < o; ++i) {
-                    const float give = up ? d[i] : d[i + o], keep = up ? d[i + o] : d[i];
+                for (int i = 0; i < m; ++i) {
+                    const float give = up ? d[i] : d[i + m], keep = up ? d[i + m] : d[i];
                     d[i] = keep + __shfl_xor_sync(0xffffffffu, give, o);
                 }
             }
-            store(t + (part >> 1), d[0]);
+#pragma unroll
+            for (int o = P / 16; o > 0; o >>= 1) d[0] += __shfl_xor_sync(0xffffffffu, d[0], o);
+            const int at = part / (P / 8);                    // the value that this lane holds: token at >> 1, column at & 1
+            if (part % (P / 8) == 0) store(t + (at >> 1), at & 1, d[0]);
         }
         for (; t < nt; ++t) {
             float d0, d1;
             token(t, d0, d1);
 #pragma unroll
-            for (int o = 4; o > 0; o >>= 1) {
+            for (int o = P / 2; o > 0; o >>= 1) {
                 d0 += __shfl_xor_sync(0xffffffffu, d0, o);
                 d1 += __shfl_xor_sync(0xffffffffu, d1, o);
             }
-            if (part < 2) store(t, part ? d1 : d0);
+            if (part < 2) store(t, part, part ? d1 : d0);
         }
         __syncthreads();                                      // this buffer is consumed
     }
@@ -286,7 +292,7 @@ state_scan_kernel(const ScanArgs p) {
         if (col0 + cb + c >= p.vcols) continue;
 #pragma unroll
         for (int j = 0; j < J; ++j) {
-            const int d = 32 * j + 4 * part;
+            const int d = 4 * P * j + 4 * part;
             if (d >= p.dim) continue;
             float4 t;
             unpack2(S[c][2 * j], t.x, t.y);
@@ -303,9 +309,15 @@ state_scan_kernel(const ScanArgs p) {
 }
 
 template <int DP, int RULE, bool VA>
-cudaError_t launch_inst(const ScanArgs& p, int n_seq, int warps, bool early, cudaStream_t st) {
+cudaError_t launch_inst(const ScanArgs& p, int n_seq, bool early, cudaStream_t st) {
+    // warps of a CTA share the staged vectors: as many as leave a CTA for every SM
+    constexpr int CW = 64 / kParts<DP>;
+    const long long total = (long long)n_seq * p.H * ((p.vcols + CW - 1) / CW);
+    int warps = 1;
+    while (warps < kMaxWarps && total >= 120 * 2 * warps && CW * warps < p.vcols) warps *= 2;
+    if (warps == kMaxWarps && total < 16 * 148) warps /= 2;
     constexpr int VECS = 1 + (RULE != kScanTied ? 1 : 0) + (VA ? 1 : 0);
-    const int VC = 8 * warps;
+    const int VC = 64 / kParts<DP> * warps;
     const size_t smem = (size_t)2 * kTokens * (VECS * DP + VC + 2) * 4;
     static size_t allowed[64] = {};
     if (smem > 48 * 1024) {
@@ -324,14 +336,10 @@ cudaError_t launch_inst(const ScanArgs& p, int n_seq, int warps, bool early, cud
 template <int RULE, bool VA>
 cudaError_t launch_scan(const ScanArgs& p, int n_seq, bool early, cudaStream_t st) {
     if (p.dim > 256 || p.H % p.G || p.H > 65535) return cudaErrorNotSupported;
-    // warps of a CTA share the staged vectors: several where there are enough columns to fill the device anyway
-    const long long total = (long long)n_seq * p.H * ((p.vcols + 7) / 8);
-    int warps = total >= 8 * 148 ? kMaxWarps : total > 148 ? 2 : 1;
-    while (warps > 1 && 8 * (warps / 2) >= p.vcols) warps /= 2;
-    if (p.dim <= 32) return launch_inst<32, RULE, VA>(p, n_seq, warps, early, st);
-    if (p.dim <= 64) return launch_inst<64, RULE, VA>(p, n_seq, warps, early, st);
-    if (p.dim <= 128) return launch_inst<128, RULE, VA>(p, n_seq, warps, early, st);
-    return launch_inst<256, RULE, VA>(p, n_seq, warps, early, st);
+    if (p.dim <= 32) return launch_inst<32, RULE, VA>(p, n_seq, early, st);
+    if (p.dim <= 64) return launch_inst<64, RULE, VA>(p, n_seq, early, st);
+    if (p.dim <= 128) return launch_inst<128, RULE, VA>(p, n_seq, early, st);
+    return launch_inst<256, RULE, VA>(p, n_seq, early, st);
 }
 
 bool aligned16(const float* base, int ld, int off, int dim) {
