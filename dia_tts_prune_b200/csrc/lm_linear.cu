@@ -98,6 +98,25 @@ ssm_prep_kernel(const float* __restrict__ proj, int ld, int x_off, int C, int H,
     }
     const float* w = cw + (size_t)c * taps;
     const float b = cb ? cb[c] : 0.f;
+    // a full tile inside one sequence whose earlier inputs all stand in this step: every input is loaded once, all of them in
+    // flight together (the sums run in the same order as below; taps that are not there weigh 0)
+    constexpr int KT = 4;
+    if (taps <= KT && r1 - r0 == kSsmRows && row_slot[r1 - 1] == row_slot[r0] && row_pos[r1 - 1] - row_pos[r0] == kSsmRows - 1 &&
+        row_pos[r0] - row_start[r0] >= KT - 1) {
+        float u[kSsmRows + KT - 1], wt[KT];
+#pragma unroll
+        for (int i = 0; i < kSsmRows + KT - 1; ++i) u[i] = proj[(size_t)(r0 - (KT - 1) + i) * ld + x_off + c];
+#pragma unroll
+        for (int o = 0; o < KT; ++o) wt[o] = o < taps ? w[taps - 1 - o] : 0.f;
+#pragma unroll
+        for (int i = 0; i < kSsmRows; ++i) {
+            float acc = b;
+#pragma unroll
+            for (int o = 0; o < KT; ++o) acc = fmaf(wt[o], u[i + KT - 1 - o], acc);
+            rec[(size_t)(r0 + i) * ldr + c] = siluf_(acc);
+        }
+        return;
+    }
     for (int r = r0; r < r1; ++r) {
         const int slot = row_slot[r], pos = row_pos[r], start = row_start[r];
         float acc = b;
