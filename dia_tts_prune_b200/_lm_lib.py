@@ -16,11 +16,11 @@ MIXER_GATED_DELTA, MIXER_RETENTION, MIXER_ROTARY_ATTENTION, MIXER_GATED_LINEAR, 
 FF_NONE, FF_ROUTED_EXPERTS, FF_DENSE = 0, 1, 2
 NORM_DYT, NORM_LAYER, NORM_RMS = 0, 1, 2
 FORM_SEQUENTIAL, FORM_PARALLEL, FORM_STREAMS = 0, 1, 2
-ACT_SILU_GLU, ACT_XIELU, ACT_CLAMPED_GLU, ACT_RELU2, ACT_GELU_GLU = 0, 1, 2, 3, 4
+ACT_SILU_GLU, ACT_XIELU, ACT_CLAMPED_GLU, ACT_RELU2, ACT_GELU_GLU, ACT_GELU = 0, 1, 2, 3, 4, 5
 ROUTER_SIGMOID_INPUT, ROUTER_SOFTMAX_TOP, ROUTER_SOFTMAX_GROUPED = 0, 1, 2
-GATE_SIGMOID, GATE_NONE, GATE_SILU = 0, 1, 2
+GATE_SIGMOID, GATE_NONE, GATE_SILU, GATE_SIGMOID_HEAD = 0, 1, 2, 3
 ROT_INTERLEAVED, ROT_HALF = 0, 1
-ABI_VERSION = 5
+ABI_VERSION = 6
 PRECISION_FP32, PRECISION_BF16 = 0, 1
 E_OK, E_INVAL, E_CUDA, E_NOMEM, E_UNSUPPORTED = 0, -1, -2, -3, -5
 
@@ -55,14 +55,17 @@ class Layer(C.Structure):
                 # more mixers, two mixers side by side, the token input
                 ("rot_amp", _f), ("values_are_keys", _i), ("decay_tau", _f), ("conv_b", _vp), ("skip_d", _vp), ("norm_groups", _i),
                 ("part", _vp * 2), ("part_scale", _f * 2), ("side_dim", _i), ("side_ld", _i), ("side_off", _i), ("side_table", _vp),
-                ("w_side_gate", _vp), ("w_side_proj", _vp), ("side_norm", _vp)]
+                ("w_side_gate", _vp), ("w_side_proj", _vp), ("side_norm", _vp),
+                # chunks
+                ("chunk", _i)]
 
 
 class Model(C.Structure):
     _fields_ = [("n_layer", _i), ("width", _i), ("vocab", _i), ("taps", _i), ("page_size", _i), ("max_pages", _i),
                 ("n_slots", _i), ("max_rows", _i), ("eps", _f), ("precision", _i), ("embed", _vp), ("head", _vp),
                 ("final_norm", Norm), ("page_table", _vp), ("step_graphs", _i), ("logit_scale", _f), ("embed_scale", _f),
-                ("embed_norm", _vp)]
+                ("embed_norm", _vp), ("bigram", _vp), ("bigram_buckets", _i), ("bigram_mul_prev", _i), ("bigram_mul_cur", _i),
+                ("token_pages", _vp)]
 
 
 _ci = C.c_int

@@ -23,7 +23,8 @@
 // The same kernel serves callers whose activations are bf16 already (terms = 1: one MMA per k-step, the operand is read
 // as it is), row tiles that belong to different weight matrices (expert groups: the group of a tile's first row picks
 // the matrix, a device-side row count skips the unused tiles), a contraction length that is not a multiple of the
-// k-block (the TMA fills the tail of both operands with zeros) and a DynamicTanh in front of the residual add.
+// k-block (the TMA fills the tail of both operands with zeros), a DynamicTanh in front of the residual add, and a gelu whose
+// result leaves as the bf16 operand of the product that follows.
 #include <algorithm>
 
 #include <cuda.h>
@@ -80,6 +81,13 @@ __device__ __forceinline__ void umma_commit(uint64_t* bar) {
 }
 
 }  // namespace
+
+// gelu in its tanh form, as z sigmoid(2 u) with u = sqrt(2 / pi) (z + 0.044715 z^3): 0.5 (1 + tanh u) = sigmoid(2 u).  Fast
+// exponential and division: the result is rounded to bf16.
+__device__ __forceinline__ float gelu_to_bf16_range(float z) {
+    const float u2 = 1.5957691216057308f * fmaf(0.044715f * z * z, z, z);
+    return __fdividef(z, 1.0f + __expf(fminf(-u2, 80.f)));
+}
 
 // x = hi + lo + lo2 per element, three stacked bf16 matrices [3][M][K]
 __global__ void split3_rows_kernel(const float* __restrict__ x, __nv_bfloat16* __restrict__ xs, long long n) {
@@ -147,7 +155,8 @@ __global__ void transpose_to_bf16_kernel(const void* __restrict__ w, int src_bf1
 __global__ void __launch_bounds__(kGemmThreads, 1)
 dia_gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b,
                         float* y, const float* residual, int M, int N, int K, int terms, const float* dyt_w,
-                        const float* dyt_b, float dyt_alpha, const int* row_group, int group_rows, const int* n_rows) {
+                        const float* dyt_b, float dyt_alpha, __nv_bfloat16* y_bf16, const int* row_group, int group_rows,
+                        const int* n_rows) {
     extern __shared__ unsigned char smem_raw[];
     unsigned char* smem = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
     unsigned char* a_ring = smem;
@@ -275,6 +284,23 @@ dia_gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_
                     const int c0 = n0 + cb * 32;
                     float* dst = y + (size_t)row * N + c0;
                     const float* res = residual ? residual + (size_t)row * N + c0 : nullptr;
+                    if (y_bf16) {                               // the activation of an up product, as the next product's operand
+                        __nv_bfloat16* dstb = y_bf16 + (size_t)row * N + c0;
+#pragma unroll
+                        for (int i = 0; i < 8; ++i) {
+                            if (c0 + 4 * i + 4 <= N) {          // (N a multiple of 4: 8-byte stores)
+                                uint2 p;
+                                __nv_bfloat162 lo = __floats2bfloat162_rn(gelu_to_bf16_range(__uint_as_float(v[4 * i])),
+                                                                          gelu_to_bf16_range(__uint_as_float(v[4 * i + 1])));
+                                __nv_bfloat162 hi = __floats2bfloat162_rn(gelu_to_bf16_range(__uint_as_float(v[4 * i + 2])),
+                                                                          gelu_to_bf16_range(__uint_as_float(v[4 * i + 3])));
+                                p.x = *reinterpret_cast<uint32_t*>(&lo);
+                                p.y = *reinterpret_cast<uint32_t*>(&hi);
+                                *reinterpret_cast<uint2*>(dstb + 4 * i) = p;
+                            }
+                        }
+                        continue;
+                    }
 #pragma unroll
                     for (int i = 0; i < 8; ++i) {
                         if (c0 + 4 * i + 4 <= N) {
@@ -373,7 +399,8 @@ cudaError_t launch_gemm_tcgen05_bf16(const void* a_bf16, int terms, const void* 
     const int sms = (dev < 0 || dev >= 64) ? n_sm[0] : n_sm[dev];
     const int n_tiles = ((N + BN - 1) / BN) * ((M + BM - 1) / BM);
     dia_gemm_tcgen05_kernel<<<std::min(n_tiles, sms), kGemmThreads, kGemmSmem, st>>>(
-        ma, mb, y, ep.residual, M, N, K, terms, ep.dyt_w, ep.dyt_b, ep.dyt_alpha, groups ? groups->row_group : nullptr,
+        ma, mb, y, ep.residual, M, N, K, terms, ep.dyt_w, ep.dyt_b, ep.dyt_alpha,
+        reinterpret_cast<__nv_bfloat16*>(ep.y_bf16), groups ? groups->row_group : nullptr,
         groups ? groups->group_rows : 0, groups ? groups->n_rows : nullptr);
     return cudaGetLastError();
 }
@@ -388,7 +415,7 @@ cudaError_t launch_gemm_tcgen05(const float* x, const float* norm_w, float eps, 
     else
         split3_rows_kernel<<<(int)std::min<long long>((n + 255) / 256, 148 * 16), 256, 0, st>>>(
             x, reinterpret_cast<__nv_bfloat16*>(workspace), n);
-    const GemmEpilogue ep{residual, nullptr, nullptr, 0.f};
+    const GemmEpilogue ep{residual, nullptr, nullptr, 0.f, nullptr};
     return launch_gemm_tcgen05_bf16(workspace, kTerms, wt, N, y, M, N, K, ep, nullptr, st);
 }
 

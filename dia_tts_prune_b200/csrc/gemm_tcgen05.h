@@ -2,7 +2,8 @@
 //
 //   Y[M][N] (fp32) = residual + f(A[M][K] (bf16) . Wt[N][K]^T (bf16)),  fp32 accumulation in tensor memory
 //
-// f is the identity or a DynamicTanh per output column.  With row groups, the rows of A are sorted by group, every
+// f is the identity, a DynamicTanh per output column, or an activation whose result is kept as the bf16 operand of the next
+// product (Yb[M][N] instead of Y).  With row groups, the rows of A are sorted by group, every
 // group starts on a multiple of kGemmRowTile rows, and group g multiplies rows [g * group_rows, g * group_rows + N)
 // of Wt.
 #pragma once
@@ -18,6 +19,7 @@ struct GemmEpilogue {
     const float* dyt_w;                      // [N]: f(a) = tanh(dyt_alpha a) dyt_w + dyt_b; null: f(a) = a
     const float* dyt_b;
     float dyt_alpha;
+    void* y_bf16;                            // [M][N] bf16: gelu(result), the tanh form, goes here and nothing to y; null: y
 };
 
 struct GemmGroups {

@@ -54,6 +54,20 @@ constexpr int kGluSilu = 0, kGluClamped = 1, kGluGelu = 2;
 __device__ __forceinline__ float gelu_tanhf_(float z) {
     return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * fmaf(0.044715f * z * z, z, z)));
 }
+// activation of a unit that is not gated (kAct* of lm_internal.h).  xIELU: z > 0: ap z^2 + z / 2;  z <= 0: an (e^z - 1 - z) + z / 2
+__device__ __forceinline__ float unit_act(int act, float z, float ap, float an) {
+    switch (act) {
+        case 1: return z > 0.f ? fmaf(ap * z, z, 0.5f * z) : fmaf(an, expm1f(z) - z, 0.5f * z);
+        case 2: return fmaxf(z, 0.f) * fmaxf(z, 0.f);
+        case 3: return gelu_tanhf_(z);
+        default: return z;
+    }
+}
+// the first key a query at position i sees behind the kept first ones: its window's, and its chunk's where they are bounded
+__device__ __forceinline__ int first_key(int i, int window, int chunk) {
+    const int w = window > 0 ? max(0, i - window + 1) : 0;
+    return chunk > 0 ? max(w, i - i % chunk) : w;
+}
 __device__ __forceinline__ float glu_act(int kind, float g, float u, float limit) {
     if (kind == kGluClamped) {
         g = fminf(g, limit);

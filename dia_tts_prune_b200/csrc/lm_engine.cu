@@ -25,7 +25,7 @@
 //   proj = h W_in^T                             linear: every projection of the mixer and the feed-forward's up rows
 //   mixer on proj -> out[:, :mixer columns]     talk_prep + talk_attention | gate_prep + column_scan + head_norm_gate |
 //                                               linear x 2 (decay, gate) + delta_prep + conv_tail + column_scan + head_norm_gate
-//   out[:, mixer columns:] = act(proj up rows)  xielu_rows
+//   out[:, mixer columns:] = act(proj up rows)  unit_act_rows
 //   x += out W_out^T                            linear with the residual add (W_out = [W_o | W_down])
 //
 // A record of the stream form (s residual streams with hyper-connection weights, layer norm without bias, a latent
@@ -59,6 +59,10 @@
 //                     (column_scan with the write rule); per-head RMS norm x silu(gate) (head_norm_gate)
 //   state-space mixer: convolution, silu, step sizes, decays (ssm_prep); tails (conv_tail); the recurrence with B / C shared by
 //                     groups of heads and the skip term (scalar_gate_scan); gate, then the grouped norm (gate_norm)
+// A record without input norms (one stream) reads the stream itself, and its sublayers' OUTPUTS may be RMS-normed: the
+// streams_step that writes an output norms it first and leaves only the bf16 operand of the next product.  The embedding may
+// add the row of a pair table picked by the previous token and this one (streams_embed; the tokens are kept in pages).  The
+// rotary attention may see only the keys of its own chunk, and gates may be one number per head.
 // A record may end with a token input:  x += rms(W_proj (gelu(W_gate x) * e)) w with e the token's slice of a second table
 //   (one streams_step writes what is pending, linear | side_gate_rows, side_act, linear; the next streams_step norms and adds)
 // A PARALLEL stream record lets both sublayers read the streams before either writes: the mixer's output waits in a buffer
@@ -175,7 +179,7 @@ bool tensor_path(const lm_b200_engine* e, int M, int N, int K) {
     return e->m.precision == LM_B200_PRECISION_BF16 && M >= kTensorRowsMin && dia::gemm_tcgen05_shape_ok(M, N, K);
 }
 
-const dia::GemmEpilogue kPlain{nullptr, nullptr, nullptr, 0.f};
+const dia::GemmEpilogue kPlain{nullptr, nullptr, nullptr, 0.f, nullptr};
 
 struct StepView {
     const int *token, *want;
@@ -270,7 +274,7 @@ StreamCols stream_cols(const lm_b200_layer& l) {
         c.q = at; at += H * d; c.k = at; at += H * d; c.v = at; at += H * dv; c.ig = at; at += H; c.fg = at; at += H;
     }
     c.gate = -1;
-    if (l.mixer_gate != LM_B200_GATE_NONE) { c.gate = at; at += H * dv; }
+    if (l.mixer_gate != LM_B200_GATE_NONE) { c.gate = at; at += l.mixer_gate == LM_B200_GATE_SIGMOID_HEAD ? H : H * dv; }
     if (l.mixer == LM_B200_MIXER_GATED_LINEAR) { c.a1 = at; at += l.rank_a; }
     c.n = (at + 3) & ~3;
     return c;
@@ -298,6 +302,10 @@ int stream_rec_cols(const lm_b200_layer& l) {
         default: return 0;
     }
 }
+// a dense unit that is not gated
+bool plain_unit(const lm_b200_layer& l) { return l.act == LM_B200_ACT_RELU2 || l.act == LM_B200_ACT_GELU; }
+// a record whose sublayers read the residual stream itself
+bool reads_plain(const lm_b200_layer& l) { return !l.norm_mix_in.w; }
 int glu_kind(int act) { return act == LM_B200_ACT_CLAMPED_GLU ? 1 : act == LM_B200_ACT_GELU_GLU ? 2 : 0; }
 bool stream_norm_ok(const lm_b200_norm& n) { return n.w && (n.kind == LM_B200_NORM_LAYER || n.kind == LM_B200_NORM_RMS); }
 // router outputs of a record and the columns of its logits (the shared unit's gate row behind them)
@@ -307,8 +315,11 @@ int route_cols(const lm_b200_layer& l) { return route_outputs(l) + (l.router == 
 // one mixer of a stream record (not a pair)
 int check_stream_mixer(const lm_b200_layer& l) {
     if (l.heads <= 0 || l.dim <= 0 || l.vdim <= 0 || l.n_in != stream_cols(l).n) return LM_B200_EINVAL;
-    if (l.mixer_gate != LM_B200_GATE_SIGMOID && l.mixer_gate != LM_B200_GATE_NONE && l.mixer_gate != LM_B200_GATE_SILU)
+    if (l.mixer_gate != LM_B200_GATE_SIGMOID && l.mixer_gate != LM_B200_GATE_NONE && l.mixer_gate != LM_B200_GATE_SILU &&
+        l.mixer_gate != LM_B200_GATE_SIGMOID_HEAD)
         return LM_B200_EINVAL;
+    if (l.mixer_gate == LM_B200_GATE_SIGMOID_HEAD && l.mixer != LM_B200_MIXER_LATENT_ATTENTION) return LM_B200_EUNSUPPORTED;
+    if (l.chunk != 0 && (l.chunk < 0 || l.mixer != LM_B200_MIXER_ROTARY_ATTENTION)) return LM_B200_EINVAL;
     const bool rot_ok = l.rot_dims >= 0 && l.rot_dims % 2 == 0 && (l.rot_dims == 0 || l.rot_freq) &&
                         (l.rot_layout == LM_B200_ROT_INTERLEAVED || l.rot_layout == LM_B200_ROT_HALF);
     switch (l.mixer) {
@@ -336,9 +347,9 @@ int check_stream_mixer(const lm_b200_layer& l) {
             if (l.dim > 256 || l.heads > 32767) return LM_B200_EUNSUPPORTED;
             break;
         case LM_B200_MIXER_ROTARY_ATTENTION:
-            if (l.kv_heads <= 0 || l.heads % l.kv_heads || l.vdim != l.dim || !l.q_norm || !l.k_norm || !l.k_pages || !l.v_pages || !rot_ok ||
-                l.rot_dims > l.dim || l.mixer_gate != LM_B200_GATE_NONE)
+            if (l.kv_heads <= 0 || l.heads % l.kv_heads || l.vdim != l.dim || !l.k_pages || !l.v_pages || !rot_ok || l.rot_dims > l.dim)
                 return LM_B200_EINVAL;
+            if (l.mixer_gate == LM_B200_GATE_SILU) return LM_B200_EUNSUPPORTED;
             if (l.dim > 256 || l.heads > 65535 || l.rot_layout != LM_B200_ROT_INTERLEAVED) return LM_B200_EUNSUPPORTED;
             break;
         case LM_B200_MIXER_GATED_LINEAR:
@@ -359,7 +370,10 @@ int check_stream_mixer(const lm_b200_layer& l) {
 
 int check_stream_layer(const lm_b200_model& m, const lm_b200_layer& l) {
     if (l.streams < 1 || l.streams > 8) return LM_B200_EUNSUPPORTED;
-    if (!stream_norm_ok(l.norm_mix_in) || !l.w_in || !l.w_o) return LM_B200_EINVAL;
+    if (!l.w_in || !l.w_o || (!reads_plain(l) && !stream_norm_ok(l.norm_mix_in))) return LM_B200_EINVAL;
+    if (reads_plain(l) && (l.streams != 1 || l.parallel)) return LM_B200_EUNSUPPORTED;
+    for (const lm_b200_norm* n : {&l.norm_mix_out, &l.norm_ff_out})      // norms on the outputs
+        if (n->w && (n->kind != LM_B200_NORM_RMS || n->b || !reads_plain(l))) return LM_B200_EUNSUPPORTED;
     for (int q = 0; q < (l.ff == LM_B200_FF_NONE ? 1 : 2); ++q)
         if (!l.hc_in[q] || !l.hc_out[q] || !l.hc_mix[q]) return LM_B200_EINVAL;
     if (l.mixer == LM_B200_MIXER_PAIR && (!l.part[0] || !l.part[1] || l.n_in != l.part[0]->n_in + l.part[1]->n_in)) return LM_B200_EINVAL;
@@ -374,9 +388,10 @@ int check_stream_layer(const lm_b200_model& m, const lm_b200_layer& l) {
         if (l.streams != 1) return LM_B200_EUNSUPPORTED;
     }
     if (l.ff == LM_B200_FF_NONE) return LM_B200_OK;
-    if (!stream_norm_ok(l.norm_ff_in)) return LM_B200_EINVAL;
+    if (reads_plain(l) ? l.norm_ff_in.w != nullptr : !stream_norm_ok(l.norm_ff_in)) return LM_B200_EINVAL;
+    if (l.norm_ff_out.w && l.ff != LM_B200_FF_DENSE) return LM_B200_EUNSUPPORTED;
     if (l.parallel && l.norm_ff_in.kind != l.norm_mix_in.kind) return LM_B200_EUNSUPPORTED;
-    if (l.ff == LM_B200_FF_DENSE && l.act == LM_B200_ACT_RELU2) return (l.dense_ff > 0 && l.ws_gate_up && l.ws_down) ? LM_B200_OK : LM_B200_EINVAL;
+    if (l.ff == LM_B200_FF_DENSE && plain_unit(l)) return (l.dense_ff > 0 && l.ws_gate_up && l.ws_down) ? LM_B200_OK : LM_B200_EINVAL;
     if (l.act != LM_B200_ACT_CLAMPED_GLU && l.act != LM_B200_ACT_SILU_GLU && l.act != LM_B200_ACT_GELU_GLU) return LM_B200_EUNSUPPORTED;
     if (l.ff == LM_B200_FF_DENSE) return (l.dense_ff > 0 && l.ws_gate_up && l.ws_down) ? LM_B200_OK : LM_B200_EINVAL;
     if (l.ff != LM_B200_FF_ROUTED_EXPERTS) return LM_B200_EUNSUPPORTED;
@@ -463,7 +478,7 @@ int mixer(lm_b200_engine* e, const lm_b200_layer& l, const float* h, const void*
     LCK(lm::launch_sink_attention(e->qk, nq + nk, l.k_pages, l.v_pages, pm, a, v.rm, e->att, tc_o ? e->attb : nullptr, e->split_ws, e->split_arrived, M, st));
     if (tc_o) {
         if (fuse_x) {
-            const dia::GemmEpilogue ep{fuse_x, l.norm_mix_out.w, l.norm_mix_out.b, l.norm_mix_out.alpha};
+            const dia::GemmEpilogue ep{fuse_x, l.norm_mix_out.w, l.norm_mix_out.b, l.norm_mix_out.alpha, nullptr};
             LCK(dia::launch_gemm_tcgen05_bf16(e->attb, 1, l.w_o, D, fuse_x, M, D, nq, ep, nullptr, st));
             return LM_B200_OK;
         }
@@ -541,7 +556,7 @@ int feed_forward(lm_b200_engine* e, const lm_b200_layer& l, const float* h, cons
 int product(lm_b200_engine* e, const float* A, const void* Ab, int lda, const void* W, float* out, int M, int N, int K,
             bool add, cudaStream_t st) {
     if (Ab && lda == K && tensor_path(e, M, N, K)) {
-        const dia::GemmEpilogue ep{add ? out : nullptr, nullptr, nullptr, 0.f};
+        const dia::GemmEpilogue ep{add ? out : nullptr, nullptr, nullptr, 0.f, nullptr};
         LCK(dia::launch_gemm_tcgen05_bf16(Ab, 1, W, N, out, M, N, K, ep, nullptr, st));
         return LM_B200_OK;
     }
@@ -639,7 +654,7 @@ int parallel_layer(lm_b200_engine* e, const lm_b200_layer& l, const StepView& v,
         if (rc) return rc;
     }
     if (only != 1 && l.ff == LM_B200_FF_DENSE)
-        LCK(lm::launch_xielu_rows(e->proj, c.n, c.up, l.act_p, l.act_q, e->outcat, ko, c.mix_out, ob, M, l.dense_ff, st));
+        LCK(lm::launch_unit_act_rows(e->proj, c.n, c.up, lm::kActXielu, l.act_p, l.act_q, e->outcat, ko, c.mix_out, ob, M, l.dense_ff, st));
     return product(e, e->outcat, ob, ko, l.w_out, only == 0 ? e->x : y_out, M, D, ko, only == 0, st);
 }
 
@@ -690,7 +705,8 @@ int stream_mixer_kernels(lm_b200_engine* e, const lm_b200_layer& l, const MixPla
             LCK(lm::launch_latent_attention_rows(e->qlat, l.latent_pages, pm, H, l.kv_rank, l.sink, v.rm, e->olat, M, st, rd,
                                                  l.window > 0 ? l.window : 0));
         // sum_j p_j (W_uv,h c_j) = W_uv,h (sum_j p_j c_j), times the sigmoid of the gate columns
-        LCK(lm::launch_head_linear(e->olat, no, l.w_uv, at.out, at.ldo, at.out_b, M, H, l.vdim, l.kv_rank, at.scale, gate, ld, st));
+        LCK(lm::launch_head_linear(e->olat, no, l.w_uv, at.out, at.ldo, at.out_b, M, H, l.vdim, l.kv_rank, at.scale, gate, ld, st,
+                                   0, 0, l.mixer_gate == LM_B200_GATE_SIGMOID_HEAD));
     } else if (l.mixer == LM_B200_MIXER_GATED_DELTA) {
         const lm::DeltaShape d{H, l.kv_heads, l.dim, l.vdim, l.conv_taps, l.unit_eps, l.conv_w, l.a_log, l.dt_bias};
         const int k0 = l.kv_heads * l.dim, v0 = 2 * k0, d0 = v0 + nv, b0 = d0 + H, ldr = stream_rec_cols(l);
@@ -710,12 +726,13 @@ int stream_mixer_kernels(lm_b200_engine* e, const lm_b200_layer& l, const MixPla
                                         l.head_decay, false, M <= lm::kRowsKernelMax));
         LCK(lm::launch_head_norm_gate(at.out, at.ldo, at.out_b, l.head_norm, gate, ld, H, l.vdim, e->m.eps, M, st, gate_act, at.scale));
     } else if (l.mixer == LM_B200_MIXER_ROTARY_ATTENTION) {
-        // the score multiplier rides on q; the raw key projection is the value when the record says so
+        // the score multiplier rides on q; the raw key projection is the value when the record says so; the gate's sigmoid is
+        // applied where the attention writes its output
         const lm::TalkShape a{H, l.kv_heads, l.dim, l.vdim, l.rot_dims, l.scale, l.rot_freq, nullptr, nullptr, 0, l.rot_amp};
         LCK(lm::launch_talk_prep(proj, ld, nullptr, c.q, c.k, c.v, -1, a, l.q_norm, l.k_norm, e->m.eps, l.k_pages, l.v_pages, pm, v.rm, M, st));
-        const lm::AttnShape s{H, l.kv_heads, l.dim, l.window > 0 ? l.window : 0, 0, 1.f, 0.f, nullptr, nullptr, l.sink};
+        const lm::AttnShape s{H, l.kv_heads, l.dim, l.window > 0 ? l.window : 0, 0, 1.f, 0.f, nullptr, nullptr, l.sink, l.chunk};
         LCK(lm::launch_sink_attention(proj + c.q, ld, l.k_pages, l.v_pages, pm, s, v.rm, at.out, at.out_b, e->split_ws, e->split_arrived, M,
-                                      st, at.ldo, at.scale));
+                                      st, at.ldo, at.scale, gate, ld));
     } else if (l.mixer == LM_B200_MIXER_GATED_LINEAR) {
         LCK(lm::launch_decay_proj(proj + c.a1, ld, l.w_a2, l.dt_bias, l.decay_tau, e->rec, H * l.dim, l.rank_a, M, st));
         const lm::ScanInputs si{c.q, c.k, 0, c.v, 0};
@@ -788,18 +805,23 @@ int token_input(lm_b200_engine* e, const lm_b200_layer& l, const float* x, const
     return product_ld(e, e->side_g, n, gb, l.w_side_proj, y, M, D, n, st);
 }
 
-// a dense unit that is not gated: out = max(h W_up^T, 0)^2 W_down^T
-int relu2_unit(lm_b200_engine* e, const float* h, const void* hb, int M, const void* w_up, const void* w_down, int F, float* out,
-               cudaStream_t st) {
+// a dense unit that is not gated: out = act(h W_up^T) W_down^T.  The activation stands in the up product's epilogue (a squared
+// relu behind the tensor-core product is a launch of its own).
+int plain_dense_unit(lm_b200_engine* e, const float* h, const void* hb, int M, int act, const void* w_up, const void* w_down, int F,
+                     float* out, cudaStream_t st) {
     const int D = e->m.width;
     if (hb && tensor_path(e, M, F, D) && tensor_path(e, M, D, F)) {
-        LCK(dia::launch_gemm_tcgen05_bf16(hb, 1, w_up, F, e->sgu, M, F, D, kPlain, nullptr, st));
-        LCK(lm::launch_xielu_rows(e->sgu, F, 0, 0.f, 0.f, nullptr, F, 0, e->smidb, M, F, st, true));
+        if (act == lm::kActGelu) {
+            const dia::GemmEpilogue ep{nullptr, nullptr, nullptr, 0.f, e->smidb};
+            LCK(dia::launch_gemm_tcgen05_bf16(hb, 1, w_up, F, e->sgu, M, F, D, ep, nullptr, st));
+        } else {
+            LCK(dia::launch_gemm_tcgen05_bf16(hb, 1, w_up, F, e->sgu, M, F, D, kPlain, nullptr, st));
+            LCK(lm::launch_unit_act_rows(e->sgu, F, 0, act, 0.f, 0.f, nullptr, F, 0, e->smidb, M, F, st));
+        }
         LCK(dia::launch_gemm_tcgen05_bf16(e->smidb, 1, w_down, D, out, M, D, F, kPlain, nullptr, st));
         return LM_B200_OK;
     }
-    LCK(lm::launch_linear(h, D, w_up, 0, e->sgu, F, M, F, D, nullptr, st));
-    LCK(lm::launch_xielu_rows(e->sgu, F, 0, 0.f, 0.f, e->smid, F, 0, nullptr, M, F, st, true));
+    LCK(lm::launch_linear(h, D, w_up, 0, e->smid, F, M, F, D, nullptr, st, act));
     LCK(lm::launch_linear(e->smid, F, w_down, 0, out, D, M, D, F, nullptr, st));
     return LM_B200_OK;
 }
@@ -833,7 +855,9 @@ int stream_ff(lm_b200_engine* e, const lm_b200_layer& l, const float* h, const v
     const int act = glu_kind(l.act);
     wr->y = e->y; wr->parts = nullptr; wr->slot_of = nullptr; wr->sel_w = nullptr; wr->top = 0;
     if (l.ff == LM_B200_FF_DENSE) {
-        if (l.act == LM_B200_ACT_RELU2) return relu2_unit(e, h, hb, M, l.ws_gate_up, l.ws_down, l.dense_ff, e->y, st);
+        if (plain_unit(l))
+            return plain_dense_unit(e, h, hb, M, l.act == LM_B200_ACT_GELU ? lm::kActGelu : lm::kActRelu2, l.ws_gate_up, l.ws_down,
+                                    l.dense_ff, e->y, st);
         return gated_unit(e, l, h, hb, M, l.ws_gate_up, l.ws_down, l.dense_ff, l.act_limit, e->y, st);
     }
     const bool grouped = l.router == LM_B200_ROUTER_SOFTMAX_GROUPED;
@@ -909,6 +933,10 @@ int lm_b200_engine_create(const lm_b200_model* model, const lm_b200_layer* layer
         // the streams run through the whole stack: a stream record stands among stream records with the same number of them
         if ((layers[i].form == LM_B200_FORM_STREAMS) != (layers[0].form == LM_B200_FORM_STREAMS)) return LM_B200_EUNSUPPORTED;
         if (layers[i].form == LM_B200_FORM_STREAMS && layers[i].streams != layers[0].streams) return LM_B200_EINVAL;
+    }
+    if (m.bigram) {
+        if (m.bigram_buckets <= 0 || m.bigram_mul_prev < 0 || m.bigram_mul_cur < 0 || !m.token_pages) return LM_B200_EINVAL;
+        if (layers[0].form != LM_B200_FORM_STREAMS) return LM_B200_EUNSUPPORTED;
     }
     Guard g(device);
     if (!g.ok) return LM_B200_ECUDA;
@@ -1089,8 +1117,13 @@ int run_stream_layers(lm_b200_engine* e, const StepView& v, int M, int n_seq, fl
     const bool bf = e->m.precision == LM_B200_PRECISION_BF16 && M >= kTensorRowsMin;
     void* hb = bf ? e->hb : nullptr;
     void* h2b = bf ? e->h2b : nullptr;
+    // A record without input norms (one stream) reads the stream where it stands: its sublayers' fp32 input is e->xs itself, and
+    // whatever writes the stream in front of such a read leaves the bf16 operand beside it.
+    const bool plain0 = reads_plain(e->layers[0]);
+    const lm::PageMap pm{e->m.page_table, e->m.max_pages, e->m.page_size};
+    const lm::BigramRows bg{e->m.bigram, e->m.bigram_buckets, e->m.bigram_mul_prev, e->m.bigram_mul_cur, e->m.token_pages, pm, v.rm};
     LCK(lm::launch_streams_embed(e->m.embed, v.token, e->m.embed_scale != 0.f ? e->m.embed_scale : 1.f, e->xs, s, M, e->m.vocab, D, st,
-                                 e->m.embed_norm, eps));
+                                 e->m.embed_norm, eps, bg, plain0 ? hb : nullptr));
     const lm::StreamWrite none{nullptr, nullptr, nullptr, nullptr, nullptr, nullptr, 0};
     // A parallel record's feed-forward reads the streams the mixer read.  With one stream and one set of read weights both
     // norms share their statistics, and the step that produces the mixer's input writes the feed-forward's beside it.
@@ -1102,16 +1135,27 @@ int run_stream_layers(lm_b200_engine* e, const StepView& v, int M, int n_seq, fl
         if (shares_read(l)) { ex.norm_w2 = l.norm_ff_in.w; ex.h2 = e->h2; ex.h2_b = h2b; }
         return ex;
     };
-    LCK(lm::launch_streams_step(e->xs, s, none, e->layers[0].hc_in[0], e->layers[0].norm_mix_in.w, eps, nullptr, e->h, hb, M, D, st,
-                                read_of(e->layers[0], lm::StreamExtra{})));
+    if (!plain0)
+        LCK(lm::launch_streams_step(e->xs, s, none, e->layers[0].hc_in[0], e->layers[0].norm_mix_in.w, eps, nullptr, e->h, hb, M, D, st,
+                                    read_of(e->layers[0], lm::StreamExtra{})));
     for (int i = 0; i < n; ++i) {
         const lm_b200_layer& l = e->layers[i];
         const bool par = l.parallel && l.ff != LM_B200_FF_NONE;
-        int rc = stream_mixer(e, l, e->h, hb, v, M, n_seq, par ? e->ymix : e->y, st);
+        const bool plain = reads_plain(l);
+        int rc = stream_mixer(e, l, plain ? e->xs : e->h, hb, v, M, n_seq, par ? e->ymix : e->y, st);
         if (rc) return rc;
         lm::StreamWrite wr{l.hc_mix[0], l.hc_out[0], e->y, nullptr, nullptr, nullptr, 0};
         lm::StreamExtra wx{};
-        if (par) {
+        wx.y_norm_w = l.norm_mix_out.w;
+        if (plain && l.ff != LM_B200_FF_NONE) {
+            LCK(lm::launch_streams_step(e->xs, s, wr, nullptr, nullptr, eps, nullptr, nullptr, hb, M, D, st, wx));
+            wx = lm::StreamExtra{};
+            rc = stream_ff(e, l, e->xs, hb, M, &wr, &wx, st);
+            if (rc) return rc;
+            wr.mix = l.hc_mix[1];
+            wr.out = l.hc_out[1];
+            wx.y_norm_w = l.norm_ff_out.w;
+        } else if (par) {
             if (!shares_read(l)) {
                 lm::StreamExtra rx{};
                 rx.rms = l.norm_ff_in.kind == LM_B200_NORM_RMS;
@@ -1146,7 +1190,10 @@ int run_stream_layers(lm_b200_engine* e, const StepView& v, int M, int n_seq, fl
         // this sublayer's write with the next layer's read, or with the closing sum of the streams
         if (i + 1 < n) {
             const lm_b200_layer& nx = e->layers[i + 1];
-            LCK(lm::launch_streams_step(e->xs, s, wr, nx.hc_in[0], nx.norm_mix_in.w, eps, nullptr, e->h, hb, M, D, st, read_of(nx, wx)));
+            if (reads_plain(nx))
+                LCK(lm::launch_streams_step(e->xs, s, wr, nullptr, nullptr, eps, nullptr, nullptr, hb, M, D, st, wx));
+            else
+                LCK(lm::launch_streams_step(e->xs, s, wr, nx.hc_in[0], nx.norm_mix_in.w, eps, nullptr, e->h, hb, M, D, st, read_of(nx, wx)));
             if (layers_out)
                 LCK(lm::launch_streams_step(e->xs, s, none, nullptr, nullptr, eps, nullptr, layers_out + (size_t)i * M * D, nullptr, M, D, st));
         } else {

@@ -21,6 +21,7 @@ struct AttnShape {
     int heads, kv_heads, dim, window, keep_first;
     float scale, softcap;
     const float* temp; const float* slopes; const float* sink;                  // per query head; each may be null
+    int chunk;                                                                  // > 0: keys of the query's own block of `chunk` positions only
 };
 // After a kernel of a short step gave x[a][n] its new value, the NEXT sublayer's input for that element can follow in the
 // same thread when every scheduled sequence has exactly one row in the step: norm, taps over the sequence's tail, and
@@ -39,6 +40,8 @@ struct GroupMap { int* a_row; float* a_scale; int* a_expert; int* n_slots; };   
 struct GroupedRoute { int n; int n_real; int count; int keep; float scale; const float* correction; };
 // activation of the gated units (kind: kGluSilu / kGluClamped / kGluGelu of lm_device.cuh; the clamp of routed / dense and shared units)
 struct GluAct { int kind; float limit; float shared_limit; };
+// activation of a unit that is not gated, and of the activated products
+constexpr int kActNone = 0, kActXielu = 1, kActRelu2 = 2, kActGelu = 3;
 
 cudaError_t launch_embed(const void* table_bf16, const int* ids, float* out, int M, int V, int D, cudaStream_t st);
 cudaError_t launch_dyt_tapmix(const float* x, const NormW& n, const float* cw, int taps, const float* tail, const RowMeta& rm,
@@ -46,7 +49,7 @@ cudaError_t launch_dyt_tapmix(const float* x, const NormW& n, const float* cw, i
 cudaError_t launch_tapmix_tail(const float* x, const NormW& n, int taps, float* tail, const SeqMeta& sm, int n_seq, int D,
                                cudaStream_t st);
 cudaError_t launch_linear(const float* A, int lda, const void* W_bf16, long long w_expert_stride, float* Y, int ldy, int M,
-                          int N, int K, const GroupMap* gm, cudaStream_t st);
+                          int N, int K, const GroupMap* gm, cudaStream_t st, int act = kActNone);
 // the fused forms for a step of at most kRowsKernelMax rows
 cudaError_t launch_dyt_tapmix_seq(const float* x, const NormW& n, const float* cw, int taps, float* tail, const SeqMeta& sm,
                                   const RowMeta& rm, int n_seq, float* out, int D, cudaStream_t st);
@@ -65,10 +68,12 @@ cudaError_t launch_router_rows(const float* h, int D, const void* Wr, int E, int
 cudaError_t launch_qk_norm_cache(float* qk, int nq, int nk, const float* qw, const float* kw, float eps, float* kcache,
                                  float* vcache, const PageMap& pm, int kv_heads, int dim, const RowMeta& rm, int M,
                                  cudaStream_t st);
-// ldo: row stride of the output (0: heads * dim); out_scale multiplies it
+// ldo: row stride of the output (0: heads * dim); out_scale multiplies it, and so does the sigmoid of gate[row * ldg + column],
+// if given
 cudaError_t launch_sink_attention(const float* qk, int q_stride, const float* kcache, const float* vcache, const PageMap& pm,
                                   const AttnShape& a, const RowMeta& rm, float* out, void* out_bf16, float* split_ws,
-                                  unsigned* arrived, int M, cudaStream_t st, int ldo = 0, float out_scale = 1.f);
+                                  unsigned* arrived, int M, cudaStream_t st, int ldo = 0, float out_scale = 1.f,
+                                  const float* gate = nullptr, int ldg = 0);
 cudaError_t launch_router_topk(const float* z, int E, int top, int M, int* sel_e, float* sel_w, cudaStream_t st,
                                const float* bias = nullptr, bool softmax_top = false, const GroupedRoute* gr = nullptr);
 cudaError_t launch_moe_group(const int* sel_e, const float* sel_w, int n_assign, int top, int E, int pad, const GroupMap& gm,
@@ -103,9 +108,9 @@ cudaError_t launch_layernorm_rows(const float* x, const int* rows, const float* 
                                   float* out, void* out_bf16, int M, int D, cudaStream_t st, bool rms = false);
 cudaError_t launch_pair_rows(const float* x, const float* x0, float* cat, void* cat_bf16, int M, int D, cudaStream_t st);
 cudaError_t launch_add_rows(float* x, const float* y, int M, int D, cudaStream_t st);
-// relu2: max(z, 0)^2 instead of the xIELU; out may be null when only the bf16 copy is wanted
-cudaError_t launch_xielu_rows(const float* proj, int ld, int off, float ap, float an, float* out, int ldo, int out_off,
-                              void* out_bf16, int M, int F, cudaStream_t st, bool relu2 = false);
+// act: kActXielu, kActRelu2 or kActGelu (ap / an are the xIELU's); out may be null when only the bf16 copy is wanted
+cudaError_t launch_unit_act_rows(const float* proj, int ld, int off, int act, float ap, float an, float* out, int ldo, int out_off,
+                                 void* out_bf16, int M, int F, cudaStream_t st);
 cudaError_t launch_talk_prep(float* proj, int ld, const float* bias, int q_off, int k_off, int v_off, int gate_off,
                              const TalkShape& a, const float* qw, const float* kw, float eps, float* kcache, float* vcache,
                              const PageMap& pm, const RowMeta& rm, int M, cudaStream_t st);
@@ -152,15 +157,20 @@ struct StreamWrite { const float* mix; const float* out; const float* y; const f
 // the same streams); ident_h [M][D] - what an assignment without a slot (slot_of < 0, an identity expert) adds, times its
 // weight; y_gate - y is multiplied by sigmoid(y_gate[row * y_gate_ld]); rms - the norm is x / sqrt(mean(x^2) + eps) w;
 // norm_w2 / h2 / h2_b - a second norm weight on the same statistics and where its result goes; y_norm_w - y is RMS-normed with
-// this weight before it is written (no parts then).
+// this weight before it is written (no parts then).  h may be null while h_bf16 is not: only the bf16 copy is written.
 struct StreamExtra { const float* y2; const float* out2; const float* ident_h; const float* y_gate; int y_gate_ld; int rms;
                      const float* norm_w2; float* h2; void* h2_b; const float* y_norm_w; };
 cudaError_t launch_streams_step(float* X, int streams, const StreamWrite& wr, const float* in, const float* norm_w, float eps,
                                 const int* rows, float* h, void* h_bf16, int M, int D, cudaStream_t st,
                                 const StreamExtra& ex = StreamExtra{});
-// norm_w: the rows get an RMS norm with this weight
+// The pair table of the embedding: row (previous * mul_prev + token * mul_cur) mod buckets, row `buckets` for position 0, is added
+// to the scaled embedding row.  The token in front of a sequence's first row of the step comes from its token pages
+// [page][page_size], into which every row writes its own token.  table == nullptr: none.
+struct BigramRows { const void* table; int buckets; int mul_prev; int mul_cur; int* token_pages; PageMap pm; RowMeta rm; };
+// norm_w: the rows get an RMS norm with this weight.  x_bf16 (streams == 1): the bf16 copy of the rows
 cudaError_t launch_streams_embed(const void* table_bf16, const int* ids, float scale, float* X, int streams, int M, int V, int D,
-                                 cudaStream_t st, const float* norm_w = nullptr, float eps = 0.f);
+                                 cudaStream_t st, const float* norm_w = nullptr, float eps = 0.f, const BigramRows& bg = BigramRows{},
+                                 void* x_bf16 = nullptr);
 // n channels of which the first `dims` turn with the position (freq [dims / 2]; pairs (2i, 2i + 1), or (i, i + dims / 2) with
 // half_layout)
 struct RotPart { int n; int dims; int half_layout; const float* freq; };
@@ -180,9 +190,10 @@ bool latent_attention_rows_supported(int H, int R);
 cudaError_t launch_latent_attention_rows(const float* q, const float* pages, const PageMap& pm, int H, int R, const float* sink,
                                          const RowMeta& rm, float* out, int M, cudaStream_t st, int key_extra = 0, int window = 0);
 // Y[m][h N + n] = alpha * sum_k A[m][h K + k] W[h][n][k]  [* sigmoid(gate[m][h N + n])], fp32 arithmetic on bf16 weights.
-// a_hs / y_hs > 0: the heads of A / Y are that many columns apart instead of K / N
+// a_hs / y_hs > 0: the heads of A / Y are that many columns apart instead of K / N.  head_gate: one gate column per head
 cudaError_t launch_head_linear(const float* A, int lda, const void* W, float* Y, int ldy, void* y_bf16, int M, int H, int N, int K,
-                               float alpha, const float* gate, int ldg, cudaStream_t st, int a_hs = 0, int y_hs = 0);
+                               float alpha, const float* gate, int ldg, cudaStream_t st, int a_hs = 0, int y_hs = 0,
+                               bool head_gate = false);
 // log-space gates of the stabilised matrix memory, per (sequence, head) along the sequence's rows: i = cap tanh((z_i + b_i) /
 // cap), f = logsigmoid(cap tanh((z_f + b_f) / cap)), m_t = max(f + m_(t-1), i) (m = 0 before position 0, carried in
 // m_state[slot][head]); the columns i_off + h, f_off + h of the row become a = exp(f + m_(t-1) - m_t), b = exp(i - m_t), and

@@ -159,13 +159,14 @@ __global__ void dyt_tapmix_seq_kernel(const float* __restrict__ x, const float* 
 // ---------------------------------------------------------------------------------------------------------------------
 // Y[a][n] = sum_k scale_a * A[src_a][k] * W_e[n][k].  Without the maps: src_a = a, scale 1, expert 0.  With them
 // (expert groups): a indexes padded assignment slots, a_row[a] < 0 is padding, the expert of a tile is a_expert of its
-// first slot.  n_slots (device) bounds the slots in use; the grid covers the host's upper bound.
+// first slot.  n_slots (device) bounds the slots in use; the grid covers the host's upper bound.  act: the unit activation of
+// the result.
 constexpr int BM = 64, BN = 64, BK = 16;
 
 __global__ void __launch_bounds__(256)
 linear_tile_kernel(const float* __restrict__ A, int lda, const __nv_bfloat16* __restrict__ W, long long w_expert_stride,
                    float* __restrict__ Y, int ldy, int M, int N, int K, const int* __restrict__ a_row,
-                   const float* __restrict__ a_scale, const int* __restrict__ a_expert, const int* __restrict__ n_slots) {
+                   const float* __restrict__ a_scale, const int* __restrict__ a_expert, const int* __restrict__ n_slots, int act) {
     __shared__ __align__(16) float As[BK][BM + 4];
     __shared__ __align__(16) float Bs[BK][BN + 4];
     const int m0 = blockIdx.y * BM, n0 = blockIdx.x * BN;
@@ -242,7 +243,7 @@ linear_tile_kernel(const float* __restrict__ A, int lda, const __nv_bfloat16* __
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const int n = n0 + tx * 4 + j;
-            if (n < N) Y[(size_t)a * ldy + n] = acc[i][j];
+            if (n < N) Y[(size_t)a * ldy + n] = act ? unit_act(act, acc[i][j], 0.f, 0.f) : acc[i][j];
         }
     }
 }
@@ -279,14 +280,14 @@ __device__ __forceinline__ void tap_out_warp(const TapOut& t, int a, int n, int 
     if (lane == 0) t.h[(size_t)a * D + n] = acc;
 }
 
-// Y[a][n] = dot, or with res_x: res_x[a][n] += DynamicTanh(dot), += dot without a norm (the residual stream takes the
+// Y[a][n] = dot (act: its activation), or with res_x: res_x[a][n] += DynamicTanh(dot), += dot without a norm (the residual stream takes the
 // sublayer's output)
 __global__ void __launch_bounds__(256)
 linear_rows_kernel(const float* __restrict__ A, int lda, const __nv_bfloat16* __restrict__ W, long long w_expert_stride,
                    float* __restrict__ Y, int ldy, int M, int N, int K, const int* __restrict__ a_row,
                    const float* __restrict__ a_scale, const int* __restrict__ a_expert, const int* __restrict__ n_slots,
                    float* __restrict__ res_x, const float* __restrict__ nw, const float* __restrict__ nb, float alpha,
-                   const TapOut next) {
+                   const TapOut next, int act) {
     pdl_release();
     const bool mapped = a_row || a_scale || a_expert || n_slots;      // the maps are an earlier kernel's output
     if (mapped) pdl_wait();
@@ -307,7 +308,7 @@ linear_rows_kernel(const float* __restrict__ A, int lda, const __nv_bfloat16* __
         if (lane == 0) res_x[(size_t)a * ldy + n] = x_new;
         if (next.h) tap_out_warp(next, a, n, ldy, x_new, lane);
     } else if (lane == 0) {
-        Y[(size_t)a * ldy + n] = acc;
+        Y[(size_t)a * ldy + n] = act ? unit_act(act, acc, 0.f, 0.f) : acc;
     }
 }
 
@@ -548,7 +549,7 @@ __global__ void qk_norm_cache_kernel(float* __restrict__ qk, int nq, int nk, con
 
 // ---------------------------------------------------------------------------------------------------------------------
 // Attention of a few rows (decoding), split over the keys.  Query position i sees key j <= i when i - j < window or
-// j < keep_first (window <= 0: every j <= i).  score = cap * tanh(q.k * scale * temp_h / cap) - slope_h * (i - j)
+// j < keep_first (window <= 0: every j <= i); with chunk > 0 only when i and j lie in the same block of `chunk` positions.  score = cap * tanh(q.k * scale * temp_h / cap) - slope_h * (i - j)
 // (cap <= 0: no cap).  One CTA per (row, up to HG query heads of one key/value head, split of the visible keys): a warp
 // takes every eighth key of the split, reads its key and value rows once for all HG heads (lanes over the head size,
 // coalesced), and keeps a running (maximum, denominator, weighted value sum) per head; the CTA's warps are merged and
@@ -561,8 +562,8 @@ constexpr int kAttnMaxDimPerLane = 8;                         // head dim <= 256
 // CTA of at least 4 warps: warp w weighs the splits of head h0 + w, then all threads sum.  scratch: >= 4 * 33 floats
 __device__ __forceinline__ void combine_splits(const float* __restrict__ part, int S, int heads, int dim,
                                                const float* __restrict__ sink, float* __restrict__ out,
-                                               __nv_bfloat16* __restrict__ out_b, int ldo, float out_scale, int r, int h0, int nh,
-                                               float* scratch) {
+                                               __nv_bfloat16* __restrict__ out_b, int ldo, float out_scale,
+                                               const float* __restrict__ gate, int ldg, int r, int h0, int nh, float* scratch) {
     static_assert(kAttnSplitsMax <= 32, "one lane per split");
     const size_t stride = (size_t)(dim + 2);
     const float* src0 = part + (size_t)(r * heads + h0) * S * stride;
@@ -590,6 +591,7 @@ __device__ __forceinline__ void combine_splits(const float* __restrict__ part, i
 #pragma unroll 8
         for (int s = 0; s < S; ++s) o = fmaf(__ldcg(src + s * stride), wgt[s], o);
         o *= wgt[32] * out_scale;
+        if (gate) o *= sigmoidf_(gate[(size_t)r * ldg + (size_t)(h0 + hh) * dim + c]);
         const size_t at = (size_t)r * ldo + (size_t)(h0 + hh) * dim + c;
         out[at] = o;
         if (out_b) out_b[at] = __float2bfloat16_rn(o);
@@ -604,7 +606,7 @@ sink_attention_split_kernel(const float* __restrict__ qk, int q_stride, const fl
                             const float* __restrict__ slopes, const float* __restrict__ sink, int window, int keep_first,
                             const int* __restrict__ row_slot, const int* __restrict__ row_pos, float* __restrict__ part,
                             unsigned* __restrict__ arrived, float* __restrict__ out, __nv_bfloat16* __restrict__ out_b, int ldo,
-                            float out_scale) {
+                            float out_scale, int chunk, const float* __restrict__ gate, int ldg) {
     __shared__ float sm_m[kSplitWarps][HG], sm_l[kSplitWarps][HG];
     __shared__ bool is_last;
     __shared__ float sm_acc[kSplitWarps][HG][32 * kAttnMaxDimPerLane];
@@ -617,7 +619,7 @@ sink_attention_split_kernel(const float* __restrict__ qk, int q_stride, const fl
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int i = row_pos[r];
     const int* pages = table + (size_t)row_slot[r] * max_pages;
-    const int lo = window > 0 ? max(0, i - window + 1) : 0;
+    const int lo = first_key(i, window, chunk);
     const int n_keep = window > 0 ? min(keep_first, lo) : 0;
     const int n_keys = n_keep + (i - lo + 1);
     const int per = (n_keys + S - 1) / S;
@@ -714,7 +716,7 @@ sink_attention_split_kernel(const float* __restrict__ qk, int q_stride, const fl
     if (!is_last) return;
     __threadfence();
     static_assert(HG <= kSplitWarps, "one warp per head in the merge");
-    combine_splits(part, S, heads, dim, sink, out, out_b, ldo, out_scale, r, h0, nh, sm_acc[0][0]);
+    combine_splits(part, S, heads, dim, sink, out, out_b, ldo, out_scale, gate, ldg, r, h0, nh, sm_acc[0][0]);
 }
 
 // ---------------------------------------------------------------------------------------------------------------------
@@ -734,7 +736,8 @@ sink_attention_tile_kernel(const float* __restrict__ qk, int q_stride, const flo
                            int heads, int kv_heads, int dim, float scale, float cap, const float* __restrict__ temp,
                            const float* __restrict__ slopes, const float* __restrict__ sink, int window, int keep_first,
                            const int* __restrict__ row_slot, const int* __restrict__ row_pos, float* __restrict__ out,
-                           __nv_bfloat16* __restrict__ out_b, int ldo, float out_scale, int M) {
+                           __nv_bfloat16* __restrict__ out_b, int ldo, float out_scale, int M, int chunk,
+                           const float* __restrict__ gate, int ldg) {
     constexpr int DP = 64 * NC, QS = DP + 4, C4 = DP / 4;
     extern __shared__ __align__(16) float sm[];
     float* Qs = sm;                                           // [64][QS]
@@ -789,7 +792,7 @@ sink_attention_tile_kernel(const float* __restrict__ qk, int q_stride, const flo
         while (seg_b < n_rows && s_slot[seg_b] == s_slot[seg_a] && s_pos[seg_b] == s_pos[seg_b - 1] + 1) ++seg_b;
         const int* pages = table + (size_t)s_slot[seg_a] * max_pages;
         const int p_first = s_pos[seg_a], p_last = s_pos[seg_b - 1];
-        const int lo = window > 0 ? max(0, p_first - window + 1) : 0;
+        const int lo = first_key(p_first, window, chunk);
         const int n_keep = window > 0 ? min(keep_first, lo) : 0;
         for (int phase = 0; phase < 2; ++phase) {
             const int k_begin = phase == 0 ? 0 : lo, k_end = phase == 0 ? n_keep : p_last + 1;
@@ -871,12 +874,12 @@ sink_attention_tile_kernel(const float* __restrict__ qk, int q_stride, const flo
                 for (int i = 0; i < 4; ++i) {
                     const int row = ty * 4 + i;
                     const bool live = row >= seg_a && row < seg_b;
-                    const int qi = s_pos[row];
+                    const int qi = s_pos[row], q_lo = live ? first_key(qi, window, chunk) : 0;
                     float mx = -CUDART_INF_F;
 #pragma unroll
                     for (int j = 0; j < 4; ++j) {
                         const int key = j0 + tx + 16 * j;
-                        const bool ok = live && key < k_end && key <= qi && (window <= 0 || qi - key < window || key < keep_first);
+                        const bool ok = live && key < k_end && key <= qi && (key >= q_lo || (window > 0 && key < keep_first));
                         float v = sc[i][j] * mult;
                         if (cap > 0.f) v = cap * tanhf(v * inv_cap);
                         v -= slope * (float)(qi - key);
@@ -946,7 +949,8 @@ sink_attention_tile_kernel(const float* __restrict__ qk, int q_stride, const flo
             for (int u = 0; u < 4; ++u) {
                 const int col = 64 * c + tx * 4 + u;
                 if (col < dim) {
-                    const float v = o[i][4 * c + u] * inv;
+                    float v = o[i][4 * c + u] * inv;
+                    if (gate) v *= sigmoidf_(gate[(size_t)(r0 + row) * ldg + (size_t)h * dim + col]);
                     out[base + col] = v;
                     if (out_b) out_b[base + col] = __float2bfloat16_rn(v);
                 }
@@ -1142,7 +1146,8 @@ cudaError_t launch_tapmix_tail(const float* x, const NormW& n, int taps, float* 
 }
 
 cudaError_t launch_linear(const float* A, int lda, const void* W, long long w_expert_stride, float* Y, int ldy, int M, int N,
-                          int K, const GroupMap* gm, cudaStream_t st) {
+                          int K, const GroupMap* gm, cudaStream_t st, int act) {
+    if (act == kActXielu) return cudaErrorNotSupported;       // (its two numbers are not handed in here)
     const int* a_row = gm ? gm->a_row : nullptr;
     const float* a_scale = gm ? gm->a_scale : nullptr;
     const int* a_expert = gm ? gm->a_expert : nullptr;
@@ -1153,10 +1158,10 @@ cudaError_t launch_linear(const float* A, int lda, const void* W, long long w_ex
     if (M <= kRowsKernelMax || (N <= kRowsKernelMaxOut && M <= 65535))
         return launch_pdl(linear_rows_kernel, dim3((N + 7) / 8, M), dim3(256), 0, st, A, lda, w, w_expert_stride, Y, ldy, M, N, K,
                           a_row, a_scale, a_expert, n_slots, (float*)nullptr, (const float*)nullptr, (const float*)nullptr, 0.f,
-                          TapOut{});
+                          TapOut{}, act);
     else
         linear_tile_kernel<<<dim3((N + BN - 1) / BN, (M + BM - 1) / BM), 256, 0, st>>>(A, lda, w, w_expert_stride, Y, ldy, M, N,
-                                                                                      K, a_row, a_scale, a_expert, n_slots);
+                                                                                      K, a_row, a_scale, a_expert, n_slots, act);
     return cudaGetLastError();
 }
 
@@ -1171,7 +1176,7 @@ cudaError_t launch_linear_rows_residual(const float* A, int lda, const void* W, 
                                         const TapOut& next, cudaStream_t st) {
     return launch_pdl(linear_rows_kernel, dim3((N + 7) / 8, M), dim3(256), 0, st, A, lda, reinterpret_cast<const __nv_bfloat16*>(W),
                       0LL, (float*)nullptr, N, M, N, K, (const int*)nullptr, (const float*)nullptr, (const int*)nullptr,
-                      (const int*)nullptr, x, n.w, n.b, n.alpha, next);
+                      (const int*)nullptr, x, n.w, n.b, n.alpha, next, 0);
 }
 
 cudaError_t launch_gated_rows(const float* A, int lda, const void* W, long long w_expert_stride, float* mid, int n_assign, int F,
@@ -1211,7 +1216,8 @@ cudaError_t launch_qk_norm_cache(float* qk, int nq, int nk, const float* qw, con
 template <int NC>
 static cudaError_t launch_attention_tiles(const float* qk, int q_stride, const float* kcache, const float* vcache,
                                           const PageMap& pm, const AttnShape& a, const RowMeta& rm, float* out,
-                                          __nv_bfloat16* out_b, int ldo, float out_scale, int M, cudaStream_t st) {
+                                          __nv_bfloat16* out_b, int ldo, float out_scale, int M, cudaStream_t st, const float* gate,
+                                          int ldg) {
     constexpr int DP = 64 * NC;
     const size_t smem = (size_t)(2 * kTQ * (DP + 4) + kTK * DP + kTQ * kTPStride) * sizeof(float) + 2 * kTQ * sizeof(int);
     static bool attr[64] = {};
@@ -1225,7 +1231,7 @@ static cudaError_t launch_attention_tiles(const float* qk, int q_stride, const f
     }
     sink_attention_tile_kernel<NC><<<dim3((M + kTQ - 1) / kTQ, a.heads), kTileThreads, smem, st>>>(
         qk, q_stride, kcache, vcache, pm.table, pm.max_pages, pm.page_size, a.heads, a.kv_heads, a.dim, a.scale, a.softcap,
-        a.temp, a.slopes, a.sink, a.window, a.keep_first, rm.slot, rm.pos, out, out_b, ldo, out_scale, M);
+        a.temp, a.slopes, a.sink, a.window, a.keep_first, rm.slot, rm.pos, out, out_b, ldo, out_scale, M, a.chunk, gate, ldg);
     return cudaGetLastError();
 }
 
@@ -1233,38 +1239,40 @@ template <int HG>
 static cudaError_t launch_attention_splits(const float* qk, int q_stride, const float* kcache, const float* vcache,
                                            const PageMap& pm, const AttnShape& a, const RowMeta& rm, float* out,
                                            __nv_bfloat16* out_b, int ldo, float out_scale, int M, float* split_ws, unsigned* arrived,
-                                           cudaStream_t st) {
+                                           cudaStream_t st, const float* gate, int ldg) {
     const int group = a.heads / a.kv_heads, chunks = (group + HG - 1) / HG;
     // enough CTAs for two per SM, at least 16 keys per split where the window bounds the keys
-    const long long max_keys = a.window > 0 ? (long long)a.window + a.keep_first : (long long)pm.max_pages * pm.page_size;
+    long long max_keys = a.window > 0 ? (long long)a.window + a.keep_first : (long long)pm.max_pages * pm.page_size;
+    if (a.chunk > 0) max_keys = std::min<long long>(max_keys, (long long)a.chunk + (a.window > 0 ? a.keep_first : 0));
     const int others = M * a.kv_heads * chunks;
     int S = (2 * 148 + others - 1) / others;
     S = (int)std::max<long long>(1, std::min<long long>(std::min(S, kAttnSplitsMax), (max_keys + 15) / 16));
     return launch_pdl(sink_attention_split_kernel<HG>, dim3(M, a.kv_heads * chunks, S), dim3(kSplitThreads), 0, st, qk, q_stride,
                       kcache, vcache, pm.table, pm.max_pages, pm.page_size, a.heads, a.kv_heads, a.dim, a.scale, a.softcap, a.temp,
-                      a.slopes, a.sink, a.window, a.keep_first, rm.slot, rm.pos, split_ws, arrived, out, out_b, ldo, out_scale);
+                      a.slopes, a.sink, a.window, a.keep_first, rm.slot, rm.pos, split_ws, arrived, out, out_b, ldo, out_scale, a.chunk,
+                      gate, ldg);
 }
 
 // a step of a few rows (decoding) splits every row's keys over CTAs; longer steps run the tiled kernel.
 // split_ws: kRowsKernelMax * heads * kAttnSplitsMax * (dim + 2) floats; arrived: kRowsKernelMax * heads zeroed counters
 cudaError_t launch_sink_attention(const float* qk, int q_stride, const float* kcache, const float* vcache, const PageMap& pm,
                                   const AttnShape& a, const RowMeta& rm, float* out, void* out_bf16, float* split_ws,
-                                  unsigned* arrived, int M, cudaStream_t st, int ldo, float out_scale) {
+                                  unsigned* arrived, int M, cudaStream_t st, int ldo, float out_scale, const float* gate, int ldg) {
     if (ldo <= 0) ldo = a.heads * a.dim;
     if (a.dim > 32 * kAttnMaxDimPerLane || a.heads % a.kv_heads) return cudaErrorNotSupported;
     __nv_bfloat16* ob = reinterpret_cast<__nv_bfloat16*>(out_bf16);
     if (M > kAttnRowsKernelMax) {
         switch ((a.dim + 63) / 64) {
-            case 1: return launch_attention_tiles<1>(qk, q_stride, kcache, vcache, pm, a, rm, out, ob, ldo, out_scale, M, st);
-            case 2: return launch_attention_tiles<2>(qk, q_stride, kcache, vcache, pm, a, rm, out, ob, ldo, out_scale, M, st);
-            case 3: return launch_attention_tiles<3>(qk, q_stride, kcache, vcache, pm, a, rm, out, ob, ldo, out_scale, M, st);
-            default: return launch_attention_tiles<4>(qk, q_stride, kcache, vcache, pm, a, rm, out, ob, ldo, out_scale, M, st);
+            case 1: return launch_attention_tiles<1>(qk, q_stride, kcache, vcache, pm, a, rm, out, ob, ldo, out_scale, M, st, gate, ldg);
+            case 2: return launch_attention_tiles<2>(qk, q_stride, kcache, vcache, pm, a, rm, out, ob, ldo, out_scale, M, st, gate, ldg);
+            case 3: return launch_attention_tiles<3>(qk, q_stride, kcache, vcache, pm, a, rm, out, ob, ldo, out_scale, M, st, gate, ldg);
+            default: return launch_attention_tiles<4>(qk, q_stride, kcache, vcache, pm, a, rm, out, ob, ldo, out_scale, M, st, gate, ldg);
         }
     }
     const int group = a.heads / a.kv_heads;
-    if (group >= 4) return launch_attention_splits<4>(qk, q_stride, kcache, vcache, pm, a, rm, out, ob, ldo, out_scale, M, split_ws, arrived, st);
-    if (group >= 2) return launch_attention_splits<2>(qk, q_stride, kcache, vcache, pm, a, rm, out, ob, ldo, out_scale, M, split_ws, arrived, st);
-    return launch_attention_splits<1>(qk, q_stride, kcache, vcache, pm, a, rm, out, ob, ldo, out_scale, M, split_ws, arrived, st);
+    if (group >= 4) return launch_attention_splits<4>(qk, q_stride, kcache, vcache, pm, a, rm, out, ob, ldo, out_scale, M, split_ws, arrived, st, gate, ldg);
+    if (group >= 2) return launch_attention_splits<2>(qk, q_stride, kcache, vcache, pm, a, rm, out, ob, ldo, out_scale, M, split_ws, arrived, st, gate, ldg);
+    return launch_attention_splits<1>(qk, q_stride, kcache, vcache, pm, a, rm, out, ob, ldo, out_scale, M, split_ws, arrived, st, gate, ldg);
 }
 
 cudaError_t launch_router_topk(const float* z, int E, int top, int M, int* sel_e, float* sel_w, cudaStream_t st, const float* bias,

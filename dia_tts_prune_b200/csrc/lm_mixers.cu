@@ -21,8 +21,8 @@
 //   gate_prep_kernel          silu(q), the bounded forget gate and biases of the gate-tied recurrence, in place
 //   head_norm_gate_kernel     per-head RMS norm of the read-out (x weight, x gate or its sigmoid / silu), fp32 in place and
 //                             the bf16 operand
-//   xielu_rows_kernel         the dense feed-forward's activation (xIELU or squared relu) on its slice of the stacked
-//                             projections
+//   unit_act_rows_kernel      the activation of a feed-forward that is not gated (xIELU, squared relu or gelu) on its slice
+//                             of the stacked projections
 // talk_attention_kernel also serves attention over cached latent rows (one key/value head whose value rows are the leading
 // channels of its key rows) and takes a window; delta_prep_kernel also serves the delta rule with ONE decay per head;
 // layernorm_rows_kernel also computes the RMS norm.  The recurrences run in lm_scan.cu.
@@ -83,15 +83,13 @@ __global__ void add_rows_kernel(float* __restrict__ x, const float* __restrict__
     for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x) x[i] += y[i];
 }
 
-__global__ void xielu_rows_kernel(const float* __restrict__ proj, int ld, int off, float ap, float an, float* __restrict__ out,
-                                  int ldo, int out_off, __nv_bfloat16* __restrict__ out_b, int F, int relu2) {
+__global__ void unit_act_rows_kernel(const float* __restrict__ proj, int ld, int off, int act, float ap, float an,
+                                     float* __restrict__ out, int ldo, int out_off, __nv_bfloat16* __restrict__ out_b, int F) {
     pdl_release();
     pdl_wait();
     const size_t r = blockIdx.x;
     for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < F; c += gridDim.y * blockDim.x) {
-        const float z = proj[r * ld + off + c];
-        const float y = relu2 ? fmaxf(z, 0.f) * fmaxf(z, 0.f)
-                              : z > 0.f ? fmaf(ap * z, z, 0.5f * z) : fmaf(an, expm1f(z) - z, 0.5f * z);
+        const float y = unit_act(act, proj[r * ld + off + c], ap, an);
         if (out) out[r * ldo + out_off + c] = y;
         if (out_b) out_b[r * ldo + out_off + c] = __float2bfloat16_rn(y);
     }
@@ -101,7 +99,7 @@ __global__ void xielu_rows_kernel(const float* __restrict__ proj, int ld, int of
 // One CTA per row, one warp per q / k head.  q <- rot(rms(q + bias) * qw) * scale in place (the score multiplier rides
 // on q), k likewise without the multiplier into the key pages, v + bias into the value pages, gate <- sigmoid(gate).
 // v_off may be k_off (vdim == dim): the projected key itself, before norm and rotation, is the value.  amp multiplies cosine
-// and sine.
+// and sine.  qw / kw may be null: a norm without weight (which is the same in front of and behind the rotation).
 __global__ void __launch_bounds__(256)
 talk_prep_kernel(float* __restrict__ proj, int ld, const float* __restrict__ bias, int q_off, int k_off, int v_off, int gate_off,
                  int H, int G, int dim, int vdim, const float* __restrict__ qw, const float* __restrict__ kw, float eps,
@@ -137,8 +135,8 @@ talk_prep_kernel(float* __restrict__ proj, int ld, const float* __restrict__ bia
         float* kdst = isq ? nullptr : kcache + (((size_t)page * G + (hh - H)) * page_size + off) * dim;
         for (int i = lane; 2 * i < dim; i += 32) {
             const int c0 = 2 * i, c1 = c0 + 1;
-            float a = (row[base + c0] + (bias ? bias[base + c0] : 0.f)) * inv * nw[c0];
-            float b = c1 < dim ? (row[base + c1] + (bias ? bias[base + c1] : 0.f)) * inv * nw[c1] : 0.f;
+            float a = (row[base + c0] + (bias ? bias[base + c0] : 0.f)) * inv * (nw ? nw[c0] : 1.f);
+            float b = c1 < dim ? (row[base + c1] + (bias ? bias[base + c1] : 0.f)) * inv * (nw ? nw[c1] : 1.f) : 0.f;
             if (c1 < rot_dims) {
                 const float sn = trig[i], cs = trig[n_turn + i];
                 const float ra = a * cs - b * sn, rb = b * cs + a * sn;
@@ -726,10 +724,10 @@ cudaError_t launch_add_rows(float* x, const float* y, int M, int D, cudaStream_t
     return launch_pdl(add_rows_kernel, dim3(blocks), dim3(256), 0, st, x, y, n);
 }
 
-cudaError_t launch_xielu_rows(const float* proj, int ld, int off, float ap, float an, float* out, int ldo, int out_off,
-                              void* out_bf16, int M, int F, cudaStream_t st, bool relu2) {
-    return launch_pdl(xielu_rows_kernel, dim3(M, F > 1024 ? (F + 1023) / 1024 : 1), dim3(256), 0, st, proj, ld, off, ap, an, out,
-                      ldo, out_off, reinterpret_cast<__nv_bfloat16*>(out_bf16), F, relu2 ? 1 : 0);
+cudaError_t launch_unit_act_rows(const float* proj, int ld, int off, int act, float ap, float an, float* out, int ldo, int out_off,
+                                 void* out_bf16, int M, int F, cudaStream_t st) {
+    return launch_pdl(unit_act_rows_kernel, dim3(M, F > 1024 ? (F + 1023) / 1024 : 1), dim3(256), 0, st, proj, ld, off, act, ap, an,
+                      out, ldo, out_off, reinterpret_cast<__nv_bfloat16*>(out_bf16), F);
 }
 
 cudaError_t launch_talk_prep(float* proj, int ld, const float* bias, int q_off, int k_off, int v_off, int gate_off,

@@ -5,8 +5,8 @@
 // sequence state it points at, in an order of operations that does not depend on what else is in the batch.  The
 // streams, norms, latents, scores, gates, running maxima and the recurrent state are fp32.
 //
-//   streams_embed_kernel      token rows of a bf16 table times a constant (optionally through an RMS norm), copied into every
-//                             stream
+//   streams_embed_kernel      token rows of a bf16 table times a constant (optionally with the row of a second table added that
+//                             the pair of the previous token and this one picks, and through an RMS norm), copied into every stream
 //   streams_step_kernel       the write of one sublayer fused with the read of the next:  x_j <- sum_s mix[s][j] x_s +
 //                             out[j] y (y: the sublayer's output, with the weighted sum of a row's expert outputs added),
 //                             then u = sum_s in[s] x_s and h = layernorm(u) w, fp32 and the bf16 GEMM operand.  Without a
@@ -14,7 +14,7 @@
 //                             Options: a second output written with its own weights (a record whose sublayers read the same
 //                             streams), a second norm weight on the same statistics, RMS instead of layer norm, the input
 //                             row for assignments without a slot (identity experts), a sigmoid gate number on y, an RMS norm
-//                             of y before it is written
+//                             of y before it is written (also the norm on a sublayer's output)
 //   latent_prep_kernel        RMS norms of the query latent (in place, + bf16 operand) and of the key/value latent (into
 //                             the pages: the latent is all an attention layer of this kind caches - and, behind it, one
 //                             key part turned with the position where the layer has one)
@@ -44,27 +44,43 @@ namespace lm {
 constexpr int kMaxStreams = 8;
 
 // ---------------------------------------------------------------------------------------------------------------------
+// A row's previous token stands in the row before it (the rows of a sequence are adjacent) or, for the first row its sequence
+// has in the step, at the position before in the sequence's token pages; every row writes its own token there.  A step reads
+// only positions in front of its first row and writes only from there on, so the rows do not race.
 __global__ void streams_embed_kernel(const __nv_bfloat16* __restrict__ table, const int* __restrict__ ids, float scale,
-                                     const float* __restrict__ norm_w, float eps, float* __restrict__ X, int streams, int V, int D) {
+                                     const float* __restrict__ norm_w, float eps, float* __restrict__ X, __nv_bfloat16* __restrict__ Xb,
+                                     int streams, int V, int D, const BigramRows bg) {
     __shared__ float red[32];
     pdl_release();
     pdl_wait();
     const int r = blockIdx.x;
     const int id = ids[r];
     const bool ok = id >= 0 && id < V;
+    const __nv_bfloat16* pair = nullptr;                      // the row of the pair table
+    if (bg.table) {
+        const int pos = bg.rm.pos[r], ps = bg.pm.page_size;
+        const int* pages = bg.pm.table + (size_t)bg.rm.slot[r] * bg.pm.max_pages;
+        const int prev = pos == 0 ? -1 : pos > bg.rm.start[r] ? ids[r - 1] : bg.token_pages[(size_t)pages[(pos - 1) / ps] * ps + (pos - 1) % ps];
+        long long row = pos == 0 ? bg.buckets : -1;
+        if (prev >= 0 && ok) row = ((long long)prev * bg.mul_prev + (long long)id * bg.mul_cur) % bg.buckets;
+        if (row >= 0) pair = reinterpret_cast<const __nv_bfloat16*>(bg.table) + (size_t)row * D;
+        if (threadIdx.x == 0) bg.token_pages[(size_t)pages[pos / ps] * ps + pos % ps] = id;
+    }
+    auto value = [&](int c) { return (ok ? bf(table[(size_t)id * D + c]) * scale : 0.f) + (pair ? bf(pair[c]) : 0.f); };
     float inv = 1.f;
     if (norm_w) {                                             // x / sqrt(mean(x^2) + eps) * w on the scaled row
         float ss = 0.f;
         for (int c = threadIdx.x; c < D; c += blockDim.x) {
-            const float v = ok ? bf(table[(size_t)id * D + c]) * scale : 0.f;
+            const float v = value(c);
             ss = fmaf(v, v, ss);
         }
         inv = 1.0f / sqrtf(block_sum(ss, red) / (float)D + eps);
     }
     for (int c = threadIdx.x; c < D; c += blockDim.x) {
-        float v = ok ? bf(table[(size_t)id * D + c]) * scale : 0.f;
+        float v = value(c);
         if (norm_w) v = v * inv * norm_w[c];
         for (int j = 0; j < streams; ++j) X[((size_t)r * streams + j) * D + c] = v;
+        if (Xb) Xb[(size_t)r * D + c] = __float2bfloat16_rn(v);
     }
 }
 
@@ -173,7 +189,7 @@ streams_step_kernel(float* __restrict__ X, const float* __restrict__ mix, const 
 #pragma unroll
                 for (int e = 0; e < VW; ++e) xs[j][e] = nx[j][e];
         }
-        if (h) {
+        if (h || h_b) {
             float uv[VW];
 #pragma unroll
             for (int e = 0; e < VW; ++e) uv[e] = 0.f;
@@ -187,12 +203,12 @@ streams_step_kernel(float* __restrict__ X, const float* __restrict__ mix, const 
             for (int e = 0; e < VW; ++e) sum += uv[e];
         }
     }
-    if (!h) return;
+    if (!h && !h_b) return;
     if (!norm_w) {                                            // the plain read (every thread re-reads what it wrote itself)
         for (int c = tid * VW; c < D; c += blockDim.x * VW)
 #pragma unroll
             for (int e = 0; e < VW; ++e) {
-                h[(size_t)blockIdx.x * D + c + e] = u_s[c + e];
+                if (h) h[(size_t)blockIdx.x * D + c + e] = u_s[c + e];
                 if (h_b) h_b[(size_t)blockIdx.x * D + c + e] = __float2bfloat16_rn(u_s[c + e]);
             }
         return;
@@ -207,7 +223,7 @@ streams_step_kernel(float* __restrict__ X, const float* __restrict__ mix, const 
     const float inv = 1.0f / sqrtf(block_sum(v, red) / (float)D + eps);
     for (int c = tid; c < D; c += blockDim.x) {
         const float n = (u_s[c] - mean) * inv, o = n * norm_w[c];
-        h[(size_t)blockIdx.x * D + c] = o;
+        if (h) h[(size_t)blockIdx.x * D + c] = o;
         if (h_b) h_b[(size_t)blockIdx.x * D + c] = __float2bfloat16_rn(o);
         if (ex.norm_w2) {                                     // a second weight on the same statistics: the other sublayer's input
             const float o2 = n * ex.norm_w2[c];
@@ -383,14 +399,14 @@ latent_attention_rows_kernel(const float* __restrict__ q, const float* __restric
 }
 
 // ---------------------------------------------------------------------------------------------------------------------
-// Y[m][h N + n] = alpha * sum_k A[m][h K + k] W[h][n][k]  [* sigmoid(gate[m][h N + n])].  64 x 64 x 16 tiles of fp32 FMAs,
-// blockIdx.z = head.
+// Y[m][h N + n] = alpha * sum_k A[m][h K + k] W[h][n][k]  [* sigmoid(gate[m][h N + n]), head_gate: gate[m][h]].  64 x 64 x 16
+// tiles of fp32 FMAs, blockIdx.z = head.
 constexpr int HB = 64, HK = 16;
 
 __global__ void __launch_bounds__(256)
 head_linear_tile_kernel(const float* __restrict__ A, int lda, const __nv_bfloat16* __restrict__ W, float* __restrict__ Y, int ldy,
                         __nv_bfloat16* __restrict__ Yb, int M, int N, int K, float alpha, const float* __restrict__ gate, int ldg,
-                        int a_hs, int y_hs) {
+                        int a_hs, int y_hs, int head_gate) {
     __shared__ __align__(16) float As[HK][HB + 4];
     __shared__ __align__(16) float Bs[HK][HB + 4];
     const int hd = blockIdx.z, m0 = blockIdx.y * HB, n0 = blockIdx.x * HB;
@@ -455,7 +471,7 @@ head_linear_tile_kernel(const float* __restrict__ A, int lda, const __nv_bfloat1
             const int n = n0 + tx * 4 + j;
             if (n >= N) continue;
             float v = acc[i][j] * alpha;
-            if (gate) v *= sigmoidf_(gate[(size_t)m * ldg + (size_t)hd * N + n]);
+            if (gate) v *= sigmoidf_(gate[(size_t)m * ldg + (head_gate ? (size_t)hd : (size_t)hd * N + n)]);
             Y[(size_t)m * ldy + (size_t)hd * y_hs + n] = v;
             if (Yb) Yb[(size_t)m * ldy + (size_t)hd * y_hs + n] = __float2bfloat16_rn(v);
         }
@@ -466,7 +482,7 @@ head_linear_tile_kernel(const float* __restrict__ A, int lda, const __nv_bfloat1
 __global__ void __launch_bounds__(256)
 head_linear_rows_kernel(const float* __restrict__ A, int lda, const __nv_bfloat16* __restrict__ W, float* __restrict__ Y, int ldy,
                         __nv_bfloat16* __restrict__ Yb, int H, int N, int K, float alpha, const float* __restrict__ gate, int ldg,
-                        int a_hs, int y_hs) {
+                        int a_hs, int y_hs, int head_gate) {
     pdl_release();
     const int m = blockIdx.y, lane = threadIdx.x & 31;
     const int col = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
@@ -496,7 +512,7 @@ head_linear_rows_kernel(const float* __restrict__ A, int lda, const __nv_bfloat1
     acc = warp_sum(acc);
     if (lane == 0) {
         float v = acc * alpha;
-        if (gate) v *= sigmoidf_(gate[(size_t)m * ldg + col]);
+        if (gate) v *= sigmoidf_(gate[(size_t)m * ldg + (head_gate ? hd : col)]);
         const size_t at = (size_t)m * ldy + (size_t)hd * y_hs + (col - hd * N);
         Y[at] = v;
         if (Yb) Yb[at] = __float2bfloat16_rn(v);
@@ -582,9 +598,10 @@ mlstm_finish_kernel(const float* __restrict__ raw, int ldr, const float* __restr
 
 // ---- launchers --------------------------------------------------------------------------------------------------------
 cudaError_t launch_streams_embed(const void* table, const int* ids, float scale, float* X, int streams, int M, int V, int D,
-                                 cudaStream_t st, const float* norm_w, float eps) {
+                                 cudaStream_t st, const float* norm_w, float eps, const BigramRows& bg, void* x_bf16) {
+    if ((x_bf16 && streams != 1) || (bg.table && (bg.buckets <= 0 || !bg.token_pages))) return cudaErrorInvalidValue;
     return launch_pdl(streams_embed_kernel, dim3(M), dim3(128), 0, st, reinterpret_cast<const __nv_bfloat16*>(table), ids, scale,
-                      norm_w, eps, X, streams, V, D);
+                      norm_w, eps, X, reinterpret_cast<__nv_bfloat16*>(x_bf16), streams, V, D, bg);
 }
 
 cudaError_t launch_streams_step(float* X, int streams, const StreamWrite& wr, const float* in, const float* norm_w, float eps,
@@ -602,15 +619,15 @@ cudaError_t launch_streams_step(float* X, int streams, const StreamWrite& wr, co
         STREAMS_CASE(5); STREAMS_CASE(6); STREAMS_CASE(7); STREAMS_CASE(8);
 #undef STREAMS_CASE
     }
-    static size_t allowed[2][64] = {};
+    static size_t allowed[kMaxStreams + 1][2][64] = {};      // (every instance is a function of its own)
     if (smem > 48 * 1024) {
         int dev = 0;
         cudaError_t e = cudaGetDevice(&dev);
         if (e != cudaSuccess) return e;
-        if (dev < 0 || dev >= 64 || allowed[vec][dev] < smem) {
+        if (dev < 0 || dev >= 64 || allowed[streams][vec][dev] < smem) {
             e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
             if (e != cudaSuccess) return e;
-            if (dev >= 0 && dev < 64) allowed[vec][dev] = smem;
+            if (dev >= 0 && dev < 64) allowed[streams][vec][dev] = smem;
         }
     }
     return launch_pdl(kernel, dim3(M), dim3(256), smem, st, X, wr.mix, wr.out, wr.y, wr.parts, wr.slot_of, wr.sel_w, wr.top,
@@ -648,17 +665,17 @@ cudaError_t launch_latent_attention_rows(const float* q, const float* pages, con
 }
 
 cudaError_t launch_head_linear(const float* A, int lda, const void* W, float* Y, int ldy, void* y_bf16, int M, int H, int N, int K,
-                               float alpha, const float* gate, int ldg, cudaStream_t st, int a_hs, int y_hs) {
+                               float alpha, const float* gate, int ldg, cudaStream_t st, int a_hs, int y_hs, bool head_gate) {
     const __nv_bfloat16* w = reinterpret_cast<const __nv_bfloat16*>(W);
     __nv_bfloat16* yb = reinterpret_cast<__nv_bfloat16*>(y_bf16);
     if (a_hs <= 0) a_hs = K;                                  // heads adjacent in A and in Y unless strides are given
     if (y_hs <= 0) y_hs = N;
     if (M <= kRowsKernelMax)
         return launch_pdl(head_linear_rows_kernel, dim3((H * N + 7) / 8, M), dim3(256), 0, st, A, lda, w, Y, ldy, yb, H, N, K, alpha,
-                          gate, ldg, a_hs, y_hs);
+                          gate, ldg, a_hs, y_hs, head_gate ? 1 : 0);
     if (H > 65535) return cudaErrorNotSupported;
     head_linear_tile_kernel<<<dim3((N + HB - 1) / HB, (M + HB - 1) / HB, H), 256, 0, st>>>(A, lda, w, Y, ldy, yb, M, N, K, alpha, gate,
-                                                                                          ldg, a_hs, y_hs);
+                                                                                          ldg, a_hs, y_hs, head_gate ? 1 : 0);
     return cudaGetLastError();
 }
 

@@ -1,5 +1,5 @@
 """Configuration schemas of the decoder-only language models (``config.json`` of a model folder): Pubopel, Kupelix,
-Luketar, Fipadra and Loduzen.
+Luketar, Fipadra, Loduzen and Forilorn.
 
 Every size and every per-model constant comes from the file.  Optional entries that are absent switch their
 mechanism off: no ``mask`` is full causal attention, no ``softcap`` leaves scores uncapped, ``mlp: null`` is a layer
@@ -494,8 +494,77 @@ class LoduzenConfig(BaseModel, frozen=True):
                 raise ValueError(f"layer {i}: rot.dims ({a.rot.dims}) must be even and at most dim ({a.dim})")
 
 
+# ---- Forilorn: norms on the sublayers' outputs only; attention inside chunks on its own keys / rotary latent attention in a window;
+# ---- a gelu dense unit; a pair table beside the embedding
+class ChunkConfig(BaseModel, frozen=True):
+    size: int = Field(gt=0)                      # position i sees j <= i of its own block of `size` positions
+
+
+class ChunkAttentionConfig(BaseModel, frozen=True):
+    heads: int = Field(gt=0)
+    kv_heads: Optional[int] = Field(default=None, gt=0)
+    dim: int = Field(gt=0)
+    vdim: int = Field(gt=0)
+    scale: float
+    rot: Optional[RotConfig] = None
+    mask: Optional[ChunkConfig] = None
+
+
+class ForilornAttentionLayer(BaseModel, frozen=True):
+    type: Literal["attention"]
+    mixer: ChunkAttentionConfig
+    mlp: Optional[DenseMlpConfig] = None
+
+
+class ForilornLatentLayer(BaseModel, frozen=True):
+    type: Literal["latent_attention"]
+    mixer: RotaryLatentMixerConfig
+    mlp: Optional[DenseMlpConfig] = None
+
+
+ForilornLayer = Annotated[Union[ForilornAttentionLayer, ForilornLatentLayer], Field(discriminator="type")]
+
+
+class BigramConfig(BaseModel, frozen=True):
+    buckets: int = Field(gt=0)                   # the table has one more row, for a sequence's first token
+    mul_prev: int = Field(ge=0)
+    mul_cur: int = Field(ge=0)
+
+
+class BigramEmbeddingConfig(BaseModel, frozen=True):
+    scale: float = 1.0
+    bigram: Optional[BigramConfig] = None
+
+
+class ForilornConfig(BaseModel, frozen=True):
+    architecture: Literal["Forilorn"] = "Forilorn"
+    vocab: int = Field(gt=0)
+    width: int = Field(gt=0)
+    layers: list[ForilornLayer] = Field(min_length=1)
+    norm: NormConfig
+    embedding: BigramEmbeddingConfig = BigramEmbeddingConfig()
+    residual_mult: float = 1.0
+
+    @classmethod
+    def load(cls, path: str | Path) -> "ForilornConfig":
+        return cls.model_validate(json.loads(Path(path).read_text(encoding="utf-8")))
+
+    def check(self) -> None:
+        for i, layer in enumerate(self.layers):
+            m = layer.mixer
+            if layer.type == "attention":
+                g = m.kv_heads or m.heads
+                if m.heads % g:
+                    raise ValueError(f"layer {i}: heads ({m.heads}) must be a multiple of kv_heads ({g})")
+                if m.vdim != m.dim:
+                    raise ValueError(f"layer {i}: the values are the projected keys, so vdim ({m.vdim}) must equal dim ({m.dim})")
+            turning = m.rot_dim if layer.type == "latent_attention" else m.dim
+            if m.rot is not None and (m.rot.dims % 2 or m.rot.dims > turning):
+                raise ValueError(f"layer {i}: rot.dims ({m.rot.dims}) must be even and at most {turning}")
+
+
 CONFIGS = {"pubopel": PubopelConfig, "kupelix": KupelixConfig, "luketar": LuketarConfig, "fipadra": FipadraConfig,
-           "loduzen": LoduzenConfig}
+           "loduzen": LoduzenConfig, "forilorn": ForilornConfig}
 
 
 def load_config(raw: dict):

@@ -13,7 +13,7 @@ import numpy as np
 import torch
 
 from . import _lm_lib
-from .lm_layers import DynamicTanh, LayerNorm, MixLayer, RmsNorm
+from .lm_layers import BigramEmbedding, DynamicTanh, LayerNorm, MixLayer, RmsNorm
 from .lm_state import PagedState, Sequence
 
 
@@ -29,9 +29,10 @@ class LMEngine:
     def __init__(self, layers: list, embed: torch.Tensor, head: torch.Tensor, final_norm: DynamicTanh | LayerNorm | RmsNorm, *,
                  width: int, vocab: int, taps: int, eps: float, state: PagedState, max_rows: int = 1024,
                  precision: str = "bfloat16", step_graphs: bool = True, logit_scale: float = 1.0, embed_scale: float = 1.0,
-                 embed_norm: torch.Tensor | None = None):
+                 embed_norm: torch.Tensor | None = None, bigram: BigramEmbedding | None = None):
         """``layers``: the layer records in execution order (a layer that runs twice per token appears twice, each time
-        with the state record of its own index)."""
+        with the state record of its own index).  ``bigram``: a pair table added to the embedding rows (stream records; the
+        state keeps the tokens)."""
         if not torch.cuda.is_available():
             raise RuntimeError("the language-model path needs a CUDA device (sm_100a); there is no CPU fallback")
         self.lib = _lm_lib.load()
@@ -62,6 +63,11 @@ class LMEngine:
         # an RMS norm weight on the embedding rows (stream records only)
         self.embed_norm = None if embed_norm is None else embed_norm.detach().to(device=self.device, dtype=torch.float32).contiguous()
         m.embed_norm = self.embed_norm.data_ptr() if self.embed_norm is not None else None
+        self.bigram = bigram
+        if bigram is not None:
+            if state.token_pages is None or tuple(bigram.table.shape) != (bigram.buckets + 1, self.width):
+                raise ValueError("a pair table needs kept tokens and one row per bucket and one more")
+            bigram.fill(m, state)
         recs = (_lm_lib.Layer * len(layers))()
         for i, layer in enumerate(layers):
             layer.fill(recs[i], state.record_state(i))

@@ -32,7 +32,6 @@ Beside ``layers.py`` (Dia's RMSNorm / rotary attention / gated MLP modules) this
     denominator;
   * options of :class:`LatentAttention`: a turned key part shared by all heads behind the cached latent (the query heads
     carry a turned part of their own), a sliding window, no sink, no gate;
-  * :class:`DenseRelu2` - up projection, squared relu, down projection;
   * options of :class:`RoutedExperts`: scores from the softmax over ALL router outputs, a correction that only the choice
     sees, choice inside the best groups of neighbouring outputs, normalised and scaled weights, identity experts, a
     sigmoid gate number on the shared unit;
@@ -43,7 +42,13 @@ Beside ``layers.py`` (Dia's RMSNorm / rotary attention / gated MLP modules) this
     skip term, the gate before a grouped norm;
   * :class:`PairMixer` - any two mixers of the stream form side by side on one input, their outputs weighted and added;
   * ``GatedUnit(act="gelu")`` - the tanh form of gelu on the gate branch;
-  * :class:`TokenInput` - what a layer adds for the token itself: a gated slice of a second embedding table, normed.
+  * :class:`TokenInput` - what a layer adds for the token itself: a gated slice of a second embedding table, normed;
+  * :class:`BigramEmbedding` - a second embedding table whose row the previous token and this one pick together;
+  * options of :class:`RotaryAttention`: no weights on the q / k norms, keys of the query's own chunk only, an elementwise
+    sigmoid output gate; of :class:`LatentAttention`: one gate number per head; of :class:`RmsNorm`: a weight stored as its
+    distance from one;
+  * :class:`DenseUnit` - up projection, squared relu or the tanh form of gelu, down projection;
+  * ``StreamLayer(None, ..., norm1_out=...)`` - sublayers that read the residual stream itself and whose outputs are normed.
 All constants are constructor arguments; a design picks and combines them per layer (:class:`MixLayer` runs its
 sublayers one after the other, :class:`ParallelLayer` feeds one norm to mixer and feed-forward and adds both,
 :class:`StreamLayer` runs pre-norm sublayers over hyper-connected streams - with ``parallel`` both sublayers read the
@@ -420,8 +425,9 @@ class HyperConnection:
         self.w_in, self.w_out, self.w_mix = _f32(w_in, device), _f32(w_out, device), _f32(w_mix, device)
 
     @classmethod
-    def residual(cls, device) -> "HyperConnection":
-        return cls(torch.ones(1), torch.ones(1), torch.ones((1, 1)), device)
+    def residual(cls, device, mult: float = 1.0) -> "HyperConnection":
+        """x <- x + mult y."""
+        return cls(torch.ones(1), torch.full((1,), float(mult), dtype=torch.float64), torch.ones((1, 1)), device)
 
 
 class LatentAttention:
@@ -429,18 +435,19 @@ class LatentAttention:
 
     def __init__(self, w_dq, q_lat_norm, w_uq, w_dkv, kv_lat_norm, w_uk, w_uv, w_gate, w_o, *, heads: int, dim: int, vdim: int,
                  scale: float, sink=None, device=None, rot_dim: int = 0, rot_angles=None, rot_half: bool = False,
-                 window: int | None = None):
+                 window: int | None = None, head_gate: bool = False):
         """``rot_dim`` > 0: every query head is ``[dim plain | rot_dim turned]`` (``w_uq`` has heads x (dim + rot_dim) rows) and
         ``w_dkv`` has ``rot_dim`` more rows behind the latent's: one turned key part for all heads, cached beside the
         latent.  ``rot_angles``: angle per position of the turning pairs (the first 2 x len channels of the turned part).
-        ``window``: a position sees itself and the ``window - 1`` before it.  ``w_gate`` None: no output gate."""
+        ``window``: a position sees itself and the ``window - 1`` before it.  ``w_gate`` None: no output gate; ``head_gate``: it
+        has one row per head (otherwise one per output channel)."""
         self.heads, self.dim, self.vdim, self.scale = int(heads), int(dim), int(vdim), float(scale)
         self.rot_dim, self.rot_half, self.window = int(rot_dim), bool(rot_half), int(window) if window else 0
         self.q_rank, self.kv_rank = int(w_dq.shape[0]), int(w_dkv.shape[0]) - self.rot_dim
         if (tuple(w_uq.shape) != (heads * (dim + self.rot_dim), self.q_rank) or tuple(w_uk.shape) != (heads * dim, self.kv_rank)
-                or tuple(w_uv.shape) != (heads * vdim, self.kv_rank) or (w_gate is not None and tuple(w_gate.shape)[0] != heads * vdim)):
+                or tuple(w_uv.shape) != (heads * vdim, self.kv_rank) or (w_gate is not None and tuple(w_gate.shape)[0] != (heads if head_gate else heads * vdim))):
             raise ValueError("projection shapes do not match heads x dim and the latent sizes")
-        self.gated = w_gate is not None
+        self.gated, self.head_gate = w_gate is not None, bool(head_gate)
         self.in_rows, self.in_bias, self.w_o = [w_dq, w_dkv] + ([w_gate] if self.gated else []), None, w_o
         self.rot = None if rot_angles is None or rot_angles.numel() == 0 else _f32(rot_angles, device)
         if self.rot is not None and 2 * self.rot.numel() > self.rot_dim:
@@ -456,9 +463,9 @@ class LatentAttention:
         return StateSpec(latent=self.kv_rank + self.rot_dim)
 
     def fill(self, rec, st) -> None:
-        from ._lm_lib import GATE_NONE, GATE_SIGMOID, MIXER_LATENT_ATTENTION, ROT_HALF, ROT_INTERLEAVED
+        from ._lm_lib import GATE_NONE, GATE_SIGMOID, GATE_SIGMOID_HEAD, MIXER_LATENT_ATTENTION, ROT_HALF, ROT_INTERLEAVED
         rec.mixer = MIXER_LATENT_ATTENTION
-        rec.mixer_gate = GATE_SIGMOID if self.gated else GATE_NONE
+        rec.mixer_gate = (GATE_SIGMOID_HEAD if self.head_gate else GATE_SIGMOID) if self.gated else GATE_NONE
         rec.rot_dim, rec.window = self.rot_dim, self.window
         rec.rot_dims = 2 * self.rot.numel() if self.rot is not None else 0
         rec.rot_freq = self.rot.data_ptr() if self.rot is not None else None
@@ -577,16 +584,20 @@ class RotaryAttention:
     kind = "rotary_attention"
 
     def __init__(self, w_q, w_k, w_v, w_o, q_norm, k_norm, *, heads: int, kv_heads: int, dim: int, scale: float, rot_angles=None,
-                 rot_amp: float = 1.0, window: int | None = None, sink=None, device=None):
+                 rot_amp: float = 1.0, window: int | None = None, sink=None, device=None, w_gate=None, chunk: int | None = None):
         """``w_v`` None: the values are the projected keys, before norm and rotation.  ``sink [heads]``: logits that join the
-        softmax's denominator only.  ``rot_amp`` multiplies cosine and sine."""
+        softmax's denominator only.  ``rot_amp`` multiplies cosine and sine.  ``q_norm`` / ``k_norm`` None: the norm has no weight
+        (it then gives the same in front of and behind the rotation).  ``chunk``: a position sees only the keys of its own block of
+        ``chunk`` positions, counted from the sequence's start.  ``w_gate [heads * dim, width]``: the heads' outputs are multiplied
+        by the sigmoid of this projection."""
         self.heads, self.kv_heads, self.dim, self.vdim, self.scale = int(heads), int(kv_heads), int(dim), int(dim), float(scale)
         if (tuple(w_q.shape)[0] != heads * dim or tuple(w_k.shape)[0] != kv_heads * dim or heads % kv_heads
-                or (w_v is not None and tuple(w_v.shape)[0] != kv_heads * dim)):
+                or (w_v is not None and tuple(w_v.shape)[0] != kv_heads * dim)
+                or (w_gate is not None and tuple(w_gate.shape)[0] != heads * dim)):
             raise ValueError("projection shapes do not match heads x dim")
-        self.own_values = w_v is not None
-        self.in_rows, self.in_bias, self.w_o = [w_q, w_k] + ([w_v] if self.own_values else []), None, w_o
-        self.q_norm, self.k_norm = _f32(q_norm, device), _f32(k_norm, device)
+        self.own_values, self.gated, self.chunk = w_v is not None, w_gate is not None, int(chunk) if chunk else 0
+        self.in_rows, self.in_bias, self.w_o = [w_q, w_k] + ([w_v] if self.own_values else []) + ([w_gate] if self.gated else []), None, w_o
+        self.q_norm, self.k_norm = (None if n is None else _f32(n, device) for n in (q_norm, k_norm))
         self.rot = None if rot_angles is None or rot_angles.numel() == 0 else _f32(rot_angles, device)
         self.rot_amp, self.window = float(rot_amp), int(window) if window else 0
         self.sink = None if sink is None else _f32(sink, device)
@@ -595,11 +606,12 @@ class RotaryAttention:
         return StateSpec(kv=(self.kv_heads, self.dim, self.dim))
 
     def fill(self, rec, st) -> None:
-        from ._lm_lib import GATE_NONE, MIXER_ROTARY_ATTENTION, ROT_INTERLEAVED
-        rec.mixer, rec.mixer_gate = MIXER_ROTARY_ATTENTION, GATE_NONE
+        from ._lm_lib import GATE_NONE, GATE_SIGMOID, MIXER_ROTARY_ATTENTION, ROT_INTERLEAVED
+        rec.mixer, rec.mixer_gate = MIXER_ROTARY_ATTENTION, GATE_SIGMOID if self.gated else GATE_NONE
         rec.heads, rec.kv_heads, rec.dim, rec.vdim, rec.scale = self.heads, self.kv_heads, self.dim, self.vdim, self.scale
-        rec.values_are_keys, rec.window = 0 if self.own_values else 1, self.window
-        rec.q_norm, rec.k_norm = self.q_norm.data_ptr(), self.k_norm.data_ptr()
+        rec.values_are_keys, rec.window, rec.chunk = 0 if self.own_values else 1, self.window, self.chunk
+        rec.q_norm = self.q_norm.data_ptr() if self.q_norm is not None else None
+        rec.k_norm = self.k_norm.data_ptr() if self.k_norm is not None else None
         rec.rot_dims = 2 * self.rot.numel() if self.rot is not None else 0
         rec.rot_freq = self.rot.data_ptr() if self.rot is not None else None
         rec.rot_layout, rec.rot_amp = ROT_INTERLEAVED, self.rot_amp
@@ -725,16 +737,32 @@ class TokenInput:
         rec.side_norm = self.norm.data_ptr()
 
 
-class DenseRelu2:
-    def __init__(self, w_up, w_down, device=None):
-        """``down(max(up h, 0)^2)``."""
-        self.ff = int(w_up.shape[0])
+class BigramEmbedding:
+    def __init__(self, table: torch.Tensor, *, buckets: int, mul_prev: int, mul_cur: int, device=None):
+        """``table [buckets + 1, width]``: row (previous x ``mul_prev`` + token x ``mul_cur``) mod ``buckets`` joins the token's
+        embedding row; the last row stands for a sequence's first token."""
+        self.table, self.buckets = _bf16(table, device), int(buckets)
+        self.mul_prev, self.mul_cur = int(mul_prev) % self.buckets, int(mul_cur) % self.buckets     # the same rows, no overflow
+
+    def fill(self, model, state) -> None:
+        model.bigram, model.bigram_buckets = self.table.data_ptr(), self.buckets
+        model.bigram_mul_prev, model.bigram_mul_cur = self.mul_prev, self.mul_cur
+        model.token_pages = state.token_pages.data_ptr()
+
+
+class DenseUnit:
+    def __init__(self, w_up, w_down, *, act: str, device=None):
+        """``down(act(up h))`` with ``act`` ``relu2`` (max(z, 0)^2) or ``gelu`` (the tanh form)."""
+        if act not in ("relu2", "gelu"):
+            raise ValueError("act must be 'relu2' or 'gelu'")
+        self.act, self.ff = act, int(w_up.shape[0])
         self.w_up, self.w_down = _bf16(w_up, device), _bf16(w_down, device)
 
 
 class RmsNorm:
-    def __init__(self, weight: torch.Tensor, device):
-        self.w = _f32(weight, device)
+    def __init__(self, weight: torch.Tensor, device, around_one: bool = False):
+        """``around_one``: the stored weight is the distance from one."""
+        self.w = _f32(weight.detach().to(torch.float32) + 1.0 if around_one else weight, device)
 
     def fill(self, rec) -> None:
         from ._lm_lib import NORM_RMS
@@ -758,15 +786,22 @@ class StreamLayer:
     with another layer's weights): each record gets a state of its own."""
 
     def __init__(self, norm1, hc1: HyperConnection, mixer, ff=None, norm2=None, hc2: HyperConnection | None = None, device=None,
-                 parallel: bool = False, rms: bool = False, side: TokenInput | None = None):
-        """``parallel``: the feed-forward reads the streams as they were before the mixer's write, and both outputs are
+                 parallel: bool = False, rms: bool = False, side: TokenInput | None = None, norm1_out: RmsNorm | None = None,
+                 norm2_out: RmsNorm | None = None):
+        """``norm1`` None (one stream): the sublayers read the stream itself, and ``norm1_out`` / ``norm2_out`` norm what they give
+        back: x += hc1.out norm1_out(mixer(x)), x += hc2.out norm2_out(ff(x)).  ``parallel``: the feed-forward reads the streams as they were before the mixer's write, and both outputs are
         written at once (with one stream: x += mixer(norm1 x) + ff(norm2 x)).  ``rms``: the norms are RMS norms.  ``side``: a
         token input after the feed-forward (one stream)."""
         self.mixer, self.ff, self.hc1, self.hc2 = mixer, ff, hc1, hc2
         self.parallel, self.rms = bool(parallel), bool(rms)
-        self.norm1 = _f32(norm1, device)
+        self.norm1 = None if norm1 is None else _f32(norm1, device)
         self.norm2 = None if norm2 is None else _f32(norm2, device)
-        if ff is not None and (norm2 is None or hc2 is None or hc2.streams != hc1.streams):
+        self.norm1_out, self.norm2_out = norm1_out, norm2_out
+        if norm1 is None and (hc1.streams != 1 or parallel or norm2 is not None):
+            raise ValueError("sublayers without input norms need one residual stream, one after the other")
+        if norm1 is not None and (norm1_out is not None or norm2_out is not None):
+            raise ValueError("norms on the outputs stand in records without input norms")
+        if ff is not None and ((norm2 is None and norm1 is not None) or hc2 is None or hc2.streams != hc1.streams):
             raise ValueError("a feed-forward sublayer needs its norm and hyper-connection weights")
         self.side = side
         if side is not None and hc1.streams != 1:
@@ -779,11 +814,15 @@ class StreamLayer:
         return self.mixer.state_spec()
 
     def fill(self, rec, st) -> None:
-        from ._lm_lib import (ACT_CLAMPED_GLU, ACT_GELU_GLU, ACT_RELU2, ACT_SILU_GLU, FF_DENSE, FF_NONE, FF_ROUTED_EXPERTS, FORM_STREAMS,
+        from ._lm_lib import (ACT_CLAMPED_GLU, ACT_GELU, ACT_GELU_GLU, ACT_RELU2, ACT_SILU_GLU, FF_DENSE, FF_NONE, FF_ROUTED_EXPERTS, FORM_STREAMS,
                               NORM_LAYER, NORM_RMS, ROUTER_SIGMOID_INPUT, ROUTER_SOFTMAX_GROUPED, ROUTER_SOFTMAX_TOP)
         norm_kind = NORM_RMS if self.rms else NORM_LAYER
         rec.form, rec.streams, rec.parallel = FORM_STREAMS, self.hc1.streams, 1 if self.parallel else 0
-        rec.norm_mix_in.w, rec.norm_mix_in.b, rec.norm_mix_in.kind = self.norm1.data_ptr(), None, norm_kind
+        if self.norm1 is not None:
+            rec.norm_mix_in.w, rec.norm_mix_in.b, rec.norm_mix_in.kind = self.norm1.data_ptr(), None, norm_kind
+        for norm, dst in ((self.norm1_out, rec.norm_mix_out), (self.norm2_out, rec.norm_ff_out)):
+            if norm is not None:
+                norm.fill(dst)
         for q, hc in enumerate((self.hc1, self.hc2)):
             if hc is not None:
                 rec.hc_in[q], rec.hc_out[q], rec.hc_mix[q] = hc.w_in.data_ptr(), hc.w_out.data_ptr(), hc.w_mix.data_ptr()
@@ -796,9 +835,10 @@ class StreamLayer:
         f = self.ff
         if f is None:
             return
-        rec.norm_ff_in.w, rec.norm_ff_in.b, rec.norm_ff_in.kind = self.norm2.data_ptr(), None, norm_kind
-        if isinstance(f, DenseRelu2):
-            rec.ff, rec.dense_ff, rec.act = FF_DENSE, f.ff, ACT_RELU2
+        if self.norm2 is not None:
+            rec.norm_ff_in.w, rec.norm_ff_in.b, rec.norm_ff_in.kind = self.norm2.data_ptr(), None, norm_kind
+        if isinstance(f, DenseUnit):
+            rec.ff, rec.dense_ff, rec.act = FF_DENSE, f.ff, ACT_GELU if f.act == "gelu" else ACT_RELU2
             rec.ws_gate_up, rec.ws_down = f.w_up.data_ptr(), f.w_down.data_ptr()
             return
         rec.act = ACT_CLAMPED_GLU if f.limit is not None else ACT_SILU_GLU

@@ -18,9 +18,9 @@ from pathlib import Path
 import torch
 
 from .checkpoint import load_safetensors
-from .lm_config import FipadraConfig, KupelixConfig, LoduzenConfig, LuketarConfig, PubopelConfig, load_config
+from .lm_config import FipadraConfig, ForilornConfig, KupelixConfig, LoduzenConfig, LuketarConfig, PubopelConfig, load_config
 from .lm_engine import LMEngine
-from .lm_layers import (ChannelDelta, DenseRelu2, DenseXielu, DynamicTanh, GatedDelta, GatedLinear, GatedUnit, Hgrn2,
+from .lm_layers import (BigramEmbedding, ChannelDelta, DenseUnit, DenseXielu, DynamicTanh, GatedDelta, GatedLinear, GatedUnit, Hgrn2,
                         HyperConnection, LatentAttention, LayerNorm, LayerRun, Mamba2, MixLayer, MLstm, PairMixer, ParallelLayer,
                         Retention, RmsNorm, RotaryAttention, RoutedExperts, SinkAttention, StreamLayer, TalkingAttention, TapMix,
                         TokenInput, rotary_angles, yarn_angles)
@@ -161,7 +161,7 @@ def build_fipadra_layers(cfg: FipadraConfig, w: dict[str, torch.Tensor], device)
         if f is not None:
             norm2 = w[f"l{i}.norm2"]
             if f.kind == "dense":
-                ff = DenseRelu2(w[q + "up"], w[q + "down"], device=device)
+                ff = DenseUnit(w[q + "up"], w[q + "down"], act="relu2", device=device)
             else:
                 E, r = f.router.experts, f.router
                 shared = (w[q + "shared.gate"], w[q + "shared.up"], w[q + "shared.down"]) if f.shared is not None else None
@@ -212,6 +212,33 @@ def build_loduzen_layers(cfg: LoduzenConfig, w: dict[str, torch.Tensor], device)
         layers.append(StreamLayer(w[f"l{i}.norm1"], residual, mixer, ff, norm2, residual if ff is not None else None, device=device,
                                   rms=True, side=side))
     return layers, RmsNorm(w["final.norm"], device)
+
+
+def build_forilorn_layers(cfg: ForilornConfig, w: dict[str, torch.Tensor], device) -> tuple[list[StreamLayer], RmsNorm]:
+    """The layer records of a Forilorn checkpoint (tensor names ``l<i>.norm1``, ``l<i>.mix.q``, ``l<i>.mix.dkv.norm``,
+    ``l<i>.mlp.up`` ...): stream records with one residual stream that the sublayers read as it is; their outputs are RMS-normed
+    (weights stored as the distance from one) and added times the residual multiplier."""
+    residual = HyperConnection.residual(device, cfg.residual_mult)
+    layers = []
+    for i, lc in enumerate(cfg.layers):
+        p, m = f"l{i}.mix.", lc.mixer
+        t = lambda name: w[p + name]                             # noqa: E731
+        angles = rotary_angles(m.rot.base, m.rot.dims, m.rot.scaling) if m.rot is not None and m.rot.dims > 0 else None
+        size = m.mask.size if m.mask is not None else None
+        if lc.type == "attention":
+            mixer = RotaryAttention(t("q"), t("k"), None, t("o"), None, None, heads=m.heads, kv_heads=m.kv_heads or m.heads,
+                                    dim=m.dim, scale=m.scale, rot_angles=angles, chunk=size, w_gate=t("g"), device=device)
+        else:
+            mixer = LatentAttention(t("dq"), t("dq.norm"), t("uq"), t("dkv"), t("dkv.norm"), t("uk"), t("uv"), t("g"), t("o"),
+                                    heads=m.heads, dim=m.dim, vdim=m.vdim, scale=m.scale, sink=None, rot_dim=m.rot_dim,
+                                    rot_angles=angles, rot_half=False, window=size, head_gate=True, device=device)
+        ff = out2 = None
+        if lc.mlp is not None:
+            ff = DenseUnit(w[f"l{i}.mlp.up"], w[f"l{i}.mlp.down"], act="gelu", device=device)
+            out2 = RmsNorm(w[f"l{i}.norm2"], device, around_one=True)
+        layers.append(StreamLayer(None, residual, mixer, ff, None, residual if ff is not None else None, device=device, rms=True,
+                                  norm1_out=RmsNorm(w[f"l{i}.norm1"], device, around_one=True), norm2_out=out2))
+    return layers, RmsNorm(w["final.norm"], device, around_one=True)
 
 
 @dataclass
@@ -300,7 +327,7 @@ class Scheduler:
 
 
 class CausalLM:
-    def __init__(self, cfg: PubopelConfig | KupelixConfig | LuketarConfig | FipadraConfig | LoduzenConfig,
+    def __init__(self, cfg: PubopelConfig | KupelixConfig | LuketarConfig | FipadraConfig | LoduzenConfig | ForilornConfig,
                  weights: dict[str, torch.Tensor], dtype: str = "bfloat16", device=None, max_tokens: int = 4096, max_sequences: int = 8, page_size: int = 16, max_rows: int = 1024,
                  max_sequence_tokens: int | None = None, step_graphs: bool = True):
         if dtype not in ("bfloat16", "float32"):
@@ -311,7 +338,7 @@ class CausalLM:
         self.config, self.dtype = cfg, dtype
         self.device = torch.device(device) if device is not None else torch.device("cuda", torch.cuda.current_device())
         # a design is its layer records (in execution order), its final norm and the constants around them
-        embed_scale, head, embed_norm = 1.0, weights.get("head"), None
+        embed_scale, head, embed_norm, bigram = 1.0, weights.get("head"), None, None
         if isinstance(cfg, FipadraConfig):
             self.layers, final_norm = build_fipadra_layers(cfg, weights, self.device)
             taps, logit_scale = 0, cfg.logit_scale
@@ -319,6 +346,13 @@ class CausalLM:
         elif isinstance(cfg, LoduzenConfig):
             self.layers, final_norm = build_loduzen_layers(cfg, weights, self.device)
             taps, logit_scale, head = 0, 1.0, weights["embed"]    # logits against the table itself
+        elif isinstance(cfg, ForilornConfig):
+            self.layers, final_norm = build_forilorn_layers(cfg, weights, self.device)
+            taps, logit_scale, embed_scale = 0, 1.0, cfg.embedding.scale
+            head = weights["embed"]                             # the table itself, without the embedding's scale
+            if cfg.embedding.bigram is not None:
+                b = cfg.embedding.bigram
+                bigram = BigramEmbedding(weights["bigram"], buckets=b.buckets, mul_prev=b.mul_prev, mul_cur=b.mul_cur, device=self.device)
         elif isinstance(cfg, KupelixConfig):
             self.layers, final_norm = build_kupelix_layers(cfg, weights, self.device)
             taps, logit_scale = 0, cfg.logit_scale
@@ -330,13 +364,15 @@ class CausalLM:
             self.layers, final_norm = build_pubopel_layers(cfg, weights, self.device)
             taps, logit_scale = cfg.canon.taps, 1.0
         self.state = PagedState([layer.state_spec() for layer in self.layers], cfg.width, taps, max_tokens, self.device,
-                                page_size=page_size, max_sequences=max_sequences, max_sequence_tokens=max_sequence_tokens)
+                                page_size=page_size, max_sequences=max_sequences, max_sequence_tokens=max_sequence_tokens,
+                                keep_tokens=bigram is not None)
         # float32: every product is fp32 arithmetic on the stored (bfloat16) weights.  bfloat16: the products of prompt
         # portions run on the tensor cores with bfloat16 operands and fp32 accumulation.  Norms, scores, the router, the
         # pages, recurrent states and the residual stream are float32 in both.
         self.engine = LMEngine(self.layers, weights["embed"], head, final_norm, width=cfg.width, vocab=cfg.vocab,
                                taps=taps, eps=cfg.norm.eps, state=self.state, max_rows=max_rows, precision=dtype,
-                               step_graphs=step_graphs, logit_scale=logit_scale, embed_scale=embed_scale, embed_norm=embed_norm)
+                               step_graphs=step_graphs, logit_scale=logit_scale, embed_scale=embed_scale, embed_norm=embed_norm,
+                               bigram=bigram)
         self._draws = 0
 
     @classmethod

@@ -7,7 +7,8 @@ and of every recurrent layer's state) and a list of fixed-size *pages* of the sh
 crosses a page border and given back when it ends.  Slots and pages are recycled last-freed-first; nothing is cleared
 on reuse, because the kernels take a sequence's state as zero when its first row of a step is position 0.  What a layer
 record keeps is described by a :class:`StateSpec`; a layer that runs several times per token has one record, and so
-one state, per run.  The kernels read the device copy of the page table; the bookkeeping is host-side and never reads
+one state, per run.  A model whose embedding looks at earlier tokens keeps every sequence's token ids in pages of their own
+on the same page table (``token_pages``).  The kernels read the device copy of the page table; the bookkeeping is host-side and never reads
 a device tensor.
 """
 
@@ -57,10 +58,11 @@ class RecordState:
 
 class PagedState:
     def __init__(self, layers: list, width: int, taps: int, max_tokens: int, device: torch.device,
-                 page_size: int = 16, max_sequences: int = 8, max_sequence_tokens: int | None = None):
+                 page_size: int = 16, max_sequences: int = 8, max_sequence_tokens: int | None = None, keep_tokens: bool = False):
         """``layers``: a :class:`StateSpec` per layer record, or ``(kv_heads, dim)`` for a record with keys and values of
         one size and two tap-mix tails.  ``max_tokens``: the most tokens all live sequences hold at one time; the pool gets
-        that many tokens' worth of pages plus one partly filled page per slot."""
+        that many tokens' worth of pages plus one partly filled page per slot.  ``keep_tokens``: the sequences' token ids are
+        part of the state."""
         if page_size <= 0 or max_tokens <= 0 or max_sequences <= 0:
             raise ValueError("page_size, max_tokens and max_sequences must be positive")
         self.device = torch.device(device)
@@ -77,6 +79,7 @@ class PagedState:
         self.tails, self.conv_tails = [r.tails for r in self.records], [r.conv_tail for r in self.records]
         self.rec_states, self.rec_aux = [r.rec_state for r in self.records], [r.rec_aux for r in self.records]
         self.latent_pages = [r.latent_pages for r in self.records]
+        self.token_pages = torch.zeros((self.n_pages, self.page_size), dtype=torch.int32, device=self.device) if keep_tokens else None
         self._table_host = torch.zeros((self.n_slots, self.max_pages), dtype=torch.int32).pin_memory() \
             if self.device.type == "cuda" else torch.zeros((self.n_slots, self.max_pages), dtype=torch.int32)
         self.page_table = torch.zeros((self.n_slots, self.max_pages), dtype=torch.int32, device=self.device)

@@ -57,6 +57,7 @@ def _ensure_builtin() -> None:
     register("Luketar", _load_causal_lm)
     register("Fipadra", _load_causal_lm)
     register("Loduzen", _load_causal_lm)
+    register("Forilorn", _load_causal_lm)
 
 
 def load_model(folder: str | Path, dtype: str = "bfloat16", device=None, **kw):

@@ -11,6 +11,8 @@
  *               u = sum_s in[s] x_s;  y = sublayer(norm(u));  x_j <- sum_s mix[s][j] x_s + out[j] y   (hyper-connections;
  *               s = 1 with unit weights is the plain pre-norm residual)
  *               with `parallel`, both sublayers read the streams before either writes: x += mixer(norm1(x)) + ff(norm2(x))
+ *               a record without input norms and with one stream reads x itself, and may norm the sublayers' OUTPUTS instead:
+ *               x += out[0] norm_a(mixer(x));  x += out[0]' norm_b(ff(x))
  * and the mechanisms (norm kind, mixer kind, feed-forward kind) are selected and parameterised per record, so a design
  * combines them as it needs.  A layer that a design runs several times with the same weights is several records that
  * share weight pointers and differ in their state pointers.  Matrices are bf16 [out][in]; vectors and scalars fp32.
@@ -33,7 +35,7 @@
 extern "C" {
 #endif
 
-#define LM_B200_ABI_VERSION 5
+#define LM_B200_ABI_VERSION 6
 
 enum lm_b200_status { LM_B200_OK = 0, LM_B200_EINVAL = -1, LM_B200_ECUDA = -2, LM_B200_ENOMEM = -3, LM_B200_EUNSUPPORTED = -5 };
 
@@ -46,7 +48,7 @@ enum lm_b200_mixer_kind {
     LM_B200_MIXER_MLSTM = 6,            /* matrix memory with exponential input gate, running maximum and normaliser */
     LM_B200_MIXER_GATED_DELTA = 7,      /* gated delta rule with ONE decay per head and token, short convolutions, silu output gate */
     LM_B200_MIXER_RETENTION = 8,        /* linear attention with a fixed decay per head, rotary q / k, no softmax, no denominator */
-    LM_B200_MIXER_ROTARY_ATTENTION = 9, /* grouped-query attention, per-head q / k norms, rotary positions, window, sink; values = a projection of their own or the raw keys */
+    LM_B200_MIXER_ROTARY_ATTENTION = 9, /* grouped-query attention, per-head q / k norms, rotary positions, window or chunks, sink, elementwise gate; values = a projection of their own or the raw keys */
     LM_B200_MIXER_GATED_LINEAR = 10,    /* linear attention with a data-dependent decay per head and key channel (two-step projection), silu output gate */
     LM_B200_MIXER_MAMBA2 = 11,          /* state-space duality: short convolution, step sizes, one decay per head, gate before a grouped norm */
     LM_B200_MIXER_PAIR = 12             /* two mixers side by side on the same input: part_scale[0] mixer_0(h) + part_scale[1] mixer_1(h) */
@@ -58,7 +60,8 @@ enum lm_b200_layer_form { LM_B200_FORM_SEQUENTIAL = 0, LM_B200_FORM_PARALLEL = 1
  * g' = min(g, limit), u' = clamp(u, -limit, limit): g' sigmoid(1.702 g') (u' + 1) */
 enum lm_b200_act_kind { LM_B200_ACT_SILU_GLU = 0, LM_B200_ACT_XIELU = 1, LM_B200_ACT_CLAMPED_GLU = 2,
                         LM_B200_ACT_RELU2 = 3, /* dense, not gated: up, max(z, 0)^2, down */
-                        LM_B200_ACT_GELU_GLU = 4 /* gated unit with the tanh form of gelu: gelu(g) u */ };
+                        LM_B200_ACT_GELU_GLU = 4, /* gated unit with the tanh form of gelu: gelu(g) u */
+                        LM_B200_ACT_GELU = 5 /* dense, not gated: up, gelu(z) in the tanh form, down */ };
 /* SIGMOID_INPUT: score sigmoid(z) multiplies the chosen expert's input.  SOFTMAX_TOP: the softmax over the chosen logits
  * alone weighs the experts' outputs */
 /* SOFTMAX_GROUPED: scores = softmax over ALL router outputs; the choice is made on score + correction, only inside the
@@ -67,7 +70,8 @@ enum lm_b200_act_kind { LM_B200_ACT_SILU_GLU = 0, LM_B200_ACT_XIELU = 1, LM_B200
  * `identity_experts` router outputs have no weights: their output is their input. */
 enum lm_b200_router_kind { LM_B200_ROUTER_SIGMOID_INPUT = 0, LM_B200_ROUTER_SOFTMAX_TOP = 1, LM_B200_ROUTER_SOFTMAX_GROUPED = 2 };
 /* what the columns `gate` of a mixer's stacked projections do to its output */
-enum lm_b200_gate_kind { LM_B200_GATE_SIGMOID = 0, LM_B200_GATE_NONE = 1, LM_B200_GATE_SILU = 2 };
+/* SIGMOID / SILU: one column per output channel (heads*vdim); SIGMOID_HEAD: one column per head */
+enum lm_b200_gate_kind { LM_B200_GATE_SIGMOID = 0, LM_B200_GATE_NONE = 1, LM_B200_GATE_SILU = 2, LM_B200_GATE_SIGMOID_HEAD = 3 };
 /* which channels of a head form a rotary pair: (2i, 2i + 1), or (i, i + rot_dims / 2) */
 enum lm_b200_rot_layout { LM_B200_ROT_INTERLEAVED = 0, LM_B200_ROT_HALF = 1 };
 /* FP32: every product is fp32 FMA arithmetic on the stored weights.  BF16: the products of a long step (a prompt portion)
@@ -75,7 +79,8 @@ enum lm_b200_rot_layout { LM_B200_ROT_INTERLEAVED = 0, LM_B200_ROT_HALF = 1 };
 enum lm_b200_precision { LM_B200_PRECISION_FP32 = 0, LM_B200_PRECISION_BF16 = 1 };
 
 /* DYT: y = tanh(alpha x) w + b.  LAYER: y = (x - mean) / sqrt(var + eps) * w + b with the model's eps.
- * RMS: y = x / sqrt(mean(x^2) + eps) * w (stream records, the final norm, the embedding norm). */
+ * RMS: y = x / sqrt(mean(x^2) + eps) * w (stream records, the final norm, the embedding norm; a norm stored as its weight's
+ * distance from one is handed over with the one added). */
 typedef struct lm_b200_norm {
     const float *w, *b;
     float alpha;
@@ -155,7 +160,7 @@ typedef struct lm_b200_layer {
      * w_in of the mixers below, in this order:
      *   GATED_DELTA       q (kv_heads*dim) | k (kv_heads*dim) | v (heads*vdim) | beta (heads) | decay (heads) | gate (heads*vdim)
      *   RETENTION         q (heads*dim) | k (heads*dim) | v (heads*vdim) | gate (heads*vdim)
-     *   LATENT_ATTENTION  query latent (q_rank) | key/value latent (kv_rank) | rotated key part (rot_dim) | gate (heads*vdim, unless GATE_NONE)
+     *   LATENT_ATTENTION  query latent (q_rank) | key/value latent (kv_rank) | rotated key part (rot_dim) | gate (heads*vdim or, SIGMOID_HEAD, heads; unless GATE_NONE)
      * GATED_DELTA uses conv_taps, conv_w, conv_tail, a_log [heads], dt_bias [heads], unit_eps, head_norm [vdim] and rec_state
      * as CHANNEL_DELTA does; its decay is exp(-exp(a_log_h) softplus(z_h + dt_bias_h)) per head.  RETENTION: S <- head_decay_h S
      * + k v^T with k times dim^-1/2 after its rotation, o = S^T q, o / rms(o) per head (head_norm NULL: no weight).
@@ -175,11 +180,12 @@ typedef struct lm_b200_layer {
 
     /* ---- more mixers of the stream form, two mixers side by side, and the per-layer token input ----
      * w_in of the mixers below, in this order:
-     *   ROTARY_ATTENTION  q (heads*dim) | k (kv_heads*dim) | v (kv_heads*dim, unless values_are_keys)
+     *   ROTARY_ATTENTION  q (heads*dim) | k (kv_heads*dim) | v (kv_heads*dim, unless values_are_keys) | gate (heads*dim, unless GATE_NONE)
      *   GATED_LINEAR      q (heads*dim) | k (heads*dim) | v (heads*vdim) | gate (heads*vdim, unless GATE_NONE) | a1 (rank_a)
      *   MAMBA2            z (heads*vdim) | x (heads*vdim) | B (kv_heads*dim) | C (kv_heads*dim) | dt (heads)
-     * ROTARY_ATTENTION (vdim == dim): q_norm / k_norm [dim] per-head RMS norms, rot_dims / rot_freq as in TALK_ATTENTION, cosines and
-     * sines times rot_amp, `scale`, `window`, `sink`, k_pages / v_pages.
+     * ROTARY_ATTENTION (vdim == dim): q_norm / k_norm [dim] per-head RMS norms (NULL: no weight), rot_dims / rot_freq as in
+     * TALK_ATTENTION, cosines and sines times rot_amp, `scale`, `window`, `chunk`, `sink`, the gate's sigmoid on the heads' outputs,
+     * k_pages / v_pages.  (A norm without weight is the same before and behind the rotation: turning keeps the mean square.)
      * GATED_LINEAR: S_t = diag(alpha_t) S_(t-1) + k_t v_t^T, o_t = S_t^T q_t with q times dim^-1/2 and alpha = sigmoid(w_a2 (a1 rows h)
      * + dt_bias)^(1 / decay_tau), dt_bias [heads*dim] (NULL: none); o / rms(o) head_norm [vdim] gate.
      * MAMBA2: `dim` is the state size and `kv_heads` the groups that share B and C; x, B, C pass conv_w [heads*vdim + 2 kv_heads*dim]
@@ -201,6 +207,12 @@ typedef struct lm_b200_layer {
     int32_t side_dim, side_ld, side_off; /* side_dim 0: none; side_table is bf16 [vocab][side_ld] */
     const void *side_table, *w_side_gate, *w_side_proj; /* [side_dim][width], [width][side_dim] */
     const float *side_norm;        /* [width] */
+
+    /* ---- chunks; norms on the sublayers' outputs ----
+     * A stream record with streams == 1 and norm_mix_in.w == NULL (and norm_ff_in.w == NULL) reads the stream itself;
+     * norm_mix_out / norm_ff_out (RMS, weight only; w NULL: none) norm the outputs of the mixer and of a dense feed-forward
+     * before hc_out weighs them. */
+    int32_t chunk;                 /* ROTARY_ATTENTION: > 0: positions i and j see one another only inside the same block of `chunk` positions, counted from position 0 */
 } lm_b200_layer;
 
 typedef struct lm_b200_model {
@@ -215,6 +227,12 @@ typedef struct lm_b200_model {
     float logit_scale;             /* multiplies the logits (0 is read as 1) */
     float embed_scale;             /* multiplies the embedding rows (0 is read as 1) */
     const float *embed_norm;       /* [width] RMS norm weight applied to the embedding rows (stream form); NULL: none */
+    /* A second table looked up by the pair (previous token, token) and added to the scaled embedding row (stream form):
+     * row (previous * bigram_mul_prev + token * bigram_mul_cur) mod bigram_buckets, row bigram_buckets for a sequence's first
+     * token.  The multipliers are given reduced mod bigram_buckets.  token_pages keeps the tokens of every sequence. */
+    const void *bigram;            /* bf16 [bigram_buckets + 1][width]; NULL: none */
+    int32_t bigram_buckets, bigram_mul_prev, bigram_mul_cur;
+    int32_t *token_pages;          /* [pages][page_size] token ids, on the page table of the keys and values */
 } lm_b200_model;
 
 typedef struct lm_b200_engine lm_b200_engine;

@@ -54,7 +54,7 @@ def test_configuration_is_read_by_layer_type_and_checked():
 
 def test_layer_records_stack_their_projections_and_describe_their_state():
     from dia_tts_prune_b200.lm_config import load_config
-    from dia_tts_prune_b200.lm_layers import DenseRelu2, GatedDelta, LatentAttention, Retention, RoutedExperts
+    from dia_tts_prune_b200.lm_layers import DenseUnit, GatedDelta, LatentAttention, Retention, RoutedExperts
     from dia_tts_prune_b200.lm_model import build_fipadra_layers
     cfg = config()
     w = O.random_weights(cfg, 3)
@@ -68,7 +68,7 @@ def test_layer_records_stack_their_projections_and_describe_their_state():
     assert torch.equal(delta.w_in[48:72].float(), w["l0.mix.g"]) and delta.mixer.conv_w.shape == (40, 3)
     sp = delta.mixer.state_spec()
     assert sp.recurrent == (4, 6, 4) and sp.conv == (3, 40) and sp.latent is None
-    assert isinstance(delta.ff, DenseRelu2) and delta.ff.ff == 12
+    assert isinstance(delta.ff, DenseUnit) and delta.ff.act == "relu2" and delta.ff.ff == 12
     # latent attention: query latent | key/value latent with the turned key part behind it | no gate rows; padded to four
     assert isinstance(att.mixer, LatentAttention) and not att.mixer.gated and att.n_in == 16 and att.w_in.shape == (16, 16)
     assert torch.equal(att.w_in[:5].float(), w["l1.mix.dq"]) and torch.equal(att.w_in[5:16].float(), w["l1.mix.dkv"])
