@@ -24,7 +24,7 @@ sizes of a real model: prefill and decode throughput through `CausalLM`, and its
 at equal size (one JSON line, metric `lm_layer_throughput`).  `--lm --lm-design luketar` measures the Luketar design
 beside Kupelix and Pubopel at equal width and its mixers beside Kupelix's.  `--lm --lm-design fipadra` measures the Fipadra
 design beside Luketar at equal width and its mixers beside their likes in Luketar and Kupelix.  `--lm --lm-design loduzen`
-measures the Loduzen design beside Fipadra with dense units.  `--lm --lm-design kupelix` measures the Kupelix design
+measures the Loduzen design beside Fipadra with dense units, `--lm --lm-design forilorn` the Forilorn design likewise.  `--lm --lm-design kupelix` measures the Kupelix design
 instead: its prefill and decode throughput beside Pubopel's at equal width, heads and vocabulary, its attention kernel
 beside Pubopel's on the same causal workload, and its recurrence kernels against the bytes and state updates they must move.
 """
@@ -1206,6 +1206,141 @@ def run_lm_loduzen(args) -> None:
                       "gpu_launches": launch_count() - launches0, "clocks": clocks, "lm": out}))
 
 
+# ---- --lm --lm-design forilorn: the Forilorn design beside Fipadra with dense units, its mixers beside their likes --------------
+FORILORN_SIZES = {
+    # the widths, head counts, latent sizes, windows and vocabularies of FIPADRA_SIZES and a dense unit of the same size; chunks of
+    # twice the window, so that a query of either attention sees as many keys on average
+    "w2048": dict(width=2048, kinds=["attention", "latent_attention", "attention", "latent_attention"], heads=16, kv_heads=4, dim=128,
+                  chunk=2048, lat_dim=96, rot_dim=32, lat_vdim=128, q_rank=768, kv_rank=256, window=1024, ff=6144, rot_dims=128,
+                  buckets=65521, scale=45.0, residual_mult=0.3, vocab=32768),
+    "w1024": dict(width=1024, kinds=["attention", "latent_attention", "attention", "latent_attention"], heads=8, kv_heads=2, dim=128,
+                  chunk=2048, lat_dim=96, rot_dim=32, lat_vdim=128, q_rank=384, kv_rank=128, window=1024, ff=1536, rot_dims=128,
+                  buckets=32749, scale=32.0, residual_mult=0.3, vocab=16384),
+}
+
+
+def run_lm_forilorn(args) -> None:
+    import torch
+    from dia_tts_prune_b200 import synthetic as SY
+    from dia_tts_prune_b200.lm_config import FipadraConfig, ForilornConfig, PubopelConfig
+    from dia_tts_prune_b200.lm_engine import launch_count
+    from dia_tts_prune_b200.lm_model import CausalLM
+
+    if not torch.cuda.is_available():
+        raise SystemExit("bench.py needs a CUDA device: the product path has no CPU fallback")
+    dev = torch.device("cuda", 0)
+    torch.cuda.set_device(dev)
+    try:
+        with open(os.path.join(REPO, "MEASURED_PEAKS.json")) as f:
+            pk = json.load(f)
+        hbm, tf, src = float(pk["hbm_gbs"]), float(pk["bf16_tflops"]), "measured"
+    except Exception:
+        hbm, tf, src = 6650.0, 1590.0, "fallback"
+    flush = torch.zeros(160 << 20, dtype=torch.uint8, device=dev)             # > the 126 MB L2
+    W, K = max(args.warmup, 3), max(args.steps, 3)
+    sampler = ClockSampler(0)
+    sampler.start()
+    launches0 = launch_count()
+    out = {}
+    T, ctx, R = args.lm_prompt, args.lm_context, args.lm_rows
+
+    def figures(entry, flops, n_bytes):
+        pf, b1 = entry["prefill"], entry["decode_b1"]
+        pf.update(model_tflops=flops / pf["ms"] / 1e9, frac_of_bf16_peak=flops / pf["ms"] / 1e9 / tf)
+        b1.update(algorithmic_bytes=n_bytes, gb_per_s=n_bytes / b1["ms_per_step"] / 1e6,
+                  frac_of_hbm_peak=n_bytes / b1["ms_per_step"] / 1e6 / hbm)
+
+    for name in (args.lm_sizes.split(",") if args.lm_sizes else FORILORN_SIZES):
+        sz, fsz, psz = FORILORN_SIZES[name], FIPADRA_SIZES[name], LM_SIZES[name]
+        D, H, G, d, V, kinds = sz["width"], sz["heads"], sz["kv_heads"], sz["dim"], sz["vocab"], sz["kinds"]
+        dp, dr, dv, rq, rk, win, chunk = (sz[k] for k in ("lat_dim", "rot_dim", "lat_vdim", "q_rank", "kv_rank", "window", "chunk"))
+        toks = torch.randint(0, V, (T,), generator=torch.Generator().manual_seed(7)).tolist()
+        cap = max(T, 8 * (ctx + 32 * (K + 2))) + 64
+        res = {"config": dict(sz)}
+        kw = dict(dtype="bfloat16", device=dev, max_tokens=cap, max_sequences=8, page_size=64, max_rows=R)
+        # products per token and (query, key) pairs of the prompt
+        lat = rq * H * (dp + dr) + H * dp * rk + H * rk * dv + H * dv * D
+        cols = {"attention": D * (2 * H * d + G * d) + H * d * D, "latent_attention": D * (rq + rk + dr + H) + lat}
+        pairs_w, pairs_c = sum(min(t + 1, win) for t in range(T)), sum(t % chunk + 1 for t in range(T))
+        attn = {"attention": 4.0 * H * d * pairs_c, "latent_attention": 2.0 * H * (2 * rk + dr) * pairs_w}
+        kv = {"attention": 8.0 * G * d * (ctx % chunk + 1), "latent_attention": 4.0 * (rk + dr) * min(ctx, win)}
+        ff = 2 * D * sz["ff"]
+        work = lambda c: 2.0 * T * sum(c[k] + ff for k in kinds) + sum(attn[k] for k in kinds) + 2.0 * D * V      # noqa: E731
+        cfg = SY.forilorn_config(**sz)
+        model = CausalLM(ForilornConfig.model_validate(cfg), SY.forilorn_weights(cfg, WEIGHT_SEED, dev), **kw)
+        res["forilorn"] = _lm_prefill_decode(model, toks, T, ctx, W, K, flush)
+        figures(res["forilorn"], work(cols), 2.0 * (sum(cols[k] + ff for k in kinds) + D * V) + sum(kv[k] for k in kinds))
+        model.engine.close()
+        del model
+        torch.cuda.empty_cache()
+        # the closest whole model: Fipadra with windowed latent attention in every layer and dense units of the same size
+        fcfg = _fipadra_config({**fsz, "kinds": ["latent_attention"] * len(kinds), "experts": 0})
+        model = CausalLM(FipadraConfig.model_validate(fcfg), SY.fipadra_weights(fcfg, WEIGHT_SEED, dev), **kw)
+        res["fipadra_latent_dense"] = _lm_prefill_decode(model, toks, T, ctx, W, K, flush)
+        f_cols, n = D * (rq + rk + dr) + lat, len(kinds)
+        figures(res["fipadra_latent_dense"], 2.0 * T * n * (f_cols + ff) + n * attn["latent_attention"] + 2.0 * D * V,
+                2.0 * (n * (f_cols + ff) + D * V) + n * kv["latent_attention"])
+        model.engine.close()
+        del model
+        torch.cuda.empty_cache()
+
+        # -- sublayers alone: one-layer models of either design
+        def timed(m1, n_seq, rows_each, start):
+            h = torch.randn(n_seq * min(rows_each, R), D, device=dev)
+            seqs = [m1.state.open(f"s{i}") for i in range(n_seq)]
+            for sq in seqs:
+                m1.state.reserve(sq, start + rows_each)
+            def run():
+                for r0 in range(0, rows_each, R):
+                    k = min(R, rows_each - r0)
+                    m1.engine.op_mixer(0, h[:n_seq * k], [(sq, k, start + r0) for sq in seqs])
+            ms = _event_ms(run, 2, K, flush)
+            for i in range(n_seq):
+                m1.state.close(f"s{i}")
+            return ms
+
+        kw1 = dict(dtype="bfloat16", device=dev, max_tokens=8 * T + 64, max_sequences=8, page_size=64, max_rows=R)
+        one = lambda conf, c, weights: CausalLM(conf.model_validate(c), weights(c, 3, dev), **kw1)      # noqa: E731
+        c_pub = SY.pubopel_config(**{**psz, "layers": 1, "vocab": 256, "experts": 1, "top": 1, "expert_ff": 8, "shared_ff": 0,
+                                     "window": win, "keep_first": 0})
+        c_fip = _fipadra_config({**fsz, "kinds": ["latent_attention"], "vocab": 256, "ff": 0, "experts": 0})
+        likes = {"attention": ("pubopel_attention", one(PubopelConfig, c_pub, SY.pubopel_weights)),
+                 "latent_attention": ("fipadra_latent_attention", one(FipadraConfig, c_fip, SY.fipadra_weights))}
+        mixers = {}
+        for kind, (label2, m2) in likes.items():
+            c1 = SY.forilorn_config(**{**sz, "kinds": [kind], "vocab": 256, "ff": 0, "buckets": 0})
+            m1 = one(ForilornConfig, c1, SY.forilorn_weights)
+            ent = {}
+            for label, (n_seq, rows_each, start) in {"prefill_1x%d" % T: (1, T, 0), "prefill_8x%d" % (T // 8): (8, T // 8, 0),
+                                                     "decode_b1": (1, 1, ctx), "decode_b8": (8, 1, ctx)}.items():
+                ent[label] = {"forilorn_ms": timed(m1, n_seq, rows_each, start), label2 + "_ms": timed(m2, n_seq, rows_each, start)}
+            mixers[kind] = ent
+            for m in (m1, m2):
+                m.engine.close()
+            del m1, m2
+            torch.cuda.empty_cache()
+        res["mixers"] = mixers
+        # the gelu unit beside Fipadra's squared-relu unit of the same size
+        units = {"forilorn": one(ForilornConfig, SY.forilorn_config(**{**sz, "kinds": ["attention"], "vocab": 256, "buckets": 0}), SY.forilorn_weights),
+                 "fipadra_relu2": one(FipadraConfig, _fipadra_config({**fsz, "kinds": ["latent_attention"], "vocab": 256, "experts": 0, "ff": sz["ff"]}),
+                                      SY.fipadra_weights)}
+        res["unit"] = {}
+        for rows in (T, 1, 8):
+            h = torch.randn(rows, D, device=dev)
+            res["unit"][f"rows_{rows}"] = {who + "_ms": _event_ms(lambda m=m: m.engine.op_ff(0, h), 2, K, flush) for who, m in units.items()}
+        for m in units.values():
+            m.engine.close()
+        del units
+        torch.cuda.empty_cache()
+        out[name] = res
+    clocks = sampler.stop()
+    print(json.dumps({"metric": "lm_layer_throughput", "design": "forilorn", "impl": "ours", "n_gpus": 1, "steps": K, "warmup": W,
+                      "dtype": "bf16", "data": "synthetic (random weights, random token ids)",
+                      "peaks": {"hbm_gbs": hbm, "bf16_tflops": tf, "source": src},
+                      "timing": "CUDA events, median; a 160 MB buffer is rewritten between timed iterations (L2 flush)",
+                      "gpu_launches": launch_count() - launches0, "clocks": clocks, "lm": out}))
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -1228,18 +1363,20 @@ def main():
     ap.add_argument("--lm", action="store_true",
                     help="instead of the headline workload: prefill / decode throughput of the decoder-only language-model path "
                          "(Pubopel, random weights) at layer sizes of a real model, beside Dia's kernels at equal size")
-    ap.add_argument("--lm-design", default="pubopel", choices=["pubopel", "kupelix", "luketar", "fipadra", "loduzen"],
+    ap.add_argument("--lm-design", default="pubopel", choices=["pubopel", "kupelix", "luketar", "fipadra", "loduzen", "forilorn"],
                     help="--lm: the design that is measured (kupelix: beside Pubopel at equal width, and its kernels beside Pubopel's; "
                          "luketar: beside Kupelix and Pubopel at equal width, and its mixers beside Kupelix's; fipadra: beside Luketar at equal "
                          "width, and its mixers beside their likes in Luketar and Kupelix; loduzen: beside Fipadra with dense units at equal "
-                         "width, and its mixers beside their likes in Pubopel, Kupelix and Fipadra)")
+                         "width, and its mixers beside their likes in Pubopel, Kupelix and Fipadra; forilorn: beside Fipadra with latent "
+                         "attention and dense units at equal width, and its mixers and unit beside their likes in Pubopel and Fipadra)")
     ap.add_argument("--lm-sizes", default="", help="--lm: comma-separated subset of " + ",".join(LM_SIZES))
     ap.add_argument("--lm-prompt", type=int, default=4096, help="--lm: prompt tokens of the prefill measurement")
     ap.add_argument("--lm-rows", type=int, default=4096, help="--lm: most rows of one engine step (longer prompts run in portions)")
     ap.add_argument("--lm-context", type=int, default=1024, help="--lm: tokens each sequence holds before the decode measurement")
     args = ap.parse_args()
     if args.lm:
-        {"kupelix": run_lm_kupelix, "luketar": run_lm_luketar, "fipadra": run_lm_fipadra, "loduzen": run_lm_loduzen}.get(args.lm_design, run_lm)(args)
+        {"kupelix": run_lm_kupelix, "luketar": run_lm_luketar, "fipadra": run_lm_fipadra, "loduzen": run_lm_loduzen,
+         "forilorn": run_lm_forilorn}.get(args.lm_design, run_lm)(args)
         return
     if args.impl == "reference":
         run_reference(args)

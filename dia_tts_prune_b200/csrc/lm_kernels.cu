@@ -748,7 +748,8 @@ sink_attention_tile_kernel(const float* __restrict__ qk, int q_stride, const flo
     int* s_pos = s_slot + kTQ;                                // [64]
 
     const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
-    const int r0 = (gridDim.x - 1 - blockIdx.x) * kTQ, h = blockIdx.y;    // later rows see more keys: they start first
+    // later rows see more keys: their tiles start first, for all heads (a tile's heads are neighbours in launch order)
+    const int r0 = (gridDim.y - 1 - blockIdx.y) * kTQ, h = blockIdx.x;
     const int n_rows = min(kTQ, M - r0);
     const int g = h / (heads / kv_heads);
     const bool vec = (dim % 4) == 0 && (q_stride % 4) == 0;
@@ -1229,7 +1230,8 @@ static cudaError_t launch_attention_tiles(const float* qk, int q_stride, const f
         if (e != cudaSuccess) return e;
         if (dev >= 0 && dev < 64) attr[dev] = true;
     }
-    sink_attention_tile_kernel<NC><<<dim3((M + kTQ - 1) / kTQ, a.heads), kTileThreads, smem, st>>>(
+    if ((M + kTQ - 1) / kTQ > 65535) return cudaErrorNotSupported;
+    sink_attention_tile_kernel<NC><<<dim3(a.heads, (M + kTQ - 1) / kTQ), kTileThreads, smem, st>>>(
         qk, q_stride, kcache, vcache, pm.table, pm.max_pages, pm.page_size, a.heads, a.kv_heads, a.dim, a.scale, a.softcap,
         a.temp, a.slopes, a.sink, a.window, a.keep_first, rm.slot, rm.pos, out, out_b, ldo, out_scale, M, a.chunk, gate, ldg);
     return cudaGetLastError();

@@ -547,6 +547,8 @@ talk_attention_kernel(const float* __restrict__ proj, int ld, int q_off, int gat
     __syncthreads();
     if (!is_last) return;
     __threadfence();
+    // the merge reads S shares of every output: the weights of the shares go to shared memory first (Rs is free), then every
+    // thread requests all shares of an output (two neighbouring ones where they are aligned) before it sums them in their order
     for (int h = warp; h < H; h += NW) {
         const float* src = part + ((size_t)r0 * H + h) * S * stride;
         const float ms = lane < S ? __ldcg(src + lane * stride) : -CUDART_INF_F;
@@ -558,19 +560,41 @@ talk_attention_kernel(const float* __restrict__ proj, int ld, int q_off, int gat
         for (int t = 0; t < S; ++t) l += __shfl_sync(0xffffffffu, ls * w, t);
         float f = l > 0.f ? 1.0f / l : 0.f;
         if (gate_off >= 0) f *= proj[(size_t)r0 * ld + gate_off + h];
-        for (int c0 = 0; c0 < vdim; c0 += 32) {
-            const int col = c0 + lane;
-            float o = 0.f;
-            for (int t = 0; t < S; ++t) {
-                const float wt = __shfl_sync(0xffffffffu, w, t);
-                if (col < vdim) o = fmaf(__ldcg(src + t * stride + 2 + col), wt, o);
-            }
-            if (col < vdim) {
-                o *= f;
-                out[(size_t)r0 * ldo + (size_t)h * vdim + col] = o;
-                if (out_b) out_b[(size_t)r0 * ldo + (size_t)h * vdim + col] = __float2bfloat16_rn(o);
-            }
+        Rs[h * TK + lane] = w;                                // (0 beyond the last share)
+        if (lane == 0) Rs[h * TK + kAttnSplitsMax] = f;
+    }
+    __syncthreads();
+    static_assert(kAttnSplitsMax == 32 && TK > kAttnSplitsMax, "a lane per share, the shares' weights in a row of Rs");
+    auto put = [&](int h, int col, float o) {
+        out[(size_t)r0 * ldo + (size_t)h * vdim + col] = o;
+        if (out_b) out_b[(size_t)r0 * ldo + (size_t)h * vdim + col] = __float2bfloat16_rn(o);
+    };
+    if (vdim % 2 == 0) {
+        const int half = vdim >> 1;
+        for (int idx = tid; idx < H * half; idx += NT) {
+            const int h = idx / half, col = 2 * (idx - h * half);
+            const float* src = part + ((size_t)r0 * H + h) * S * stride + 2 + col;
+            const float* wgt = Rs + h * TK;
+            float2 v[kAttnSplitsMax];
+#pragma unroll
+            for (int t = 0; t < kAttnSplitsMax; ++t)
+                v[t] = t < S ? __ldcg(reinterpret_cast<const float2*>(src + t * stride)) : make_float2(0.f, 0.f);
+            float a = 0.f, b = 0.f;
+#pragma unroll
+            for (int t = 0; t < kAttnSplitsMax; ++t) { a = fmaf(v[t].x, wgt[t], a); b = fmaf(v[t].y, wgt[t], b); }
+            put(h, col, a * wgt[kAttnSplitsMax]);
+            put(h, col + 1, b * wgt[kAttnSplitsMax]);
         }
+        return;
+    }
+    for (int idx = tid; idx < H * vdim; idx += NT) {
+        const int h = idx / vdim, col = idx - h * vdim;
+        const float* src = part + ((size_t)r0 * H + h) * S * stride + 2 + col;
+        const float* wgt = Rs + h * TK;
+        float o = 0.f;
+#pragma unroll 8
+        for (int t = 0; t < S; ++t) o = fmaf(__ldcg(src + t * stride), wgt[t], o);
+        put(h, col, o * wgt[kAttnSplitsMax]);
     }
 }
 

@@ -15,6 +15,8 @@
 //                             streams), a second norm weight on the same statistics, RMS instead of layer norm, the input
 //                             row for assignments without a slot (identity experts), a sigmoid gate number on y, an RMS norm
 //                             of y before it is written (also the norm on a sublayer's output)
+//   residual_norm_kernel      the same step where the sublayers read the (one) stream itself and their outputs are normed:
+//                             x <- mix x + out rms(y) w and the bf16 copy of x, in one pass over registers
 //   latent_prep_kernel        RMS norms of the query latent (in place, + bf16 operand) and of the key/value latent (into
 //                             the pages: the latent is all an attention layer of this kind caches - and, behind it, one
 //                             key part turned with the position where the layer has one)
@@ -234,6 +236,55 @@ streams_step_kernel(float* __restrict__ X, const float* __restrict__ mix, const 
 }
 
 // ---------------------------------------------------------------------------------------------------------------------
+// The step of a record whose sublayers read the stream itself (one stream, plain weights): x <- mix x + out norm(y), with
+// norm(y) = y / sqrt(mean(y^2) + eps) w, and the bf16 copy of x.  One CTA per row; a thread holds its 4 NV columns of x and y in
+// registers, so that both rows are in flight before the reduction.  The arithmetic is streams_step_kernel's.
+template <int NV>
+__global__ void __launch_bounds__(256)
+residual_norm_kernel(float* __restrict__ x, const float* __restrict__ mix, const float* __restrict__ out, const float* __restrict__ y,
+                     const float* __restrict__ w, float eps, __nv_bfloat16* __restrict__ x_b, int D) {
+    __shared__ float red[8];
+    pdl_release();
+    const float mw = mix[0], ow = out[0];
+    const int n4 = D >> 2;
+    float4 wv[NV];
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        const int c = threadIdx.x + i * blockDim.x;
+        wv[i] = c < n4 ? reinterpret_cast<const float4*>(w)[c] : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    pdl_wait();
+    float4* xr = reinterpret_cast<float4*>(x + (size_t)blockIdx.x * D);
+    const float4* yr = reinterpret_cast<const float4*>(y + (size_t)blockIdx.x * D);
+    float4 xv[NV], yv[NV];
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        const int c = threadIdx.x + i * blockDim.x;
+        yv[i] = c < n4 ? yr[c] : make_float4(0.f, 0.f, 0.f, 0.f);
+        xv[i] = c < n4 ? xr[c] : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+#pragma unroll
+    for (int i = 0; i < NV; ++i) ss = fmaf(yv[i].x, yv[i].x, fmaf(yv[i].y, yv[i].y, fmaf(yv[i].z, yv[i].z, fmaf(yv[i].w, yv[i].w, ss))));
+    const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)D + eps);
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        const int c = threadIdx.x + i * blockDim.x;
+        if (c >= n4) break;
+        float4 v;
+        v.x = fmaf(ow, yv[i].x * (inv * wv[i].x), mw * xv[i].x);
+        v.y = fmaf(ow, yv[i].y * (inv * wv[i].y), mw * xv[i].y);
+        v.z = fmaf(ow, yv[i].z * (inv * wv[i].z), mw * xv[i].z);
+        v.w = fmaf(ow, yv[i].w * (inv * wv[i].w), mw * xv[i].w);
+        xr[c] = v;
+        if (x_b) {
+            const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+            reinterpret_cast<uint2*>(x_b + (size_t)blockIdx.x * D)[c] =
+                make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+        }
+    }
+}
+
 // turns the pair (a, b) by angle pos * f
 __device__ __forceinline__ void turn_pair(float& a, float& b, int pos, float f) {
     float sn, cs;
@@ -610,6 +661,15 @@ cudaError_t launch_streams_step(float* X, int streams, const StreamWrite& wr, co
     const size_t smem = (size_t)D * 4;
     auto aligned = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
     const bool vec = D % 4 == 0 && aligned(X) && aligned(wr.y) && aligned(wr.parts) && aligned(ex.y2) && aligned(ex.ident_h);
+    // nothing but the normed output written into the one stream, and at most the bf16 copy of the stream asked for
+    if (streams == 1 && vec && D <= 4096 && wr.mix && wr.y && !wr.parts && !rows && !h && !in && !norm_w && ex.y_norm_w && !ex.y2 &&
+        !ex.y_gate && aligned(ex.y_norm_w) && aligned(h_bf16)) {
+        const int threads = D <= 256 ? 64 : D <= 512 ? 128 : 256, nv = (D / 4 + threads - 1) / threads;
+        void (*k)(float*, const float*, const float*, const float*, const float*, float, __nv_bfloat16*, int) =
+            nv <= 1 ? residual_norm_kernel<1> : nv <= 2 ? residual_norm_kernel<2> : residual_norm_kernel<4>;
+        return launch_pdl(k, dim3(M), dim3(threads), 0, st, X, wr.mix, wr.out, wr.y, ex.y_norm_w, eps,
+                          reinterpret_cast<__nv_bfloat16*>(h_bf16), D);
+    }
     using Kernel = void (*)(float*, const float*, const float*, const float*, const float*, const int*, const float*, int, const float*,
                             const float*, float, const int*, float*, __nv_bfloat16*, int, const StreamExtra);
     Kernel kernel = nullptr;

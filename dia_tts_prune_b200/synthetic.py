@@ -454,3 +454,64 @@ def loduzen_weights(cfg: dict, seed: int = 1234, device="cpu", rank: int = 16) -
         if side:
             w[p + "side.gate"], w[p + "side.proj"], w[p + "side.norm"] = mat(side, D), mat(D, side), vec(D, 0.3, 0.05)
     return w
+
+
+def forilorn_config(width: int, kinds: list[str], heads: int, dim: int, vocab: int, kv_heads: int = 0, chunk: int = 0, lat_heads: int = 0,
+                    lat_dim: int = 0, rot_dim: int = 0, lat_vdim: int = 0, q_rank: int = 0, kv_rank: int = 0, window: int = 0,
+                    ff: int = 0, rot_dims: int = 0, buckets: int = 0, scale: float = 1.0, residual_mult: float = 1.0) -> dict:
+    """A Forilorn ``config.json`` as a dictionary: one layer per entry of ``kinds`` (``attention`` / ``latent_attention``), each with a
+    dense unit of ``ff`` hidden units (none when 0); ``buckets``: the pair table's (no table when 0)."""
+    layers = []
+    for kind in kinds:
+        if kind == "attention":
+            m = {"heads": heads, "kv_heads": kv_heads or heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5,
+                 "rot": {"base": 10000.0, "dims": rot_dims or dim}}
+            size = chunk
+        else:
+            h, d = lat_heads or heads, lat_dim or dim
+            m = {"heads": h, "dim": d, "rot_dim": rot_dim, "vdim": lat_vdim or d, "q_rank": q_rank, "kv_rank": kv_rank,
+                 "scale": (d + rot_dim) ** -0.5, "rot": {"base": 10000.0, "dims": rot_dim}}
+            size = window
+        if size:
+            m["mask"] = {"size": size}
+        layers.append({"type": kind, "mixer": m, "mlp": {"kind": "dense", "ff": ff} if ff else None})
+    emb = {"scale": scale}
+    if buckets:
+        emb["bigram"] = {"buckets": buckets, "mul_prev": 40503, "mul_cur": 10007}
+    return {"architecture": "Forilorn", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "residual_mult": residual_mult,
+            "embedding": emb, "layers": layers}
+
+
+def forilorn_weights(cfg: dict, seed: int = 1234, device="cpu") -> dict:
+    """Random bfloat16 tensors under the checkpoint's names: matrices ~ N(0, 1 / fan_in), norm weights stored around zero."""
+    import torch
+    g = torch.Generator(device=device).manual_seed(seed)
+    D, V = cfg["width"], cfg["vocab"]
+
+    def mat(n, k, gain=1.0):
+        return (torch.randn((n, k), generator=g, device=device) * (gain * k ** -0.5)).to(torch.bfloat16)
+
+    def vec(n, mean, spread):
+        return (mean + spread * torch.randn((n,), generator=g, device=device)).to(torch.bfloat16)
+
+    w = {"embed": mat(V, D), "final.norm": vec(D, 0.0, 0.05)}
+    bigram = cfg["embedding"].get("bigram")
+    if bigram:
+        w["bigram"] = mat(bigram["buckets"] + 1, D)
+    for i, lc in enumerate(cfg["layers"]):
+        p, m = f"l{i}.", lc["mixer"]
+        q, H, d, dv = p + "mix.", m["heads"], m["dim"], m["vdim"]
+        w[p + "norm1"] = vec(D, 0.0, 0.05)
+        if lc["type"] == "attention":
+            G = m["kv_heads"]
+            w[q + "q"], w[q + "k"], w[q + "g"], w[q + "o"] = mat(H * d, D), mat(G * d, D), mat(H * d, D), mat(D, H * d)
+        else:
+            r, Rq, R = m["rot_dim"], m["q_rank"], m["kv_rank"]
+            w[q + "dq"], w[q + "dq.norm"], w[q + "uq"] = mat(Rq, D), vec(Rq, 1.0, 0.05), mat(H * (d + r), Rq)
+            w[q + "dkv"], w[q + "dkv.norm"] = mat(R + r, D), vec(R, 1.0, 0.05)
+            w[q + "uk"], w[q + "uv"], w[q + "g"], w[q + "o"] = mat(H * d, R), mat(H * dv, R), mat(H, D), mat(D, H * dv)
+        f = lc.get("mlp")
+        if f:
+            w[p + "norm2"] = vec(D, 0.0, 0.05)
+            w[p + "mlp.up"], w[p + "mlp.down"] = mat(f["ff"], D), mat(D, f["ff"])
+    return w
