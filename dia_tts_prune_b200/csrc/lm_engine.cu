@@ -1087,8 +1087,8 @@ size_t lm_b200_engine_workspace_bytes(const lm_b200_engine* e) { return e ? e->a
 
 namespace {
 
-// the final norm of the wanted rows of e->x and the logits
-int head_rows(lm_b200_engine* e, const StepView& v, int n_want, float* logits_out, cudaStream_t st) {
+// the final norm of the wanted rows of x [M][width] and the logits
+int head_rows(lm_b200_engine* e, const float* x, const StepView& v, int n_want, float* logits_out, cudaStream_t st) {
     const int D = e->m.width;
     if (n_want > 0) {
         // the head is the largest single weight stream: from kHeadTensorRowsMin wanted rows on (a batch of decoding
@@ -1096,11 +1096,11 @@ int head_rows(lm_b200_engine* e, const StepView& v, int n_want, float* logits_ou
         const bool tc = e->m.precision == LM_B200_PRECISION_BF16 && n_want >= kHeadTensorRowsMin &&
                         dia::gemm_tcgen05_shape_ok(n_want, e->m.vocab, D) && (reinterpret_cast<uintptr_t>(logits_out) & 15) == 0;
         if (e->m.final_norm.kind == LM_B200_NORM_LAYER || e->m.final_norm.kind == LM_B200_NORM_RMS)
-            LCK(lm::launch_layernorm_rows(e->x, v.want, e->m.final_norm.w, e->m.final_norm.b, e->m.eps,
+            LCK(lm::launch_layernorm_rows(x, v.want, e->m.final_norm.w, e->m.final_norm.b, e->m.eps,
                                           e->m.logit_scale != 0.f ? e->m.logit_scale : 1.f, e->hw, tc ? e->hwb : nullptr, n_want, D, st,
                                           e->m.final_norm.kind == LM_B200_NORM_RMS));
         else
-            LCK(lm::launch_dyt_gather(e->x, v.want, N(e->m.final_norm), e->hw, tc ? e->hwb : nullptr, n_want, D, st));
+            LCK(lm::launch_dyt_gather(x, v.want, N(e->m.final_norm), e->hw, tc ? e->hwb : nullptr, n_want, D, st));
         if (tc)
             LCK(dia::launch_gemm_tcgen05_bf16(e->hwb, 1, e->m.head, e->m.vocab, logits_out, n_want, e->m.vocab, D, kPlain, nullptr, st));
         else
@@ -1110,7 +1110,7 @@ int head_rows(lm_b200_engine* e, const StepView& v, int n_want, float* logits_ou
 }
 
 
-// every layer of a stream-form model: the streams end up summed in e->x
+// every layer of a stream-form model: the streams end up summed in e->x (one stream: it stays where it is, in e->xs)
 int run_stream_layers(lm_b200_engine* e, const StepView& v, int M, int n_seq, float* layers_out, cudaStream_t st) {
     const int D = e->m.width, s = e->layers[0].streams, n = e->m.n_layer;
     const float eps = e->m.eps;
@@ -1197,8 +1197,8 @@ int run_stream_layers(lm_b200_engine* e, const StepView& v, int M, int n_seq, fl
             if (layers_out)
                 LCK(lm::launch_streams_step(e->xs, s, none, nullptr, nullptr, eps, nullptr, layers_out + (size_t)i * M * D, nullptr, M, D, st));
         } else {
-            LCK(lm::launch_streams_step(e->xs, s, wr, nullptr, nullptr, eps, nullptr, e->x, nullptr, M, D, st, wx));
-            if (layers_out && cudaMemcpyAsync(layers_out + (size_t)i * M * D, e->x, (size_t)M * D * 4, cudaMemcpyDeviceToDevice, st) !=
+            LCK(lm::launch_streams_step(e->xs, s, wr, nullptr, nullptr, eps, nullptr, s == 1 ? nullptr : e->x, nullptr, M, D, st, wx));
+            if (layers_out && cudaMemcpyAsync(layers_out + (size_t)i * M * D, s == 1 ? e->xs : e->x, (size_t)M * D * 4, cudaMemcpyDeviceToDevice, st) !=
                                   cudaSuccess)
                 return cuda_fail(cudaGetLastError());
         }
@@ -1214,7 +1214,7 @@ int run_step(lm_b200_engine* e, const int32_t* step, int M, int n_seq, int n_wan
     if (e->stream_form) {
         const int rc = run_stream_layers(e, v, M, n_seq, layers_out, st);
         if (rc) return rc;
-        return head_rows(e, v, n_want, logits_out, st);
+        return head_rows(e, e->layers[0].streams == 1 ? e->xs : e->x, v, n_want, logits_out, st);
     }
     LCK(lm::launch_embed(e->m.embed, v.token, e->x, M, e->m.vocab, D, st));
     bool keep_x0 = false;
@@ -1260,7 +1260,7 @@ int run_step(lm_b200_engine* e, const int32_t* step, int M, int n_seq, int n_wan
                 return cuda_fail(cudaGetLastError());
         }
     }
-    return head_rows(e, v, n_want, logits_out, st);
+    return head_rows(e, e->x, v, n_want, logits_out, st);
 }
 
 // A step of a few rows is some forty short dependent launches: it is captured once per (rows, sequences, wanted) over

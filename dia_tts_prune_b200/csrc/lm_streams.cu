@@ -49,6 +49,8 @@ constexpr int kMaxStreams = 8;
 // A row's previous token stands in the row before it (the rows of a sequence are adjacent) or, for the first row its sequence
 // has in the step, at the position before in the sequence's token pages; every row writes its own token there.  A step reads
 // only positions in front of its first row and writes only from there on, so the rows do not race.
+// VW = 8: D is a multiple of 8 and the table rows are moved in 16-byte pieces.
+template <int VW>
 __global__ void streams_embed_kernel(const __nv_bfloat16* __restrict__ table, const int* __restrict__ ids, float scale,
                                      const float* __restrict__ norm_w, float eps, float* __restrict__ X, __nv_bfloat16* __restrict__ Xb,
                                      int streams, int V, int D, const BigramRows bg) {
@@ -68,21 +70,65 @@ __global__ void streams_embed_kernel(const __nv_bfloat16* __restrict__ table, co
         if (row >= 0) pair = reinterpret_cast<const __nv_bfloat16*>(bg.table) + (size_t)row * D;
         if (threadIdx.x == 0) bg.token_pages[(size_t)pages[pos / ps] * ps + pos % ps] = id;
     }
-    auto value = [&](int c) { return (ok ? bf(table[(size_t)id * D + c]) * scale : 0.f) + (pair ? bf(pair[c]) : 0.f); };
+    const __nv_bfloat16* own = ok ? table + (size_t)id * D : nullptr;
+    auto load = [](const __nv_bfloat16* p, float (&v)[VW]) {
+        if (VW == 8) {
+            const uint4 t = *reinterpret_cast<const uint4*>(p);
+            const __nv_bfloat162* q = reinterpret_cast<const __nv_bfloat162*>(&t);
+#pragma unroll
+            for (int e = 0; e < VW / 2; ++e) { v[2 * e] = __low2float(q[e]); v[2 * e + 1] = __high2float(q[e]); }
+        } else {
+            v[0] = bf(*p);
+        }
+    };
+    auto value = [&](int c, float (&v)[VW]) {
+        float a[VW], b[VW];
+#pragma unroll
+        for (int e = 0; e < VW; ++e) a[e] = b[e] = 0.f;
+        if (own) load(own + c, a);
+        if (pair) load(pair + c, b);
+#pragma unroll
+        for (int e = 0; e < VW; ++e) v[e] = a[e] * scale + b[e];
+    };
     float inv = 1.f;
     if (norm_w) {                                             // x / sqrt(mean(x^2) + eps) * w on the scaled row
         float ss = 0.f;
-        for (int c = threadIdx.x; c < D; c += blockDim.x) {
-            const float v = value(c);
-            ss = fmaf(v, v, ss);
+        for (int c = threadIdx.x * VW; c < D; c += blockDim.x * VW) {
+            float v[VW];
+            value(c, v);
+#pragma unroll
+            for (int e = 0; e < VW; ++e) ss = fmaf(v[e], v[e], ss);
         }
         inv = 1.0f / sqrtf(block_sum(ss, red) / (float)D + eps);
     }
-    for (int c = threadIdx.x; c < D; c += blockDim.x) {
-        float v = value(c);
-        if (norm_w) v = v * inv * norm_w[c];
-        for (int j = 0; j < streams; ++j) X[((size_t)r * streams + j) * D + c] = v;
-        if (Xb) Xb[(size_t)r * D + c] = __float2bfloat16_rn(v);
+    for (int c = threadIdx.x * VW; c < D; c += blockDim.x * VW) {
+        float v[VW];
+        value(c, v);
+        if (norm_w) {
+#pragma unroll
+            for (int e = 0; e < VW; ++e) v[e] = v[e] * inv * norm_w[c + e];
+        }
+        for (int j = 0; j < streams; ++j) {
+            float* x = X + ((size_t)r * streams + j) * D + c;
+            if (VW == 8) {
+                reinterpret_cast<float4*>(x)[0] = make_float4(v[0], v[1 % VW], v[2 % VW], v[3 % VW]);
+                reinterpret_cast<float4*>(x)[1] = make_float4(v[4 % VW], v[5 % VW], v[6 % VW], v[7 % VW]);
+            } else {
+                *x = v[0];
+            }
+        }
+        if (Xb) {
+            __nv_bfloat16* xb = Xb + (size_t)r * D + c;
+            if (VW == 8) {
+                uint4 t;
+                __nv_bfloat162* q = reinterpret_cast<__nv_bfloat162*>(&t);
+#pragma unroll
+                for (int e = 0; e < VW / 2; ++e) q[e] = __floats2bfloat162_rn(v[2 * e], v[(2 * e + 1) % VW]);
+                *reinterpret_cast<uint4*>(xb) = t;
+            } else {
+                *xb = __float2bfloat16_rn(v[0]);
+            }
+        }
     }
 }
 
@@ -651,7 +697,10 @@ mlstm_finish_kernel(const float* __restrict__ raw, int ldr, const float* __restr
 cudaError_t launch_streams_embed(const void* table, const int* ids, float scale, float* X, int streams, int M, int V, int D,
                                  cudaStream_t st, const float* norm_w, float eps, const BigramRows& bg, void* x_bf16) {
     if ((x_bf16 && streams != 1) || (bg.table && (bg.buckets <= 0 || !bg.token_pages))) return cudaErrorInvalidValue;
-    return launch_pdl(streams_embed_kernel, dim3(M), dim3(128), 0, st, reinterpret_cast<const __nv_bfloat16*>(table), ids, scale,
+    auto aligned = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+    const bool vec = D % 8 == 0 && aligned(table) && aligned(bg.table) && aligned(X) && aligned(x_bf16);
+    const int threads = vec ? std::min(256, ((D / 8 + 31) / 32) * 32) : 128;
+    return launch_pdl(vec ? streams_embed_kernel<8> : streams_embed_kernel<1>, dim3(M), dim3(threads), 0, st, reinterpret_cast<const __nv_bfloat16*>(table), ids, scale,
                       norm_w, eps, X, reinterpret_cast<__nv_bfloat16*>(x_bf16), streams, V, D, bg);
 }
 
