@@ -674,18 +674,20 @@ def test_drawn_configurations_whole_portioned_and_decoded(seed):
 
 # ---- generation through the scheduler, the registry and the command line ---------------------------------------------------
 def test_greedy_generation_through_the_scheduler():
-    cfg = small_config()
+    # a small embedding beside large sublayer outputs: logits against the table itself would otherwise repeat the last token
+    cfg = small_config(residual_mult=1.6, embedding={"scale": 0.8, "bigram": dict(BIGRAM)})
     model, w = build(cfg, 17, max_tokens=400, max_sequences=3, max_rows=24)
     prompts = [tokens(cfg, 37, 20), tokens(cfg, 5, 21), tokens(cfg, 1, 22), tokens(cfg, 50, 23), tokens(cfg, 18, 24)]
     outs = model.generate(prompts, max_new_tokens=10, max_step_tokens=24)      # 5 requests over 3 slots, portioned prompts
     assert model.state.free_slots == 3 and model.state.free_pages == model.state.n_pages
     for p, o in zip(prompts, outs):
-        assert len(o) == 10
+        assert len(o) == 10 and len(set(o)) >= 2
         ref = O.forward(cfg, w, p + o[:-1])[len(p) - 1:]
         top2 = torch.topk(ref, 2, dim=-1)
         for t, tok in enumerate(o):
             if tok != int(top2.indices[t, 0]):                 # only an exact near-tie may go the other way
                 assert tok == int(top2.indices[t, 1]) and float(top2.values[t, 0] - top2.values[t, 1]) < 1e-4
+    assert len({t for o in outs for t in o}) >= 8
     assert model.generate(prompts[:2], max_new_tokens=10) == outs[:2]
 
 
